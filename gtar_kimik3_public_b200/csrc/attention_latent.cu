@@ -32,12 +32,12 @@ __global__ void __launch_bounds__(PREP_THREADS) latent_prepare_kernel(
     const float* __restrict__ cos_table, const float* __restrict__ sin_table, const int* __restrict__ tok_pos,
     const int* __restrict__ tok_seq, const int* __restrict__ slots, const int* __restrict__ block_table,
     T* __restrict__ q_latent, T* __restrict__ pages, int q_rank, int rank, int rot, int rot_dims, int max_pages,
-    int page_size) {
+    int page_size, long long ld) {
     __shared__ float scratch[33];
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
-    const T* row = proj + (size_t)t * (q_rank + rank + rot);
+    const T* row = proj + (size_t)t * ld;
     // the q latent
     float ss = 0.f;
     for (int i = threadIdx.x; i < q_rank; i += PREP_THREADS) {
@@ -178,19 +178,20 @@ GK_EXPORT int gk_latent_prepare(const void* proj, int dtype, const float* w_q, c
                                 const float* cos_table, const float* sin_table, const int* tok_pos, const int* tok_seq,
                                 const int* slots, const int* block_table, void* q_latent, void* pages, int n_tokens,
                                 int q_rank, int rank, int rot, int rot_dims, int max_pages, int page_size, int max_position,
-                                int table_rows, void* stream) {
+                                int table_rows, long long ld, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(dtype), "latent_prepare: bad dtype %d", dtype);
     GK_REQUIRE(n_tokens >= 0 && q_rank > 0 && rank > 0 && rot >= 0, "latent_prepare: bad sizes");
     GK_REQUIRE(rot_dims >= 0 && rot_dims <= rot && rot_dims % 2 == 0, "latent_prepare: %d of %d entries cannot turn in pairs",
                rot_dims, rot);
     GK_REQUIRE(rot_dims == 0 || (cos_table && sin_table && table_rows > max_position),
                "latent_prepare: the rotation tables hold %d positions, the step reaches %d", table_rows, max_position);
+    GK_REQUIRE(ld >= q_rank + rank + rot, "latent_prepare: rows of %lld are shorter than %d + %d + %d", ld, q_rank, rank, rot);
     GK_REQUIRE(eps > 0.f, "latent_prepare: eps must be positive");
     if (n_tokens == 0) return GK_OK;
     GK_DISPATCH_DTYPE(dtype, T, {
         gk_launch(latent_prepare_kernel<T>, dim3(n_tokens), dim3(PREP_THREADS), 0, (cudaStream_t)stream, (const T*)proj, w_q,
                   w_kv, eps, cos_table, sin_table, tok_pos, tok_seq, slots, block_table, (T*)q_latent, (T*)pages, q_rank, rank,
-                  rot, rot_dims, max_pages, page_size);
+                  rot, rot_dims, max_pages, page_size, ld);
     })
     GK_CHECK_LAUNCH("latent_prepare");
     return GK_OK;

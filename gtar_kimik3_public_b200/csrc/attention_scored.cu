@@ -12,6 +12,7 @@
 //                the sequence's first position
 //   temp:        a number per query head on the product:  (q . k_j) * scale * temp_h
 //   dist_bias:   a table [n_dist, n_q] of terms ADDED to the score, read at row min(i - j, n_dist - 1)
+//   softcap > 0: the product so far becomes softcap * tanh(product / softcap), before any distance term
 //   sink:        a number per query head whose exponential joins the softmax's denominator (and nothing else):
 //                weights_j = exp(s_j) / (exp(sink_h) + sum_visible exp(s))
 //
@@ -74,7 +75,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_scored_kernel(
     const int* __restrict__ block_table, int n_tokens, int n_q, int n_kv, int d, int dv, int max_pages, int page_size,
     float scale, int window, int keep_first, const float* __restrict__ r1, const float* __restrict__ r2,
     const float* __restrict__ head_bias, int chunk, const float* __restrict__ temp, const float* __restrict__ dist_bias,
-    int n_dist, const float* __restrict__ sink) {
+    int n_dist, const float* __restrict__ sink, float softcap) {
     extern __shared__ float q_smem[];  // WARPS * d
     pdl_launch_dependents();
     pdl_wait();
@@ -121,6 +122,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_scored_kernel(
         float s = -INFINITY;
         if (valid) {
             s = dot_row<T>(qs, k_pages + (row0 + lane) * d, d) * scale;
+            if (softcap > 0.f) s = softcap * tanhf(s / softcap);
             if (biased) s -= b1 * log1pf(b2 * (float)(pos - j));
             if (dist_bias != nullptr) s += dist_bias[(size_t)min(pos - j, n_dist - 1) * n_q + hq];
         }
@@ -165,7 +167,7 @@ GK_EXPORT int gk_attention_scored_exact(const void* q, const void* k_pages, cons
                                         int n_tokens, int n_q, int n_kv, int d, int dv, int max_pages, int page_size, float scale,
                                         int window, int keep_first, const float* r1, const float* r2, const float* head_bias,
                                         int weights, int chunk, const float* temp, const float* dist_bias, int n_dist,
-                                        const float* sink, void* stream) {
+                                        const float* sink, float softcap, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(dtype), "attention_scored: bad dtype %d", dtype);
     GK_REQUIRE(n_tokens >= 0 && n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_scored: bad head counts %d/%d", n_q, n_kv);
     GK_REQUIRE(d > 0 && dv > 0 && dv <= 32 * MAX_ACC, "attention_scored: keys of %d must be positive, values of %d at most %d", d, dv,
@@ -176,6 +178,7 @@ GK_EXPORT int gk_attention_scored_exact(const void* q, const void* k_pages, cons
     GK_REQUIRE(weights == 0 || weights == 1, "attention_scored: weights are softmax (0) or sigmoid (1)");
     GK_REQUIRE(chunk >= 0 && (dist_bias == nullptr || n_dist > 0), "attention_scored: bad chunk or distance table");
     GK_REQUIRE(sink == nullptr || weights == 0, "attention_scored: a sink belongs to the softmax");
+    GK_REQUIRE(softcap >= 0.f && (softcap == 0.f || weights == 0), "attention_scored: capped scores belong to the softmax");
     if (n_tokens == 0) return GK_OK;
     const long long warps = (long long)n_tokens * n_q;
     const long long blocks = (warps + WARPS - 1) / WARPS;
@@ -186,11 +189,11 @@ GK_EXPORT int gk_attention_scored_exact(const void* q, const void* k_pages, cons
         if (weights == 1)
             gk_launch(attention_scored_kernel<T, true>, dim3((unsigned)blocks), dim3(WARPS * 32), smem, s, (const T*)q, (const T*)k_pages,
                       (const T*)v_pages, (T*)out, tok_pos, tok_seq, slots, block_table, n_tokens, n_q, n_kv, d, dv, max_pages, page_size,
-                      scale, window, keep_first, r1, r2, head_bias, chunk, temp, dist_bias, n_dist, sink);
+                      scale, window, keep_first, r1, r2, head_bias, chunk, temp, dist_bias, n_dist, sink, softcap);
         else
             gk_launch(attention_scored_kernel<T, false>, dim3((unsigned)blocks), dim3(WARPS * 32), smem, s, (const T*)q, (const T*)k_pages,
                       (const T*)v_pages, (T*)out, tok_pos, tok_seq, slots, block_table, n_tokens, n_q, n_kv, d, dv, max_pages, page_size,
-                      scale, window, keep_first, r1, r2, head_bias, chunk, temp, dist_bias, n_dist, sink);
+                      scale, window, keep_first, r1, r2, head_bias, chunk, temp, dist_bias, n_dist, sink, softcap);
     })
     GK_CHECK_LAUNCH("attention_scored");
     return GK_OK;

@@ -7,7 +7,8 @@
 // and, each only where its argument is given: keys of the token's own chunk only (chunks of `chunk` positions counted
 // from the sequence's start), a number per query head on the product (temp), a table [n_dist, n_q] of terms added to
 // the score by distance (row min(i - j, n_dist - 1)), a number per query head whose exponential joins the softmax's
-// denominator and carries no value (sink).
+// denominator and carries no value (sink), and a cap on the product, softcap * tanh(product / softcap), before any distance
+// term.
 //
 // The rows of a block's tile are (token, query head of one kv group) pairs, token-major, so the query heads that
 // share a kv head share every loaded page; a warp owns 16 rows and K and V pages stream through a three-stage
@@ -44,17 +45,24 @@ __device__ __forceinline__ float lg2_fast(float x) {
     return y;
 }
 
-// MORE: which of the further rules are compiled in: 0 none, 1 the sink alone, 2 the chunk, the head temperature, the
-// distance table and the sink.  Without them the kernel is the windowed one alone and keeps its registers (a third block
+// cap * tanh(t / cap) for a score in the base-2 domain, t2 = t log2(e), and its result in that domain again:
+// tanh(x) = 1 - 2 / (1 + e^(2x)); two_by_cap = 2 / cap, cap2 = cap log2(e).  The hardware's exponential and division: the
+// result is off by about 3e-7 of the cap.
+__device__ __forceinline__ float soft_limit2(float t2, float two_by_cap, float cap2) {
+    return cap2 - __fdividef(2.f * cap2, 1.f + exp2_fast(t2 * two_by_cap));
+}
+
+// CAP: the cap on the scores is compiled in.  MORE: which of the further rules are: 0 none, 1 the sink alone, 2 the chunk,
+// the head temperature, the distance table and the sink.  Without them the kernel is the windowed one alone and keeps its registers (a third block
 // a multiprocessor at heads of 64); the sink alone costs none.
-template <int D, bool SIGMOID, int MORE>
+template <int D, bool SIGMOID, int MORE, bool CAP>
 __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0) attention_scored_mma_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages, const __nv_bfloat16* __restrict__ v_pages,
     __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ cu_q,
     const int* __restrict__ kv_len, const int* __restrict__ slots, const int* __restrict__ block_table, int n_tokens, int n_q,
     int n_kv, int max_pages, float sl2, int window, int keep_first, const float* __restrict__ r1, const float* __restrict__ r2,
     const float* __restrict__ head_bias, int n_split, int chunk, const float* __restrict__ temp,
-    const float* __restrict__ dist_bias, int n_dist, const float* __restrict__ sink) {
+    const float* __restrict__ dist_bias, int n_dist, const float* __restrict__ sink, float two_by_cap, float cap2) {
     constexpr bool RULES = MORE == 2;
     extern __shared__ __align__(128) unsigned char smem_raw[];
     ScoredSmem<D>& sm = *reinterpret_cast<ScoredSmem<D>*>(smem_raw);
@@ -179,6 +187,7 @@ __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0)
                         const int gap = pos[h] - key;
                         const bool hidden = gap < 0 || (window > 0 && gap >= window && key >= keep_first) || (RULES && key < first[h]);
                         float t = s[n][2 * h + c] * (RULES ? sl2h[h] : sl2);
+                        if (CAP) t = soft_limit2(t, two_by_cap, cap2);
                         if (biased) t -= b1[h] * lg2_fast(fmaf(b2[h], (float)max(gap, 0), 1.f));
                         if (RULES && dist_bias != nullptr)
                             t = fmaf(__ldg(dist_bias + (size_t)min(max(gap, 0), n_dist - 1) * n_q + head[h]), LOG2E, t);
@@ -259,26 +268,26 @@ __global__ void __launch_bounds__(128) attention_scored_join_kernel(const float*
     for (int c = 0; c < D / 32; ++c) out[(size_t)item * D + lane + 32 * c] = __float2bfloat16(acc[c] * inv);
 }
 
-template <int D, bool SIGMOID, int MORE>
+template <int D, bool SIGMOID, int MORE, bool CAP>
 int launch_scored(const void* q, const void* k_pages, const void* v_pages, void* out, float* part_o, float* part_ml, const int* cu_q,
                   const int* kv_len, const int* slots, const int* block_table, int n_seqs, int max_q_len, int n_tokens, int n_q,
                   int n_kv, int max_pages, float scale, int window, int keep_first, const float* r1, const float* r2,
                   const float* head_bias, int n_split, int chunk, const float* temp, const float* dist_bias, int n_dist,
-                  const float* sink, cudaStream_t stream) {
+                  const float* sink, float softcap, cudaStream_t stream) {
     const size_t smem = sizeof(ScoredSmem<D>);
     static bool configured = false;
     if (!configured) {
-        cudaError_t err = cudaFuncSetAttribute(attention_scored_mma_kernel<D, SIGMOID, MORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t err = cudaFuncSetAttribute(attention_scored_mma_kernel<D, SIGMOID, MORE, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (err != cudaSuccess) return gk_fail(GK_CUDA_ERROR, "attention_scored_mma: %s", cudaGetErrorString(err));
         configured = true;
     }
     const int group = n_q / n_kv;
     const long long blocks = (((long long)max_q_len * group + SC_ROWS - 1) / SC_ROWS) * n_split;
     GK_REQUIRE(blocks <= 2147483647LL, "attention_scored_mma: too many rows");
-    gk_launch(attention_scored_mma_kernel<D, SIGMOID, MORE>, dim3((unsigned)blocks, n_kv, n_seqs), dim3(SC_WARPS * 32), smem, stream,
+    gk_launch(attention_scored_mma_kernel<D, SIGMOID, MORE, CAP>, dim3((unsigned)blocks, n_kv, n_seqs), dim3(SC_WARPS * 32), smem, stream,
               (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, (__nv_bfloat16*)out, part_o, part_ml,
               cu_q, kv_len, slots, block_table, n_tokens, n_q, n_kv, max_pages, scale * LOG2E, window, keep_first, r1, r2, head_bias,
-              n_split, chunk, temp, dist_bias, n_dist, sink);
+              n_split, chunk, temp, dist_bias, n_dist, sink, CAP ? 2.f / softcap : 0.f, softcap * LOG2E);
     GK_CHECK_LAUNCH("attention_scored_mma");
     if (n_split > 1) {
         const long long items = (long long)n_tokens * n_q;
@@ -300,7 +309,7 @@ GK_EXPORT int gk_attention_scored_bf16(const void* q, const void* k_pages, const
                                        int n_seqs, int max_q_len, int n_tokens, int n_q, int n_kv, int head_dim, int max_pages,
                                        int page_size, float scale, int window, int keep_first, const float* r1, const float* r2,
                                        const float* head_bias, int weights, int n_split, int chunk, const float* temp,
-                                       const float* dist_bias, int n_dist, const float* sink, void* stream) {
+                                       const float* dist_bias, int n_dist, const float* sink, float softcap, void* stream) {
     GK_REQUIRE(n_seqs >= 0 && n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_scored_mma: bad head counts %d/%d", n_q, n_kv);
     GK_REQUIRE(page_size == attn::PAGE, "attention_scored_mma: page_size must be %d, got %d", attn::PAGE, page_size);
     GK_REQUIRE(head_dim == 64 || head_dim == 128, "attention_scored_mma: head size %d is not 64 or 128 (use the exact kernel)", head_dim);
@@ -312,28 +321,36 @@ GK_EXPORT int gk_attention_scored_bf16(const void* q, const void* k_pages, const
                "attention_scored_mma: %d parts need their workspaces", n_split);
     GK_REQUIRE(chunk >= 0 && (dist_bias == nullptr || n_dist > 0), "attention_scored_mma: bad chunk or distance table");
     GK_REQUIRE(sink == nullptr || weights == 0, "attention_scored_mma: a sink belongs to the softmax");
+    GK_REQUIRE(softcap >= 0.f && (softcap == 0.f || weights == 0), "attention_scored_mma: capped scores belong to the softmax");
     if (n_seqs == 0 || max_q_len == 0 || n_tokens == 0) return GK_OK;
     cudaStream_t s = (cudaStream_t)stream;
     const int more = (chunk > 0 || temp != nullptr || dist_bias != nullptr) ? 2 : sink != nullptr ? 1 : 0;
-#define GK_SCORED(D, SIG)                                                                                                             \
-    do {                                                                                                                              \
-        if (more == 2)                                                                                                                \
-            return launch_scored<D, SIG, 2>(q, k_pages, v_pages, out, part_o, part_ml, cu_q, kv_len, slots, block_table, n_seqs,      \
-                                            max_q_len, n_tokens, n_q, n_kv, max_pages, scale, window, keep_first, r1, r2,             \
-                                            head_bias, n_split, chunk, temp, dist_bias, n_dist, sink, s);                             \
-        if (more == 1)                                                                                                                \
-            return launch_scored<D, SIG, 1>(q, k_pages, v_pages, out, part_o, part_ml, cu_q, kv_len, slots, block_table, n_seqs,      \
-                                            max_q_len, n_tokens, n_q, n_kv, max_pages, scale, window, keep_first, r1, r2,             \
-                                            head_bias, n_split, chunk, temp, dist_bias, n_dist, sink, s);                             \
-        return launch_scored<D, SIG, 0>(q, k_pages, v_pages, out, part_o, part_ml, cu_q, kv_len, slots, block_table, n_seqs,      \
-                                            max_q_len, n_tokens, n_q, n_kv, max_pages, scale, window, keep_first, r1, r2, head_bias,  \
-                                            n_split, chunk, temp, dist_bias, n_dist, sink, s);                                        \
+#define GK_SCORED_AS(D, SIG, MORE, CAP)                                                                                              \
+    return launch_scored<D, SIG, MORE, CAP>(q, k_pages, v_pages, out, part_o, part_ml, cu_q, kv_len, slots, block_table, n_seqs,     \
+                                            max_q_len, n_tokens, n_q, n_kv, max_pages, scale, window, keep_first, r1, r2, head_bias, \
+                                            n_split, chunk, temp, dist_bias, n_dist, sink, softcap, s)
+#define GK_SCORED(D, SIG)                              \
+    do {                                               \
+        if (more == 2) GK_SCORED_AS(D, SIG, 2, false); \
+        if (more == 1) GK_SCORED_AS(D, SIG, 1, false); \
+        GK_SCORED_AS(D, SIG, 0, false);                \
     } while (0)
+#define GK_CAPPED(D)                                    \
+    do {                                                \
+        if (more == 2) GK_SCORED_AS(D, false, 2, true); \
+        GK_SCORED_AS(D, false, 1, true);                \
+    } while (0)
+    if (softcap > 0.f) {
+        if (head_dim == 64) GK_CAPPED(64);
+        GK_CAPPED(128);
+    }
     if (head_dim == 64) {
         if (weights == 1) GK_SCORED(64, true);
         GK_SCORED(64, false);
     }
     if (weights == 1) GK_SCORED(128, true);
     GK_SCORED(128, false);
+#undef GK_CAPPED
 #undef GK_SCORED
+#undef GK_SCORED_AS
 }

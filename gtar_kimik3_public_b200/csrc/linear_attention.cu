@@ -3,7 +3,8 @@
 //   heads_prepare:  a warp per (token, head) of the packed projection q | k | v: optional SiLU (on q and k, on v),
 //                   rotation by position of the first `rot` entries of a q or k head (entry i paired with i + rot/2;
 //                   cosines and sines from tables of rot/2 angles a position), then optional division of a q or k
-//                   head by its root mean square (eps inside the root, no weight), then a constant on k.  With flag 8
+//                   head by its root mean square (eps inside the root; times a weight per entry that all query heads or all
+//                   key heads share, where one is given), then a constant on k.  With flag 8
 //                   every value head turns by its own position over ALL of its dv entries (entry m paired with
 //                   m + dv/2, tables of dv/2 angles a position of their own), so that it is cached turned.  The results
 //                   go either to 32-bit arrays q, k [T, heads, d] and v [T, heads, dv] (what a recurrence reads), or
@@ -11,8 +12,9 @@
 //   decay_scan:     per (sequence, head):  S <- decay_h S + k_t v_t^T ;  o_t = S^T q_t,  S [d, dv] 32-bit, read from
 //                   the sequence's slot at the start of the step and written back at its end.  Prompts, portions and
 //                   single tokens take the same path; a token's sums have the same order in all of them.
-//   group_norm_gate: rows cut into groups (a head, or all heads together) that are divided by their root mean
-//                   square, multiplied by an optional weight and by sigmoid or SiLU of a gate.
+//   group_norm_gate: rows cut into groups (a head, or all heads together), each first divided by a number of its own
+//                   where one is given, that are divided by their root mean square, multiplied by an optional weight (one
+//                   for all groups of a row, or one for the whole row) and by sigmoid or SiLU of a gate.
 //
 // Everything is 32-bit except the projection that is read and the activations that are handed on.
 
@@ -31,7 +33,8 @@ template <typename T, typename TQ>
 __global__ void __launch_bounds__(PREP_WARPS * 32) heads_prepare_kernel(
     const T* __restrict__ proj, long long ld, int q_at, int k_at, int v_at, int n_q, int n_k, int d, int dv, int flags,
     int rot, const float* __restrict__ cos_t, const float* __restrict__ sin_t, const float* __restrict__ v_cos,
-    const float* __restrict__ v_sin, float unit_eps, float k_scale, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ slots,
+    const float* __restrict__ v_sin, float unit_eps, const float* __restrict__ w_q, const float* __restrict__ w_k, float k_scale,
+    const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ slots,
     TQ* __restrict__ q_out, float* __restrict__ k_out, float* __restrict__ v_out, T* __restrict__ k_pages,
     T* __restrict__ v_pages, const int* __restrict__ block_table, int max_pages, int page_size, int write_kv, long long n_items) {
     extern __shared__ float stage[];  // PREP_WARPS * max(d, dv)
@@ -88,6 +91,12 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) heads_prepare_kernel(
             const float r = 1.0f / sqrtf(ss / (float)d + unit_eps);
 #pragma unroll
             for (int c = 0; c < PREP_MAX; ++c) x[c] *= r;
+            const float* w = kind == 0 ? w_q : w_k;
+            if (w != nullptr) {
+#pragma unroll
+                for (int c = 0; c < PREP_MAX; ++c)
+                    if (lane + 32 * c < width) x[c] *= w[lane + 32 * c];
+            }
         }
         if (kind == 1 && k_scale != 1.f) {
 #pragma unroll
@@ -257,7 +266,8 @@ __global__ void __launch_bounds__(SCAN_LANES * SCAN_MAX_COLS) decay_scan_kernel(
 
 // gate_kind: 0 sigmoid, 1 SiLU
 template <typename T, typename TG>
-__global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ weight,
+__global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ divisor,
+                                                              const float* __restrict__ weight, int row_weight,
                                                               const TG* __restrict__ gate, long long ld_gate, T* __restrict__ out,
                                                               long long n_rows, int n_groups, int size, float eps, int gate_kind) {
     pdl_launch_dependents();
@@ -271,7 +281,10 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
     float ss = 0.f;
     for (int i = lane; i < size; i += 32) ss = fmaf(xr[i], xr[i], ss);
     ss = warp_sum(ss);
-    const float r = 1.f / sqrtf(ss / (float)size + eps);
+    // a group divided by c first: x / c has the mean square ss / c^2
+    const float c = divisor != nullptr ? 1.f / divisor[row] : 1.f;
+    const float r = c / sqrtf(ss * c * c / (float)size + eps);
+    if (weight != nullptr && row_weight) weight += (size_t)g * size;
     const TG* gt = gate + (size_t)t * ld_gate + (size_t)g * size;
     for (int i = lane; i < size; i += 32) {
         const float z = to_float(gt[i]);
@@ -283,7 +296,8 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
 
 // The same for wide groups, a block per row: a warp alone would walk a row of a thousand entries in 32 dependent rounds.
 template <typename T, typename TG>
-__global__ void __launch_bounds__(256) group_norm_gate_wide_kernel(const float* __restrict__ x, const float* __restrict__ weight,
+__global__ void __launch_bounds__(256) group_norm_gate_wide_kernel(const float* __restrict__ x, const float* __restrict__ divisor,
+                                                                   const float* __restrict__ weight, int row_weight,
                                                                    const TG* __restrict__ gate, long long ld_gate, T* __restrict__ out,
                                                                    int n_groups, int size, float eps, int gate_kind) {
     __shared__ float scratch[33];
@@ -296,7 +310,10 @@ __global__ void __launch_bounds__(256) group_norm_gate_wide_kernel(const float* 
     float ss = 0.f;
     for (int i = threadIdx.x; i < size; i += 256) ss = fmaf(xr[i], xr[i], ss);
     ss = block_sum(ss, scratch);
-    const float r = 1.f / sqrtf(ss / (float)size + eps);
+    // a group divided by c first: x / c has the mean square ss / c^2
+    const float c = divisor != nullptr ? 1.f / divisor[row] : 1.f;
+    const float r = c / sqrtf(ss * c * c / (float)size + eps);
+    if (weight != nullptr && row_weight) weight += (size_t)g * size;
     const TG* gt = gate + (size_t)t * ld_gate + (size_t)g * size;
     for (int i = threadIdx.x; i < size; i += 256) {
         const float z = to_float(gt[i]);
@@ -310,7 +327,7 @@ __global__ void __launch_bounds__(256) group_norm_gate_wide_kernel(const float* 
 
 GK_EXPORT int gk_heads_prepare(const void* proj, int dtype, long long ld, int q_at, int k_at, int v_at, int n_q, int n_k, int d,
                                int dv, int flags, int rot, const float* cos_t, const float* sin_t, const float* v_cos,
-                               const float* v_sin, float unit_eps, float k_scale, const int* tok_pos, const int* tok_seq, const int* slots, void* q_out, int q_dtype, float* k_out,
+                               const float* v_sin, float unit_eps, const float* w_q, const float* w_k, float k_scale, const int* tok_pos, const int* tok_seq, const int* slots, void* q_out, int q_dtype, float* k_out,
                                float* v_out, void* k_pages, void* v_pages, const int* block_table, int max_pages, int page_size,
                                int write_kv, int n_tokens, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(dtype) && GK_VALID_DTYPE(q_dtype), "heads_prepare: bad dtype");
@@ -319,6 +336,7 @@ GK_EXPORT int gk_heads_prepare(const void* proj, int dtype, long long ld, int q_
     GK_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= d, "heads_prepare: %d rotated entries in heads of %d", rot, d);
     GK_REQUIRE(rot == 0 || (cos_t != nullptr && sin_t != nullptr), "heads_prepare: a rotation needs its tables");
     GK_REQUIRE(!(flags & 4) || unit_eps > 0.f, "heads_prepare: eps must be positive");
+    GK_REQUIRE((w_q == nullptr && w_k == nullptr) || (flags & 4), "heads_prepare: weights belong to the norm of a head");
     GK_REQUIRE(!(flags & 8) || (v_cos != nullptr && v_sin != nullptr && dv % 2 == 0),
                "heads_prepare: turned values need their tables and an even size");
     const bool to_pages = k_pages != nullptr;
@@ -334,11 +352,11 @@ GK_EXPORT int gk_heads_prepare(const void* proj, int dtype, long long ld, int q_
     GK_DISPATCH_DTYPE(dtype, T, {
         if (to_pages) {
             gk_launch(heads_prepare_kernel<T, T>, dim3((unsigned)blocks), dim3(PREP_WARPS * 32), smem, s, (const T*)proj, ld, q_at,
-                      k_at, v_at, n_q, n_k, d, dv, flags, rot, cos_t, sin_t, v_cos, v_sin, unit_eps, k_scale, tok_pos, tok_seq, slots, (T*)q_out,
+                      k_at, v_at, n_q, n_k, d, dv, flags, rot, cos_t, sin_t, v_cos, v_sin, unit_eps, w_q, w_k, k_scale, tok_pos, tok_seq, slots, (T*)q_out,
                       (float*)nullptr, (float*)nullptr, (T*)k_pages, (T*)v_pages, block_table, max_pages, page_size, write_kv, items);
         } else {
             gk_launch(heads_prepare_kernel<T, float>, dim3((unsigned)blocks), dim3(PREP_WARPS * 32), smem, s, (const T*)proj, ld,
-                      q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot, cos_t, sin_t, v_cos, v_sin, unit_eps, k_scale, tok_pos, tok_seq, slots,
+                      q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot, cos_t, sin_t, v_cos, v_sin, unit_eps, w_q, w_k, k_scale, tok_pos, tok_seq, slots,
                       (float*)q_out, k_out, v_out, (T*)nullptr, (T*)nullptr, block_table, max_pages, page_size, write_kv, items);
         }
     })
@@ -375,7 +393,7 @@ GK_EXPORT int gk_decay_scan(const float* q, const float* k, const float* v, cons
     return GK_OK;
 }
 
-GK_EXPORT int gk_group_norm_gate(const float* x, const float* weight, const void* gate, int gate_dtype, long long ld_gate, void* out,
+GK_EXPORT int gk_group_norm_gate(const float* x, const float* divisor, const float* weight, int row_weight, const void* gate, int gate_dtype, long long ld_gate, void* out,
                                  int out_dtype, long long n_tokens, int n_groups, int size, float eps, int gate_kind, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(gate_dtype) && GK_VALID_DTYPE(out_dtype), "group_norm_gate: bad dtype");
     GK_REQUIRE(n_groups > 0 && size > 0 && eps > 0.f && (gate_kind == 0 || gate_kind == 1), "group_norm_gate: bad sizes");
@@ -388,10 +406,10 @@ GK_EXPORT int gk_group_norm_gate(const float* x, const float* weight, const void
     GK_DISPATCH_DTYPE(out_dtype, T, {
         GK_DISPATCH_DTYPE(gate_dtype, TG, {
             if (wide)
-                gk_launch(group_norm_gate_wide_kernel<T, TG>, dim3((unsigned)rows), dim3(256), 0, s, x, weight, (const TG*)gate, ld_gate,
+                gk_launch(group_norm_gate_wide_kernel<T, TG>, dim3((unsigned)rows), dim3(256), 0, s, x, divisor, weight, row_weight, (const TG*)gate, ld_gate,
                           (T*)out, n_groups, size, eps, gate_kind);
             else
-                gk_launch(group_norm_gate_kernel<T, TG>, dim3((unsigned)blocks), dim3(256), 0, s, x, weight, (const TG*)gate, ld_gate,
+                gk_launch(group_norm_gate_kernel<T, TG>, dim3((unsigned)blocks), dim3(256), 0, s, x, divisor, weight, row_weight, (const TG*)gate, ld_gate,
                           (T*)out, rows, n_groups, size, eps, gate_kind);
         })
     })

@@ -5,8 +5,10 @@
 //                two largest choice scores and only the experts of the best `keep` groups may be chosen.  The `top`
 //                largest choice scores among them are chosen (ties: the lower index); a chosen expert's weight is its s
 //                (without the correction) times a constant.
-//                With `logits` = 1 the score is the logit itself plus a stored bias, s = z + b (no sigmoid, choice by s),
+//                With the flag for logits the score is the logit itself plus a stored bias, s = z + b (no sigmoid, choice by s),
 //                and the chosen experts' weights are the softmax over the chosen scores alone, times the constant.
+//                Further rules (flags): s = softmax(z) over all experts; a group's score is its largest choice score; the
+//                chosen experts' s are divided by their sum (plus 1e-20) before the constant.
 //   experts_up   act[pair] = silu(W_gate[e] h_t) * (W_up[e] h_t) for every pair (token, chosen expert)
 //   experts_down out_t = add_t + sum over the token's pairs, in the order they were chosen, of weight * W_down[e] act[pair]
 //                (32-bit result: it is what goes into the residual stream)
@@ -67,10 +69,12 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_scores_kernel(const T*
         }
 }
 
+enum RouteFlags : int { ROUTE_LOGITS = 1, ROUTE_SOFTMAX = 2, ROUTE_GROUP_BEST = 4, ROUTE_RENORMALISE = 8 };
+
 // The choice from the scores: one warp per token.
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_choose_kernel(
     const float* __restrict__ z, const float* __restrict__ correction, int* __restrict__ ids, float* __restrict__ weights,
-    int n_tokens, int n_experts, int top, int n_groups, int keep, float scale, int logits) {
+    int n_tokens, int n_experts, int top, int n_groups, int keep, float scale, int flags) {
     extern __shared__ float route_smem[];  // per warp: s [E] | choice [E] | group score [n_groups]
     pdl_launch_dependents();
     pdl_wait();
@@ -80,9 +84,17 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_choose_kernel(
     float* s = route_smem + (size_t)warp * (2 * n_experts + n_groups);
     float* choice = s + n_experts;
     float* group_score = choice + n_experts;
+    const bool logits = (flags & ROUTE_LOGITS) != 0, softmax = (flags & ROUTE_SOFTMAX) != 0;
+    float largest_z = -INFINITY, denom = 0.f;
+    if (softmax) {
+        for (int e = lane; e < n_experts; e += 32) largest_z = fmaxf(largest_z, z[(size_t)t * n_experts + e]);
+        largest_z = warp_max(largest_z);
+        for (int e = lane; e < n_experts; e += 32) denom += expf(z[(size_t)t * n_experts + e] - largest_z);
+        denom = warp_sum(denom);
+    }
     for (int e = lane; e < n_experts; e += 32) {
         const float ze = z[(size_t)t * n_experts + e];
-        const float sg = logits ? ze + correction[e] : 1.f / (1.f + expf(-ze));
+        const float sg = logits ? ze + correction[e] : softmax ? expf(ze - largest_z) / denom : 1.f / (1.f + expf(-ze));
         s[e] = sg;
         choice[e] = logits ? sg : sg + correction[e];
     }
@@ -96,7 +108,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_choose_kernel(
                 if (c > first) { second = first; first = c; }
                 else if (c > second) second = c;
             }
-            group_score[gidx] = per > 1 ? first + second : first;
+            group_score[gidx] = per > 1 && !(flags & ROUTE_GROUP_BEST) ? first + second : first;
         }
         __syncwarp();
         // the groups that are not among the best `keep` lose their experts
@@ -125,10 +137,16 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_choose_kernel(
         if (arg == 0x7fffffff) arg = 0;  // nothing left to choose from: cannot happen when top <= allowed experts
         if (lane == 0) {
             ids[(size_t)t * top + pick] = arg;
-            weights[(size_t)t * top + pick] = logits ? s[arg] : s[arg] * scale;
+            weights[(size_t)t * top + pick] = logits || (flags & ROUTE_RENORMALISE) ? s[arg] : s[arg] * scale;
             choice[arg] = -INFINITY;
         }
         __syncwarp();
+    }
+    if ((flags & ROUTE_RENORMALISE) && lane == 0) {
+        float* w = weights + (size_t)t * top;
+        float sum = 0.f;
+        for (int pick = 0; pick < top; ++pick) sum += w[pick];
+        for (int pick = 0; pick < top; ++pick) w[pick] = w[pick] / (sum + 1e-20f) * scale;
     }
     if (logits && lane == 0) {
         // softmax over the chosen scores, in the order they were chosen (the first is the largest)
@@ -387,7 +405,7 @@ GK_EXPORT int gk_experts_combine(const void* y, int dtype, const int* place_of, 
 }
 
 GK_EXPORT int gk_route_groups(const void* h, int dtype, const float* w_router, const float* correction, float* z, int* ids,
-                              float* weights, int n_tokens, int width, int n_experts, int top, int n_groups, int keep, float scale, int logits,
+                              float* weights, int n_tokens, int width, int n_experts, int top, int n_groups, int keep, float scale, int flags,
                               void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(dtype), "route_groups: bad dtype %d", dtype);
     GK_REQUIRE(n_experts > 0 && top > 0 && top <= n_experts, "route_groups: %d of %d experts", top, n_experts);
@@ -395,6 +413,7 @@ GK_EXPORT int gk_route_groups(const void* h, int dtype, const float* w_router, c
                n_groups, keep, n_experts);
     GK_REQUIRE(top <= keep * (n_experts / n_groups), "route_groups: %d experts cannot come from %d groups of %d", top, keep,
                n_experts / n_groups);
+    GK_REQUIRE(!(flags & ROUTE_LOGITS) || !(flags & (ROUTE_SOFTMAX | ROUTE_RENORMALISE)), "route_groups: logits have a rule of their own");
     if (n_tokens == 0) return GK_OK;
     const size_t smem = (size_t)ROUTE_WARPS * (2 * n_experts + n_groups) * sizeof(float);
     GK_REQUIRE(smem <= 48 * 1024, "route_groups: too many experts (%d)", n_experts);
@@ -413,7 +432,7 @@ GK_EXPORT int gk_route_groups(const void* h, int dtype, const float* w_router, c
     })
     GK_CHECK_LAUNCH("route_scores");
     gk_launch(route_choose_kernel, dim3((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, s, (const float*)z,
-              correction, ids, weights, n_tokens, n_experts, top, n_groups, keep, scale, logits);
+              correction, ids, weights, n_tokens, n_experts, top, n_groups, keep, scale, flags);
     GK_CHECK_LAUNCH("route_groups");
     return GK_OK;
 }

@@ -1136,13 +1136,13 @@ def gelu_tanh(x: torch.Tensor) -> torch.Tensor:
 def latent_prepare(proj: torch.Tensor, q_rank: int, rank: int, rot: int, rot_dims: int, w_q: torch.Tensor, w_kv: torch.Tensor,
                    eps: float, cos: torch.Tensor | None, sin: torch.Tensor | None, tok_pos: torch.Tensor, tok_seq: torch.Tensor,
                    slots: torch.Tensor, cache: PagedRows, max_position: int, write: bool = True) -> torch.Tensor:
-    """From the packed projection rows ``[q latent | kv latent | shared key part]``: returns the normed q latent
+    """From the packed projection rows ``[q latent | kv latent | shared key part]`` (more columns may follow): returns the normed q latent
     ``[n, q_rank]`` and writes each position's cache row (normed kv latent, rotated shared key part)."""
     require_device(proj.device)
     _check(proj, "proj", dims=2)
     n = proj.shape[0]
-    if proj.shape[1] != q_rank + rank + rot:
-        raise KernelError(f"projection rows of {proj.shape[1]} are not {q_rank} + {rank} + {rot}")
+    if proj.shape[1] < q_rank + rank + rot:
+        raise KernelError(f"projection rows of {proj.shape[1]} are shorter than {q_rank} + {rank} + {rot}")
     _check(w_q, "w_q", torch.float32, 1)
     _check(w_kv, "w_kv", torch.float32, 1)
     _check(cache.rows, "cache rows", proj.dtype, 3)
@@ -1158,7 +1158,8 @@ def latent_prepare(proj: torch.Tensor, q_rank: int, rank: int, rot: int, rot_dim
     out = torch.empty((n, q_rank), dtype=proj.dtype, device=proj.device)
     call("gk_latent_prepare", ptr(proj), dtype_code(proj.dtype), ptr(w_q), ptr(w_kv), float(eps), ptr(cos), ptr(sin),
          ptr(tok_pos), ptr(tok_seq), ptr(slots), ptr(cache.block_table), ptr(out), ptr(cache.rows) if write else None, n, q_rank,
-         rank, rot, rot_dims, cache.max_pages, cache.page_size, int(max_position), table_rows, stream_ptr())
+         rank, rot, rot_dims, cache.max_pages, cache.page_size, int(max_position), table_rows,
+         proj.shape[1], stream_ptr())
     return out
 
 
@@ -1350,11 +1351,14 @@ def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, ga
 
 # ------------------------------------------------------------------ routed experts
 def route_groups(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor, top: int, n_groups: int, keep: int,
-                 scale: float, logits: bool = False) -> tuple[torch.Tensor, torch.Tensor]:
+                 scale: float, logits: bool = False, softmax: bool = False, best_of_group: bool = False,
+                 renormalise: bool = False) -> tuple[torch.Tensor, torch.Tensor]:
     """Chosen experts ``[T, top]`` (int32) and their weights (float32): sigmoid scores, choice by score plus
     ``correction`` among the experts of the best ``keep`` of ``n_groups`` groups, weight = score times ``scale``.
     ``logits``: the score is the logit plus ``correction`` (a bias), the choice goes by it, and the weights are the
-    softmax over the chosen scores alone, times ``scale``."""
+    softmax over the chosen scores alone, times ``scale``.  ``softmax``: scores are the softmax of the logits over all experts;
+    ``best_of_group``: a group's score is its largest choice score (else its two largest added); ``renormalise``: the chosen
+    scores are divided by their sum plus 1e-20 before ``scale``."""
     require_device(h.device)
     _check(h, "h", dims=2)
     _check(w_router, "w_router", torch.float32, 2)
@@ -1367,7 +1371,7 @@ def route_groups(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tens
     weights = torch.empty((T, top), dtype=torch.float32, device=h.device)
     z = torch.empty((T, n_experts), dtype=torch.float32, device=h.device)
     call("gk_route_groups", ptr(h), dtype_code(h.dtype), ptr(w_router), ptr(correction), ptr(z), ptr(ids), ptr(weights), T, width, n_experts,
-         top, n_groups, keep, float(scale), int(bool(logits)), stream_ptr())
+         top, n_groups, keep, float(scale), bool(logits) + 2 * bool(softmax) + 4 * bool(best_of_group) + 8 * bool(renormalise), stream_ptr())
     return ids, weights
 
 
@@ -1645,12 +1649,13 @@ def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int,
                   tok_seq: torch.Tensor, slots: torch.Tensor, *, silu_qk: bool = False, silu_v: bool = False, rot: int = 0,
                   cos: torch.Tensor | None = None, sin: torch.Tensor | None = None, unit_eps: float | None = None,
                   k_scale: float = 1.0, kv: PagedKV | None = None, write_kv: bool = True, max_position: int | None = None,
-                  v_cos: torch.Tensor | None = None, v_sin: torch.Tensor | None = None):
+                  v_cos: torch.Tensor | None = None, v_sin: torch.Tensor | None = None, w_q: torch.Tensor | None = None,
+                  w_k: torch.Tensor | None = None):
     """What stands between a packed projection and a mixer's core.  ``proj [T, >= ...]`` holds ``n_q`` query heads of ``d``
     from column ``q_at``, ``n_k`` key heads of ``d`` from ``k_at`` and ``n_k`` value heads of ``dv`` from ``v_at``.  In this
     order: SiLU (``silu_qk`` on q and k, ``silu_v`` on v); rotation of the first ``rot`` entries of every q and k head by
     the token's position (entry ``i`` with ``i + rot/2``; ``cos``, ``sin`` ``[positions, rot/2]``); with ``unit_eps`` every q
-    and k head divided by its root mean square; ``k_scale`` on k; with ``v_cos``, ``v_sin`` ``[positions, dv/2]`` every
+    and k head divided by its root mean square (and multiplied by ``w_q [d]`` or ``w_k [d]`` where given); ``k_scale`` on k; with ``v_cos``, ``v_sin`` ``[positions, dv/2]`` every
     value head turned by its token's position over all of its entries (entry ``m`` with ``m + dv/2``).  With ``kv`` the keys and values are written into the
     cache's pages and q ``[T, n_q, d]`` comes back in the projection's type; without, q, k ``[T, n, d]`` and v ``[T, n_k,
     dv]`` come back as 32-bit arrays."""
@@ -1669,6 +1674,11 @@ def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int,
             raise KernelError(f"heads_prepare: tables of {cos.shape[1]} angles for {rot} rotated entries")
         if max_position is not None and cos.shape[0] <= max_position:
             raise KernelError(f"heads_prepare: tables hold {cos.shape[0]} positions, the step reaches {max_position}")
+    for name, t in (("w_q", w_q), ("w_k", w_k)):
+        if t is not None:
+            _check(t, name, torch.float32, 1)
+            if t.shape[0] != d or unit_eps is None:
+                raise KernelError(f"heads_prepare: {name} has {t.shape[0]} entries for the norm of heads of {d}")
     flags = (PREPARE_SILU_QK if silu_qk else 0) | (PREPARE_SILU_V if silu_v else 0) | (PREPARE_UNIT_RMS if unit_eps is not None else 0)
     if v_cos is not None:
         _check(v_cos, "v_cos", torch.float32, 2)
@@ -1686,7 +1696,7 @@ def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int,
             raise KernelError(f"heads_prepare: pages {tuple(kv.k.shape)} / {tuple(kv.v.shape)} do not hold {n_k} heads of {d} / {dv}")
         q = torch.empty((T, n_q, d), dtype=proj.dtype, device=dev)
         call("gk_heads_prepare", ptr(proj), dtype_code(proj.dtype), proj.shape[1], q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot,
-             ptr(cos) if rot else None, ptr(sin) if rot else None, ptr(v_cos), ptr(v_sin), float(unit_eps or 0.0), float(k_scale),
+             ptr(cos) if rot else None, ptr(sin) if rot else None, ptr(v_cos), ptr(v_sin), float(unit_eps or 0.0), ptr(w_q), ptr(w_k), float(k_scale),
              ptr(tok_pos), ptr(tok_seq), ptr(slots), ptr(q), dtype_code(q.dtype), None, None, ptr(kv.k), ptr(kv.v), ptr(kv.block_table), kv.max_pages,
              kv.page_size, int(write_kv), T, stream_ptr())
         return q
@@ -1694,7 +1704,7 @@ def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int,
     k = torch.empty((T, n_k, d), dtype=torch.float32, device=dev)
     v = torch.empty((T, n_k, dv), dtype=torch.float32, device=dev)
     call("gk_heads_prepare", ptr(proj), dtype_code(proj.dtype), proj.shape[1], q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot,
-         ptr(cos) if rot else None, ptr(sin) if rot else None, ptr(v_cos), ptr(v_sin), float(unit_eps or 0.0), float(k_scale),
+         ptr(cos) if rot else None, ptr(sin) if rot else None, ptr(v_cos), ptr(v_sin), float(unit_eps or 0.0), ptr(w_q), ptr(w_k), float(k_scale),
          ptr(tok_pos), ptr(tok_seq), ptr(slots), ptr(q), dtype_code(q.dtype), ptr(k), ptr(v), None, None, None, 0, 0, 0, T, stream_ptr())
     return q, k, v
 
@@ -1754,10 +1764,11 @@ def decay_scan_chunked(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay:
 
 
 def group_norm_gate(x: torch.Tensor, group: int, weight: torch.Tensor | None, gate: torch.Tensor, gate_at: int, eps: float,
-                    out_dtype: torch.dtype, gate_kind: str = "sigmoid") -> torch.Tensor:
+                    out_dtype: torch.dtype, gate_kind: str = "sigmoid", divisor: torch.Tensor | None = None) -> torch.Tensor:
     """Rows of ``x [T, width]`` (32-bit) cut into groups of ``group`` entries; every group divided by its root mean square
-    (eps inside the root), multiplied by ``weight [group]`` (if given) and by sigmoid or SiLU of
-    ``gate[:, gate_at : gate_at + width]``.  Returns ``[T, width]`` in ``out_dtype``."""
+    (eps inside the root), multiplied by ``weight`` (if given: ``[group]`` for every group alike, or ``[width]``) and by sigmoid or
+    SiLU of ``gate[:, gate_at : gate_at + width]``.  ``divisor [T, width / group]``: every group is divided by its own number
+    before its norm.  Returns ``[T, width]`` in ``out_dtype``."""
     require_device(x.device)
     _check(x, "x", torch.float32, 2)
     _check(gate, "gate", dims=2)
@@ -1766,11 +1777,15 @@ def group_norm_gate(x: torch.Tensor, group: int, weight: torch.Tensor | None, ga
         raise KernelError("group_norm_gate: the groups or the gate do not fit the rows")
     if weight is not None:
         _check(weight, "weight", torch.float32, 1)
-        if weight.shape[0] != group:
-            raise KernelError(f"group_norm_gate: a weight of {weight.shape[0]} for groups of {group}")
+        if weight.shape[0] not in (group, width):
+            raise KernelError(f"group_norm_gate: a weight of {weight.shape[0]} for groups of {group} in rows of {width}")
+    if divisor is not None:
+        _check(divisor, "divisor", torch.float32, 2)
+        if tuple(divisor.shape) != (T, width // group):
+            raise KernelError(f"group_norm_gate: divisors {tuple(divisor.shape)} for {width // group} groups a row")
     kinds = {"sigmoid": 0, "silu": 1}
     out = torch.empty((T, width), dtype=out_dtype, device=x.device)
-    call("gk_group_norm_gate", ptr(x), ptr(weight), gate.data_ptr() + gate_at * gate.element_size(), dtype_code(gate.dtype),
+    call("gk_group_norm_gate", ptr(x), ptr(divisor), ptr(weight), int(weight is not None and weight.shape[0] == width), gate.data_ptr() + gate_at * gate.element_size(), dtype_code(gate.dtype),
          gate.shape[1], ptr(out), dtype_code(out_dtype), T, width // group, group, float(eps), kinds[gate_kind], stream_ptr())
     return out
 
@@ -1779,13 +1794,15 @@ def attention_scored_exact(q: torch.Tensor, kv: PagedKV, tok_pos: torch.Tensor, 
                            scale: float, window: int = 0, keep_first: int = 0, r1: torch.Tensor | None = None,
                            r2: torch.Tensor | None = None, head_bias: torch.Tensor | None = None,
                            weights: str = "softmax", chunk: int = 0, temp: torch.Tensor | None = None,
-                           dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None) -> torch.Tensor:
+                           dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None,
+                           softcap: float = 0.0) -> torch.Tensor:
     """Causal grouped-query attention of ``q [T, n_q, d]`` over pages of keys ``[.., d]`` and values ``[.., dv]`` (exact
     kernel): a key at ``j`` is seen from ``i`` if ``i - j < window`` or ``j < keep_first``; the score is ``q . k * scale -
     r1_h ln(1 + r2_h (i - j))``; the weights are the softmax over the seen keys, or ``sigmoid(score + head_bias_h)``
     without a sum that divides.  ``chunk``: only keys of the token's own chunk of that many positions are seen; ``temp``
     ``[n_q]`` multiplies the product per head; ``dist_bias [n_dist, n_q]`` is added by distance (the last row for
-    every distance beyond); ``sink [n_q]`` joins the softmax's denominator as ``exp(sink_h)``.  Returns ``[T, n_q, dv]``."""
+    every distance beyond); ``sink [n_q]`` joins the softmax's denominator as ``exp(sink_h)``; ``softcap > 0``: the product
+    becomes ``softcap * tanh(product / softcap)`` before any distance term.  Returns ``[T, n_q, dv]``."""
     require_device(q.device)
     _check(q, "q", dims=3)
     n, n_q, d = q.shape
@@ -1806,7 +1823,7 @@ def attention_scored_exact(q: torch.Tensor, kv: PagedKV, tok_pos: torch.Tensor, 
     call("gk_attention_scored_exact", ptr(q), ptr(kv.k), ptr(kv.v), ptr(out), dtype_code(q.dtype), ptr(tok_pos), ptr(tok_seq),
          ptr(slots), ptr(kv.block_table), n, n_q, n_kv, d, dv, kv.max_pages, kv.page_size, float(scale), int(window),
          int(keep_first), ptr(r1), ptr(r2), ptr(head_bias), {"softmax": 0, "sigmoid": 1}[weights], int(chunk), ptr(temp),
-         ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], ptr(sink), stream_ptr())
+         ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], ptr(sink), float(softcap), stream_ptr())
     return out
 
 
@@ -1840,7 +1857,7 @@ def attention_scored(q: torch.Tensor, kv: PagedKV, cu_q: torch.Tensor, kv_len: t
                      scale: float, window: int = 0, keep_first: int = 0, r1: torch.Tensor | None = None,
                      r2: torch.Tensor | None = None, head_bias: torch.Tensor | None = None, weights: str = "softmax",
                      n_parts: int = 1, chunk: int = 0, temp: torch.Tensor | None = None, dist_bias: torch.Tensor | None = None,
-                     sink: torch.Tensor | None = None) -> torch.Tensor:
+                     sink: torch.Tensor | None = None, softcap: float = 0.0) -> torch.Tensor:
     """:func:`attention_scored_exact` on the tensor cores: bfloat16, keys and values of 64 or 128 entries both, pages of 64
     keys.  The new tokens ``q [n_tokens, n_q, d]`` are packed by sequence (``cu_q``), ``kv_len`` counts each sequence's
     cached tokens including them.  ``n_parts`` > 1 cuts every block's keys into that many blocks whose sums a second
@@ -1873,5 +1890,91 @@ def attention_scored(q: torch.Tensor, kv: PagedKV, cu_q: torch.Tensor, kv_len: t
     call("gk_attention_scored_bf16", ptr(q), ptr(kv.k), ptr(kv.v), ptr(out), ptr(part_o), ptr(part_ml), ptr(cu_q), ptr(kv_len),
          ptr(slots), ptr(kv.block_table), n_seqs, int(max_q_len), n, n_q, kv.k.shape[1], d, kv.max_pages, kv.page_size, float(scale),
          int(window), int(keep_first), ptr(r1), ptr(r2), ptr(head_bias), sigmoid, int(n_parts), int(chunk), ptr(temp),
-         ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], ptr(sink), stream_ptr())
+         ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], ptr(sink), float(softcap), stream_ptr())
     return out
+
+
+# ------------------------------------------------------------------ gated branches, PolyNorm, matrix memory
+def gated_merge(h: torch.Tensor, dtype: torch.dtype, z: torch.Tensor | None = None, branch_1: torch.Tensor | None = None,
+                gate_gain_1: float = 0.0, bias_1: torch.Tensor | None = None, branch_2: torch.Tensor | None = None,
+                gate_gain_2: float = 0.0, bias_2: torch.Tensor | None = None, gain_1: float | None = None,
+                gain_2: float | None = None, next_eps: float = 0.0):
+    """``h += sigmoid(gate_gain_1 z_1 + bias_1) * branch_1 + sigmoid(gate_gain_2 z_2 + bias_2) * branch_2`` on the 32-bit
+    stream in place (``z [T, 2 width]`` or ``[T, width]``; without ``branch_1`` nothing is added, without ``branch_2`` only the
+    first term is).  With ``gain_1``: also returns ``(u, n_1, n_2)`` in ``dtype``, the new stream divided by its root mean
+    square, that times ``gain_1`` and that times ``gain_2`` (None without ``gain_2``)."""
+    require_device(h.device)
+    _check(h, "h", torch.float32, 2)
+    T, width = h.shape
+    if branch_1 is not None:
+        _check(z, "z", dtype, 2)
+        _check(branch_1, "branch_1", dtype, 2)
+        _check(bias_1, "bias_1", torch.float32, 1)
+        if z.shape[0] != T or z.shape[1] < width * (1 if branch_2 is None else 2) or branch_1.shape != h.shape or bias_1.shape[0] != width:
+            raise KernelError(f"gated_merge: the first branch or its gate does not fit a stream of {tuple(h.shape)}")
+    if branch_2 is not None:
+        _check(branch_2, "branch_2", dims=2)
+        _check(bias_2, "bias_2", torch.float32, 1)
+        if branch_1 is None or branch_2.shape != h.shape or bias_2.shape[0] != width:
+            raise KernelError(f"gated_merge: the second branch or its gate does not fit a stream of {tuple(h.shape)}")
+    u = n_1 = n_2 = None
+    if gain_1 is not None:
+        u, n_1 = torch.empty((2, T, width), dtype=dtype, device=h.device).unbind(0)
+        n_2 = None if gain_2 is None else torch.empty((T, width), dtype=dtype, device=h.device)
+    call("gk_gated_merge", ptr(h), dtype_code(dtype), ptr(z), 0 if z is None else z.shape[1], ptr(branch_1), ptr(branch_2),
+         dtype_code(dtype if branch_2 is None else branch_2.dtype), ptr(bias_1), ptr(bias_2), float(gate_gain_1), float(gate_gain_2), ptr(u),
+         ptr(n_1), ptr(n_2), float(gain_1 or 0.0), float(gain_2 or 0.0), float(next_eps), T, width, stream_ptr())
+    return u, n_1, n_2
+
+
+def poly_norm(z: torch.Tensor, numbers: tuple, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` row by row, ``N`` dividing a row by its root mean square, ``numbers = (a, b, c, e)``."""
+    require_device(z.device)
+    _check(z, "z", dims=2)
+    out = torch.empty(z.shape, dtype=out_dtype, device=z.device)
+    a, b, c, e = (float(n) for n in numbers)
+    call("gk_poly_norm", ptr(z), dtype_code(z.dtype), ptr(out), dtype_code(out_dtype), z.shape[0], z.shape[1], a, b, c, e, float(eps),
+         stream_ptr())
+    return out
+
+
+@dataclass(frozen=True)
+class MemoryColumns:
+    """Where a matrix memory's numbers stand in a packed projection row: the first column of q, k, v, the read-outs' gate, and
+    the two gates of the recurrence."""
+
+    q: int
+    k: int
+    v: int
+    g: int
+    i: int
+    f: int
+
+
+def _check_memory(proj: torch.Tensor, at: MemoryColumns, gate_bias: torch.Tensor, state: torch.Tensor, n_state: torch.Tensor):
+    _check(proj, "proj", dims=2)
+    _check(state, "state", torch.float32, 4)
+    _check(n_state, "n_state", torch.float32, 3)
+    _check(gate_bias, "gate_bias", torch.float32, 1)
+    H, d, dv = state.shape[1], state.shape[2] - 1, state.shape[3]
+    if tuple(n_state.shape) != (state.shape[0], H, d + 1) or gate_bias.shape[0] != 2 * H:
+        raise KernelError("matrix memory: the two states or the gates' biases do not fit one another")
+    ends = (at.q + H * d, at.k + H * d, at.v + H * dv, at.g + H * dv, at.i + H, at.f + H)
+    if min(at.q, at.k, at.v, at.g, at.i, at.f) < 0 or max(ends) > proj.shape[1]:
+        raise KernelError(f"matrix memory: a projection of {proj.shape[1]} columns is too narrow for these heads")
+    return H, d, dv
+
+
+def memory_scan(proj: torch.Tensor, at: MemoryColumns, gate_bias: torch.Tensor, cap: float, state: torch.Tensor, n_state: torch.Tensor,
+                cu_q: torch.Tensor, slots: torch.Tensor, n_seqs: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """The matrix memory's recurrence over the step's tokens of every sequence, token by token, from and to
+    ``state [slots, H, d + 1, dv]`` and ``n_state [slots, H, d + 1]`` (32-bit; the last row and entry hold the running maximum).
+    Returns the read-outs before their division ``[T, H, dv]`` and what divides them ``[T, H]``, both 32-bit."""
+    require_device(proj.device)
+    H, d, dv = _check_memory(proj, at, gate_bias, state, n_state)
+    T = proj.shape[0]
+    out = torch.empty((T, H, dv), dtype=torch.float32, device=proj.device)
+    den = torch.empty((T, H), dtype=torch.float32, device=proj.device)
+    call("gk_memory_scan", ptr(proj), dtype_code(proj.dtype), proj.shape[1], at.q, at.k, at.v, at.i, at.f, ptr(gate_bias), float(cap),
+         ptr(state), ptr(n_state), ptr(out), ptr(den), ptr(cu_q), ptr(slots), int(n_seqs), H, d, dv, stream_ptr())
+    return out, den

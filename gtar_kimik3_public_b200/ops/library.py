@@ -42,7 +42,7 @@ _SIGNATURES: dict[str, list] = {
     "gk_conv_state": [P, P, P, P, I, I, I, P],
     "gk_gelu_tanh": [P, P, I, L, P],
     "gk_heads_product_bf16": [P, L, L, P, P, L, L, I, I, I, I, P],
-    "gk_latent_prepare": [P, I, P, P, F, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
+    "gk_latent_prepare": [P, I, P, P, F, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, P],
     "gk_attention_latent_tiled": [P, L, L, P, I, I, P, P, P, P, L, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P],
     "gk_attention_latent_exact": [P, L, L, P, I, I, P, P, P, P, L, L, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P],
     "gk_attention_exact": [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, F, I, I, P],
@@ -87,12 +87,15 @@ _SIGNATURES: dict[str, list] = {
     "gk_scaled_sum": [P, F, P, F, I, P, L, P],
     "gk_relu_squared": [P, P, I, L, P],
     "gk_scale": [P, L, F, P],
-    "gk_heads_prepare": [P, I, L, I, I, I, I, I, I, I, I, I, P, P, P, P, F, F, P, P, P, P, I, P, P, P, P, P, I, I, I, I, P],
+    "gk_heads_prepare": [P, I, L, I, I, I, I, I, I, I, I, I, P, P, P, P, F, P, P, F, P, P, P, P, I, P, P, P, P, P, I, I, I, I, P],
     "gk_decay_scan": [P, P, P, P, P, P, P, P, I, I, I, I, P],
     "gk_decay_scan_chunked": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
-    "gk_group_norm_gate": [P, P, P, I, L, P, I, L, I, I, F, I, P],
-    "gk_attention_scored_exact": [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, P, P, I, P, P],
-    "gk_attention_scored_bf16": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, I, P, P, I, P, P],
+    "gk_group_norm_gate": [P, P, P, I, P, I, L, P, I, L, I, I, F, I, P],
+    "gk_attention_scored_exact": [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, P, P, I, P, F, P],
+    "gk_gated_merge": [P, I, P, L, P, P, I, P, P, F, F, P, P, P, F, F, F, I, I, P],
+    "gk_poly_norm": [P, I, P, I, I, I, F, F, F, F, F, P],
+    "gk_memory_scan": [P, I, L, I, I, I, I, I, P, F, P, P, P, P, P, P, I, I, I, I, P],
+    "gk_attention_scored_bf16": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, I, P, P, I, P, F, P],
 }
 
 

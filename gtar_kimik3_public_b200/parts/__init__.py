@@ -2,7 +2,7 @@
 Importing the package registers the built-in parts."""
 
 from . import (  # noqa: F401
-    attention, block, delta_rule, embedding, experts, latent_attention, linear_attention, mlp, norms, rope, scored_attention,
+    attention, block, delta_rule, embedding, experts, latent_attention, linear_attention, mlp, mlstm, norms, rope, scored_attention,
     side_by_side, wide_norm_attention,
 )
 from .base import (  # noqa: F401

@@ -1,14 +1,15 @@
 """Pre-norm residual block: ``h += mixer(norm_in(h)); h += ffn(norm_post(h))``
 (src/models/transformer.py:47-48).  The adds are fused into the norm that follows them: the
 block hands its last branch output on as ``pending`` instead of adding it itself.  Beside it: the block with
-convolutions over time in front of its sublayers, the block whose branches share one norm, the block that norms
-every branch on both sides, and the block that norms every branch on its way OUT only."""
+convolutions over time in front of its sublayers, the block whose branches share one norm, the block whose two gated branches
+have norms of their own, the block that norms every branch on both sides, and the block that norms every branch on its way OUT only."""
 
 from __future__ import annotations
 
 import torch
 
 from ..ops import functional as F
+from ..ops.linear import linear
 from .base import Block, FeedForward, Mixer, Norm, StepContext, register_part
 
 
@@ -241,6 +242,86 @@ class ParallelBlock(Block):
 
 
 register_part("block", "parallel", ParallelBlock)
+
+
+class GatedParallelBlock(Block):
+    """A layer whose two branches read the same stream through norms of their own and are gated entry by entry:
+
+        n_1 = norm_1(x);  n_2 = norm_2(x)
+        x += sigmoid(W_1 n_1 + b_1) * mixer(n_1) + sigmoid(W_2 n_2 + b_2) * feed_forward(n_2)
+
+    (the second term left out for a layer without feed-forward).  The norms have one number each (``gain``), so with
+    ``u`` the stream divided by its root mean square, ``n_i = gain_i u`` and ``W_i n_i = gain_i (W_i u)``: one packed product of
+    ``u`` with ``[W_1; W_2]`` gives both gates' arguments.  The gates, both products, the add into the 32-bit stream and
+    the NEXT layer's ``u``, ``n_1`` and ``n_2`` are one kernel (``gated_merge``); only a layer that nothing hands its rows (the model's
+    first) forms them with a launch of its own.  ``next_block``: the layer that follows, if it is of this kind."""
+
+    def __init__(self, width: int, norm_1: Norm, mixer: Mixer, norm_2: Norm | None, feed_forward: FeedForward | None,
+                 names: dict[str, str] | None = None):
+        if (feed_forward is None) != (norm_2 is None):
+            raise ValueError("a feed-forward comes with the norm before it, or not at all")
+        self.width = int(width)
+        self.norm_1, self.mixer, self.norm_2, self.feed_forward = norm_1, mixer, norm_2, feed_forward
+        self.names = {"mixer": "mix.", "feed_forward": "mlp.", "gate_1": "rg1", "gate_2": "rg2", **(names or {})}
+        self.next_block: GatedParallelBlock | None = None
+        self.w_gates = self.bias_1 = self.bias_2 = None
+
+    def children(self):
+        parts = [("", self.norm_1), (self.names["mixer"], self.mixer)]
+        if self.feed_forward is not None:
+            parts += [("", self.norm_2), (self.names["feed_forward"], self.feed_forward)]
+        return parts
+
+    def _gate_names(self):
+        return [self.names["gate_1"]] + ([self.names["gate_2"]] if self.feed_forward is not None else [])
+
+    def tensor_specs(self):
+        from .base import TensorSpec
+
+        specs = {prefix + name: spec for prefix, part in self.children() for name, spec in part.tensor_specs().items()}
+        for name in self._gate_names():
+            specs[name] = TensorSpec((self.width, self.width))
+            specs[name + ".b"] = TensorSpec((self.width,), "vector", init=(0.0, 0.5))
+        return specs
+
+    def load(self, tensors):
+        for prefix, part in self.children():
+            part.load({name: tensors[prefix + name] for name in part.tensor_specs() if prefix + name in tensors})
+        gates = [tensors[name] for name in self._gate_names()]
+        if len({t.dtype for t in gates}) != 1:
+            gates = [t.float() for t in gates]
+        self.w_gates = torch.cat(gates, dim=0).contiguous()
+        biases = [tensors[name + ".b"].float().contiguous() for name in self._gate_names()]
+        self.bias_1, self.bias_2 = biases[0], biases[1] if len(biases) > 1 else None
+
+    def weight_bytes(self):
+        own = sum(t.numel() * t.element_size() for t in (self.w_gates, self.bias_1, self.bias_2) if t is not None)
+        return own + sum(part.weight_bytes() for _, part in self.children())
+
+    def norm_rule(self) -> dict:
+        """What the kernel that forms this layer's rows needs of its norms."""
+        return dict(gain_1=self.norm_1.gain, gain_2=None if self.norm_2 is None else self.norm_2.gain, next_eps=self.norm_1.eps)
+
+    def forward(self, h, pending, ctx: StepContext, cache):
+        if pending is not None:
+            raise ValueError("a layer of this kind takes its stream whole: the layer before must not leave a branch unadded")
+        rows = ctx.extras.pop("gated_rows", None)
+        if rows is None or rows[0] is not self:
+            rows = (self, *F.gated_merge(h, ctx.dtype, **self.norm_rule()))
+        _, u, n_1, n_2 = rows
+        z = linear(u, self.w_gates)
+        branch_1 = self.mixer.forward(n_1, ctx, cache)
+        branch_2 = None if self.feed_forward is None else self.feed_forward.forward(n_2, ctx)
+        follower = self.next_block
+        out = F.gated_merge(h, ctx.dtype, z=z, branch_1=branch_1, gate_gain_1=self.norm_1.gain, bias_1=self.bias_1, branch_2=branch_2,
+                            gate_gain_2=0.0 if self.norm_2 is None else self.norm_2.gain, bias_2=self.bias_2,
+                            **({} if follower is None else follower.norm_rule()))
+        if follower is not None:
+            ctx.extras["gated_rows"] = (follower, *out)
+        return h, None
+
+
+register_part("block", "gated_parallel", GatedParallelBlock)
 
 
 class SandwichBlock(Block):

@@ -13,6 +13,11 @@ With ``logit_weights`` the router is plainer: scores are the logits plus a store
 name is the builder's, ``bias_name``), the ``top`` largest are chosen, and the chosen experts' weights are the softmax
 over the chosen scores alone (times ``route_scale``).
 
+Further rules, each a parameter: ``scores="softmax"``: ``s`` is the softmax of the logits over all experts;
+``group_rule="best"``: a group's score is its largest choice score; ``renormalise``: the chosen experts' ``s`` are divided
+by their sum (plus 1e-20) before ``route_scale``; ``shared_size``: one more expert of that inner size, of the same form
+(tensors ``shared.gate``, ``shared.up``, ``shared.down``), runs for every token and is added with weight one.
+
 The result is 32-bit (it goes into the residual stream); ``forward_added`` folds another branch's output into the
 same sum, for blocks whose branches read one norm.
 """
@@ -22,7 +27,7 @@ from __future__ import annotations
 import torch
 
 from ..ops import functional as F
-from ..ops.linear import grouped_product_ok, linear_grouped
+from ..ops.linear import grouped_product_ok, linear, linear_grouped
 from .base import FeedForward, StepContext, TensorSpec, register_part
 
 
@@ -30,7 +35,8 @@ class RoutedExperts(FeedForward):
     graph_safe = True
 
     def __init__(self, hidden_size: int, expert_size: int, n_experts: int, top: int, route_scale: float = 1.0,
-                 n_groups: int = 1, keep_groups: int = 1, logit_weights: bool = False, bias_name: str = "correction"):
+                 n_groups: int = 1, keep_groups: int = 1, logit_weights: bool = False, bias_name: str = "correction",
+                 scores: str = "sigmoid", group_rule: str = "two_best", renormalise: bool = False, shared_size: int | None = None):
         self.hidden_size, self.ff, self.n_experts, self.top = int(hidden_size), int(expert_size), int(n_experts), int(top)
         self.route_scale, self.n_groups, self.keep = float(route_scale), int(n_groups), int(keep_groups)
         if self.n_experts % self.n_groups or not 1 <= self.keep <= self.n_groups:
@@ -38,6 +44,13 @@ class RoutedExperts(FeedForward):
         if not 1 <= self.top <= self.keep * (self.n_experts // self.n_groups):
             raise ValueError(f"{self.top} experts cannot be chosen from {self.keep} groups of {self.n_experts // self.n_groups}")
         self.logit_weights, self.bias_name = bool(logit_weights), bias_name
+        if scores not in ("sigmoid", "softmax") or group_rule not in ("two_best", "best"):
+            raise ValueError("scores are 'sigmoid' or 'softmax', group_rule is 'two_best' or 'best'")
+        if self.logit_weights and (scores != "sigmoid" or renormalise):
+            raise ValueError("logit weights come with a rule of their own for scores and weights")
+        self.scores, self.group_rule, self.renormalise = scores, group_rule, bool(renormalise)
+        self.shared_ff = int(shared_size) if shared_size else 0
+        self.w_shared_gate_up = self.w_shared_down = None
         self.w_gate_up = self.w_down = self.w_router = self.correction = None
         # from this many (token, expert) pairs on, a bfloat16 step sorts its pairs by expert and runs each expert's rows
         # through one tensor-core product; below, every pair streams its expert's weights by itself
@@ -51,7 +64,13 @@ class RoutedExperts(FeedForward):
             specs[f"e{e}.up"] = TensorSpec((ff, W))
             specs[f"e{e}.down"] = TensorSpec((W, ff))
         specs["router"] = TensorSpec((self.n_experts, W), init=(0.0, 0.5))
-        specs[self.bias_name] = TensorSpec((self.n_experts,), "vector", init=(0.0, 0.3))
+        # softmax scores are small numbers: a correction of the usual size would decide the choice alone
+        spread = 0.3 if self.scores == "sigmoid" else 0.3 / self.n_experts
+        specs[self.bias_name] = TensorSpec((self.n_experts,), "vector", init=(0.0, spread))
+        if self.shared_ff:
+            specs["shared.gate"] = TensorSpec((self.shared_ff, W))
+            specs["shared.up"] = TensorSpec((self.shared_ff, W))
+            specs["shared.down"] = TensorSpec((W, self.shared_ff))
         return specs
 
     def load(self, tensors):
@@ -62,18 +81,30 @@ class RoutedExperts(FeedForward):
         self.w_down = torch.stack([tensors[f"e{e}.down"].to(kind) for e in range(E)]).contiguous()
         self.w_router = tensors["router"].float().contiguous()
         self.correction = tensors[self.bias_name].float().contiguous()
+        if self.shared_ff:
+            gate, up, down = (tensors["shared." + part] for part in ("gate", "up", "down"))
+            if gate.dtype != up.dtype:
+                gate, up = gate.float(), up.float()
+            # gate and up rows alternate: the activation is the product's output stage
+            self.w_shared_gate_up = torch.stack([gate, up], dim=1).reshape(2 * self.shared_ff, self.hidden_size).contiguous()
+            self.w_shared_down = down.contiguous()
 
     def weight_bytes(self):
-        """What a single token reads: its ``top`` experts and the router."""
+        """What a single token reads: its ``top`` experts, the shared one and the router."""
         per_expert = (self.w_gate_up[0].numel() + self.w_down[0].numel()) * self.w_down.element_size()
-        return self.top * per_expert + self.w_router.numel() * 4
+        shared = sum(t.numel() * t.element_size() for t in (self.w_shared_gate_up, self.w_shared_down) if t is not None)
+        return self.top * per_expert + self.w_router.numel() * 4 + shared
 
     def route(self, x: torch.Tensor):
         return F.route_groups(x, self.w_router, self.correction, self.top, self.n_groups, self.keep, self.route_scale,
-                              logits=self.logit_weights)
+                              logits=self.logit_weights, softmax=self.scores == "softmax", best_of_group=self.group_rule == "best",
+                              renormalise=self.renormalise)
 
     def forward_added(self, x: torch.Tensor, ctx: StepContext, add: torch.Tensor | None) -> torch.Tensor:
         """``add + experts(x)`` as one 32-bit sum (``add``: another branch's output for the same tokens, or None)."""
+        if self.shared_ff:
+            shared = linear(linear(x, self.w_shared_gate_up, swiglu=True), self.w_shared_down)
+            add = shared if add is None else F.scaled_sum(add, 1.0, shared, 1.0).to(x.dtype)
         ids, weights = self.route(x)
         if x.shape[0] * self.top >= self.grouped_from_pairs and self.ff % 8 == 0 and grouped_product_ok(x, self.w_down):
             # many tokens: the pairs in the order of their experts, each expert's rows through one product

@@ -10,6 +10,11 @@ Only the normed latent and the rotated key part are kept per position (one row f
 matrices never touch the cache: ``q_n . U_k c = (U_k^T q_n) . c``, so the query is carried into the latent before
 attention, attention runs over the cached rows with the latent as the value, and ``U_v`` is applied to the result.
 
+Two further rules, each a parameter: ``pairing="neighbours"``: rotated entry ``2i`` turns with ``2i + 1`` (the default pairs
+``i`` with ``i + dims/2``); the rows of the two matrices that make rotated parts are put in the other order at load, on the
+query's and the key's side alike, so that scores and kernels stay as they are.  ``gated``: every entry of the heads' outputs
+is multiplied by the sigmoid of ``W_g x`` (tensor ``g``, packed behind the down-projection) before ``W_o``.
+
 A step's kernels: the packed down-projection ``[W_dq; W_dkv]``; one kernel for both norms, the key part's rotation and
 the cache write; the up-projection of the queries; a batched product (one per head) that carries the queries; the
 attention kernel, which rotates the queries' own part itself; a batched product for the values; the output projection.
@@ -23,8 +28,9 @@ from ..ops import attention as attention_ops
 from ..ops import functional as F
 from ..ops.linear import linear
 from .base import Mixer, PositionEncoding, RowsRequest, StepContext, TensorSpec, register_part
+from .delta_rule import _pad_rows
 
-_NAMES = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "o": "o"}
+_NAMES = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "o": "o", "g": "g"}
 
 
 class LatentAttention(Mixer):
@@ -32,7 +38,7 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden_size: int, n_heads: int, head_dim: int, rot_dim: int, value_dim: int, q_rank: int, kv_rank: int,
                  scale: float, norm_eps: float, position: PositionEncoding | None, window: int | None = None,
-                 names: dict[str, str] | None = None):
+                 names: dict[str, str] | None = None, pairing: str = "halves", gated: bool = False):
         """``position``: tables of cos and sin for ``position.dim`` of the ``rot_dim`` rotated entries (the first ones;
         the rest pass unchanged), or None for no rotation.  ``scale`` multiplies every score as it is given."""
         self.hidden_size, self.n_heads, self.head_dim, self.rot_dim = int(hidden_size), int(n_heads), int(head_dim), int(rot_dim)
@@ -44,12 +50,15 @@ class LatentAttention(Mixer):
             raise ValueError(f"{self.rot_dims} rotated dimensions in a part of {self.rot_dim}")
         if min(self.n_heads, self.head_dim, self.value_dim, self.q_rank, self.kv_rank) <= 0 or self.rot_dim < 0:
             raise ValueError("latent attention sizes must be positive")
+        if pairing not in ("halves", "neighbours"):
+            raise ValueError(f"rotated entries are paired as 'halves' or 'neighbours', not {pairing!r}")
+        self.pairing, self.gated = pairing, bool(gated)
         self.names = {**_NAMES, **(names or {})}
         self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = self.q_norm = self.kv_norm = None
 
     def tensor_specs(self):
         n, H = self.names, self.n_heads
-        return {
+        specs = {
             n["dq"]: TensorSpec((self.q_rank, self.hidden_size)),
             n["dq_norm"]: TensorSpec((self.q_rank,), "vector"),
             n["uq"]: TensorSpec((H * (self.head_dim + self.rot_dim), self.q_rank)),
@@ -59,14 +68,30 @@ class LatentAttention(Mixer):
             n["uv"]: TensorSpec((H * self.value_dim, self.kv_rank)),
             n["o"]: TensorSpec((self.hidden_size, H * self.value_dim)),
         }
+        if self.gated:
+            specs[n["g"]] = TensorSpec((H * self.value_dim, self.hidden_size))
+        return specs
+
+    def _halves(self, rows: torch.Tensor) -> torch.Tensor:
+        """``rows [..., rot_dim, k]`` of a rotated part in the order the kernels turn them: of every pair of neighbours the
+        first entries, then the second ones."""
+        if self.pairing == "halves" or not self.rot_dims:
+            return rows
+        order = [*range(0, self.rot_dims, 2), *range(1, self.rot_dims, 2), *range(self.rot_dims, self.rot_dim)]
+        return rows[..., torch.tensor(order, device=rows.device), :]
 
     def load(self, tensors):
         n, H = self.names, self.n_heads
-        down = [tensors[n["dq"]], tensors[n["dkv"]]]
-        if down[0].dtype != down[1].dtype:
+        dkv = tensors[n["dkv"]]
+        down = [tensors[n["dq"]], dkv[:self.kv_rank], self._halves(dkv[self.kv_rank:])]
+        if self.gated:
+            down.append(tensors[n["g"]])
+        if len({t.dtype for t in down}) != 1:
             down = [t.float() for t in down]
-        self.w_down = torch.cat(down, dim=0).contiguous()  # one product for both latents
-        self.w_uq = tensors[n["uq"]].contiguous()
+        self.gate_at = self.q_rank + self.kv_rank + self.rot_dim
+        self.w_down = _pad_rows(torch.cat(down, dim=0)).contiguous()  # one product for both latents (and the gate)
+        uq = tensors[n["uq"]].view(H, self.head_dim + self.rot_dim, self.q_rank)
+        self.w_uq = torch.cat([uq[:, :self.head_dim], self._halves(uq[:, self.head_dim:])], dim=1).reshape(-1, self.q_rank).contiguous()
         # per head: [kv_rank, dim] so that the product with a head's unrotated query gives its carried form
         self.w_uk_t = tensors[n["uk"]].view(H, self.head_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = tensors[n["uv"]].view(H, self.value_dim, self.kv_rank).contiguous()
@@ -97,6 +122,8 @@ class LatentAttention(Mixer):
                                        self.window or 0, mixed.transpose(0, 1))
         o = torch.empty((T, H * self.value_dim), dtype=x.dtype, device=x.device)
         F.linear_batched(mixed, self.w_uv, o.view(T, H, self.value_dim).transpose(0, 1))
+        if self.gated:
+            o = F.sigmoid_gate(o, both, self.gate_at)
         return linear(o, self.w_o)
 
 

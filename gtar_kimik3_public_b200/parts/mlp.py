@@ -152,3 +152,42 @@ class XieluFeedForward(FeedForward):
 
 
 register_part("feed_forward", "xielu", XieluFeedForward)
+
+
+class PolyNormFeedForward(FeedForward):
+    """``down(act(up(x)))`` with an activation that norms three powers of a token's whole row: with ``N(y)`` the row ``y``
+    divided by its root mean square (eps inside the root),
+
+        act(z) = a N(z) + b N(z^2) + c N(z^3) + e              (powers entry by entry; tensor ``act`` holds a, b, c, e)
+
+    No gate, no biases.  The sums over a row need all of it, so the activation is a kernel of its own between the products;
+    it reads the up product's 32-bit sums where few tokens leave them in 32-bit, else its bfloat16 result."""
+
+    graph_safe = True
+
+    def __init__(self, hidden_size: int, intermediate_size: int, eps: float, up_name: str = "up", down_name: str = "down",
+                 act_name: str = "act"):
+        self.hidden_size, self.intermediate_size, self.eps = int(hidden_size), int(intermediate_size), float(eps)
+        self.up_name, self.down_name, self.act_name = up_name, down_name, act_name
+        self.w_up = self.w_down = None
+        self.numbers = (0.0, 0.0, 0.0, 0.0)
+
+    def tensor_specs(self):
+        h, i = self.hidden_size, self.intermediate_size
+        return {self.up_name: TensorSpec((i, h)), self.down_name: TensorSpec((h, i)),
+                self.act_name: TensorSpec((4,), "vector", init=(0.4, 0.3))}
+
+    def load(self, tensors):
+        self.w_up = tensors[self.up_name].contiguous()
+        self.w_down = tensors[self.down_name].contiguous()
+        self.numbers = tuple(tensors[self.act_name].float().tolist())
+
+    def weight_bytes(self):
+        return sum(t.numel() * t.element_size() for t in (self.w_up, self.w_down))
+
+    def forward(self, x, ctx: StepContext) -> torch.Tensor:
+        z = linear(x, self.w_up, torch.float32 if x.shape[0] <= F.GEMV_MAX_TOKENS else None)
+        return linear(F.poly_norm(z, self.numbers, self.eps, ctx.dtype), self.w_down)
+
+
+register_part("feed_forward", "poly_norm", PolyNormFeedForward)

@@ -46,6 +46,36 @@ class RMSNorm(Norm):
 register_part("norm", "rmsnorm", RMSNorm)
 
 
+class ScalarRMSNorm(Norm):
+    """RMS norm with ONE number for all entries, ``g * x / sqrt(mean(x^2) + eps)`` in 32-bit (the tensor has no dimensions).
+    ``gain`` is that number on the host, for kernels that form several norms of one stream; by itself the norm is the
+    RMS norm of the library with the number in every entry of its weight."""
+
+    graph_safe = True
+
+    def __init__(self, size: int, eps: float, weight_name: str = "weight"):
+        self.size, self.eps, self.weight_name = int(size), float(eps), weight_name
+        self.gain: float | None = None
+        self.weight: torch.Tensor | None = None
+
+    def tensor_specs(self):
+        return {self.weight_name: TensorSpec((), "vector", init=(1.0, 0.2))}
+
+    def load(self, tensors):
+        gain = tensors[self.weight_name].float()
+        self.gain = float(gain.item())
+        self.weight = gain.reshape(1).expand(self.size).contiguous()
+
+    def weight_bytes(self):
+        return self.weight.numel() * self.weight.element_size()
+
+    def forward(self, h, delta, out_dtype, rows=None):
+        return F.add_rmsnorm(h, delta, self.weight, self.eps, out_dtype, rows)
+
+
+register_part("norm", "rmsnorm_scalar", ScalarRMSNorm)
+
+
 class LayerNorm(Norm):
     """Layer norm with a weight and no bias, ``(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight`` in 32-bit, fused with
     the add of a pending branch output into the stream; ``delta_scale`` multiplies that branch as it is added (a model

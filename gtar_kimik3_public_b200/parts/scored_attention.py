@@ -18,6 +18,9 @@ Further rules, each switched on by the builder:
 
 * ``wide_norm``: before anything else the whole query row (all heads at once) is divided by its root mean square and
   multiplied by a weight per entry (tensor ``q.norm``), and so is the whole key row (``k.norm``);
+* ``head_norm``: every query head is divided by its root mean square (eps inside the root) and multiplied by one weight of
+  ``key_dim`` entries that all query heads share (tensor ``q.norm``), and so are the key heads (``k.norm``);
+* ``softcap``: the score (before any distance term) becomes ``softcap * tanh(score / softcap)``;
 * ``temperature``: the product is multiplied by a number per query head (tensor ``temp``), ``q . k * scale * temp_h``;
 * ``distance_table = (rows, far)``: a learned term per query head and distance is ADDED to the score (the scale does not
   touch it), read from ``rel [rows, heads]`` (a model file's tensor chooses ``rows``) at row ``bucket(i - j)``: ``bucket(n) = n`` below ``rows // 2``, then
@@ -78,7 +81,7 @@ class ScoredAttention(Mixer):
                  names: dict[str, str] | None = None, wide_norm: bool = False, temperature: bool = False,
                  distance_table: tuple[int, float] | None = None, chunk: int | None = None, sink: str | None = None,
                  value_position: PositionEncoding | None = None, head_gate: bool = False, own_kv: bool = True,
-                 cache_span: int | None | str = "own"):
+                 cache_span: int | None | str = "own", head_norm: bool = False, softcap: float | None = None):
         if n_q_heads % n_kv_heads:
             raise ValueError("query heads must be a multiple of key heads")
         if weights not in ("softmax", "sigmoid"):
@@ -99,6 +102,11 @@ class ScoredAttention(Mixer):
         self.wide_norm, self.temperature, self.sink_kind = bool(wide_norm), bool(temperature), sink
         if self.wide_norm and (self.rot or self.unit_qk):
             raise ValueError("norms over whole rows come without rotation and unit lengths")
+        self.head_norm, self.softcap = bool(head_norm), float(softcap or 0.0)
+        if self.head_norm and (self.rot or self.unit_qk or self.wide_norm):
+            raise ValueError("norms per head come without rotation, unit lengths and norms over whole rows")
+        if self.softcap and weights != "softmax":
+            raise ValueError("capped scores belong to the softmax")
         self.distance_table = None if distance_table is None else (int(distance_table[0]), float(distance_table[1]))
         self.dist_rows = None  # formed at load: the table's height is the tensor's
         self.chunk = None if not chunk else int(chunk)
@@ -131,6 +139,10 @@ class ScoredAttention(Mixer):
             specs[n["q_norm"]] = TensorSpec((self.n_q * self.d,), "vector")
             if self.own_kv:
                 specs[n["k_norm"]] = TensorSpec((self.n_kv * self.d,), "vector")
+        if self.head_norm:
+            specs[n["q_norm"]] = TensorSpec((self.d,), "vector")
+            if self.own_kv:
+                specs[n["k_norm"]] = TensorSpec((self.d,), "vector")
         if self.temperature:
             specs[n["temp"]] = TensorSpec((self.n_q,), "vector", init=(1.0, 0.3))
         if self.distance_table is not None:
@@ -155,7 +167,7 @@ class ScoredAttention(Mixer):
             self.r1, self.r2 = tensors[n["r1"]].float().contiguous(), tensors[n["r2"]].float().contiguous()
         if self.head_bias:
             self.pb = tensors[n["pb"]].float().contiguous()
-        if self.wide_norm:
+        if self.wide_norm or self.head_norm:
             self.q_norm = tensors[n["q_norm"]].float().contiguous()
             self.k_norm = tensors[n["k_norm"]].float().contiguous() if self.own_kv else self.q_norm
         if self.temperature:
@@ -197,10 +209,11 @@ class ScoredAttention(Mixer):
         else:
             k_at, v_at = (nq, nq + nk) if self.own_kv else (0, 0)
             q = F.heads_prepare(proj, 0, k_at, v_at, self.n_q, self.n_kv, self.d, self.dv, ctx.tok_pos, ctx.tok_seq, ctx.slots,
-                                rot=self.rot, cos=cos, sin=sin, unit_eps=self.norm_eps if self.unit_qk else None, kv=cache,
+                                rot=self.rot, cos=cos, sin=sin, unit_eps=self.norm_eps if self.unit_qk or self.head_norm else None, kv=cache,
+                                w_q=self.q_norm if self.head_norm else None, w_k=self.k_norm if self.head_norm else None,
                                 write_kv=write, max_position=ctx.max_position, v_cos=v_cos if self.own_kv else None,
                                 v_sin=v_sin if self.own_kv else None)
-        rules = dict(chunk=self.chunk or 0, temp=self.temp, dist_bias=self.dist_bias, sink=self.sink)
+        rules = dict(chunk=self.chunk or 0, temp=self.temp, dist_bias=self.dist_bias, sink=self.sink, softcap=self.softcap)
         if q.dtype == torch.bfloat16 and self.d == self.dv and self.d in (64, 128) and cache.page_size == 64:
             # what a row can see at most, whatever the lengths of later steps that replay this one from a graph
             spans = [s for s in (self.window + self.keep_first if self.window else None, self.chunk) if s]

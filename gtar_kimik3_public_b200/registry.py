@@ -84,3 +84,7 @@ def _ensure_builtin() -> None:
     from .models.zasorax import build_zasorax_plan
 
     register_architecture(ZasoraxConfig.ARCH_NAMES, ZasoraxConfig, build_zasorax_plan)
+    from .config.topezen import TopezenConfig
+    from .models.topezen import build_topezen_plan
+
+    register_architecture(TopezenConfig.ARCH_NAMES, TopezenConfig, build_topezen_plan)
