@@ -1978,3 +1978,58 @@ def memory_scan(proj: torch.Tensor, at: MemoryColumns, gate_bias: torch.Tensor, 
     call("gk_memory_scan", ptr(proj), dtype_code(proj.dtype), proj.shape[1], at.q, at.k, at.v, at.i, at.f, ptr(gate_bias), float(cap),
          ptr(state), ptr(n_state), ptr(out), ptr(den), ptr(cu_q), ptr(slots), int(n_seqs), H, d, dv, stream_ptr())
     return out, den
+
+
+def memory_single_fits(d: int, dv: int) -> bool:
+    """Whether :func:`memory_single` takes heads of these sizes."""
+    return 0 < d <= 512 and dv % 4 == 0 and 0 < dv <= 512
+
+
+def _check_memory_norm(norm_w: torch.Tensor, H: int, dv: int) -> None:
+    _check(norm_w, "norm_w", torch.float32, 1)
+    if norm_w.shape[0] != H * dv:
+        raise KernelError(f"matrix memory: a norm weight of {norm_w.shape[0]} for {H} heads of {dv}")
+
+
+def memory_single(proj: torch.Tensor, at: MemoryColumns, gate_bias: torch.Tensor, cap: float, state: torch.Tensor, n_state: torch.Tensor,
+                  norm_w: torch.Tensor, eps: float, cu_q: torch.Tensor, slots: torch.Tensor, n_seqs: int) -> torch.Tensor:
+    """:func:`memory_scan` for steps of one token a sequence, with the division, the norm of every head, ``norm_w [H dv]`` and the
+    sigmoid of the gate's columns in the same kernel.  Returns ``[T, H dv]`` in the projection's type."""
+    require_device(proj.device)
+    H, d, dv = _check_memory(proj, at, gate_bias, state, n_state)
+    _check_memory_norm(norm_w, H, dv)
+    if not memory_single_fits(d, dv) or proj.shape[0] != n_seqs:
+        raise KernelError(f"memory_single: {proj.shape[0]} tokens of {n_seqs} sequences, heads of {d} / {dv}")
+    y = torch.empty((proj.shape[0], H * dv), dtype=proj.dtype, device=proj.device)
+    call("gk_memory_single", ptr(proj), dtype_code(proj.dtype), proj.shape[1], at.q, at.k, at.v, at.g, at.i, at.f, ptr(gate_bias),
+         float(cap), ptr(state), ptr(n_state), ptr(norm_w), float(eps), ptr(y), ptr(cu_q), ptr(slots), int(n_seqs), H, d, dv, stream_ptr())
+    return y
+
+
+def memory_chunked_fits(d: int, dv: int, at: MemoryColumns, ld: int) -> bool:
+    """Whether :func:`memory_chunked` takes heads of these sizes at these columns of rows of ``ld`` entries."""
+    return (d % 16 == 0 and dv % 16 == 0 and 0 < d <= 256 and 0 < dv <= 512 and ld % 8 == 0
+            and at.q % 8 == 0 and at.k % 8 == 0 and at.v % 8 == 0 and at.g % 2 == 0)
+
+
+def memory_chunked(proj: torch.Tensor, at: MemoryColumns, gate_bias: torch.Tensor, cap: float, state: torch.Tensor, n_state: torch.Tensor,
+                   norm_w: torch.Tensor, eps: float, cu_q: torch.Tensor, slots: torch.Tensor, n_seqs: int, max_q_len: int) -> torch.Tensor:
+    """:func:`memory_scan` for bfloat16 steps of many tokens, in chunks of 64 tokens whose inner work is matrix products, with
+    the division, the norm of every head, ``norm_w [H dv]`` and the sigmoid of the gate's columns in the last kernel.  The sums
+    have another order than token by token, so the two agree within rounding.  ``max_q_len`` bounds the sequences' token
+    counts in this step.  Returns ``[T, H dv]`` in bfloat16."""
+    require_device(proj.device)
+    H, d, dv = _check_memory(proj, at, gate_bias, state, n_state)
+    _check(proj, "proj", torch.bfloat16, 2)
+    _check_memory_norm(norm_w, H, dv)
+    y = torch.empty((proj.shape[0], H * dv), dtype=proj.dtype, device=proj.device)
+    chunks = max(1, -(-int(max_q_len) // DECAY_CHUNK))
+    per_chunk = max(1, n_seqs) * H * (d * dv + d)
+    wave = max(1, min(chunks, DECAY_WORKSPACE_FLOATS // per_chunk))
+    states = torch.empty((wave * per_chunk,), dtype=torch.float32, device=proj.device)
+    scalars = torch.empty((max(1, n_seqs) * H * (3 * wave + 1),), dtype=torch.float32, device=proj.device)
+    start = scalars[max(1, n_seqs) * H * 3 * wave:]
+    call("gk_memory_chunked", ptr(proj), proj.shape[1], at.q, at.k, at.v, at.g, at.i, at.f, ptr(gate_bias), float(cap), ptr(state),
+         ptr(n_state), ptr(norm_w), float(eps), ptr(y), ptr(states), ptr(scalars), ptr(start), ptr(cu_q), ptr(slots), int(n_seqs), H, d, dv,
+         int(max_q_len), wave, stream_ptr())
+    return y

@@ -84,8 +84,16 @@ class MatrixMemory(Mixer):
         H, d, dv = self.n_heads, self.d, self.dv
         proj = linear(x, self.w_in)
         at = F.MemoryColumns(q=0, k=H * d, v=2 * H * d, g=2 * H * d + H * dv, i=2 * H * d + 2 * H * dv, f=2 * H * d + 2 * H * dv + H)
-        o, den = F.memory_scan(proj, at, self.gate_bias, self.gate_cap, state, n_state, ctx.cu_q, ctx.slots, ctx.n_seqs)
-        y = F.group_norm_gate(o.view(ctx.n_tokens, H * dv), dv, self.norm_w, proj, at.g, self.norm_eps, ctx.dtype, divisor=den)
+        core = (proj, at, self.gate_bias, self.gate_cap, state, n_state)
+        steps = (ctx.cu_q, ctx.slots, ctx.n_seqs)
+        if ctx.all_single and F.memory_single_fits(d, dv):
+            y = F.memory_single(*core, self.norm_w, self.norm_eps, *steps)
+        elif (ctx.dtype == torch.bfloat16 and proj.dtype == torch.bfloat16 and ctx.max_q_len >= self.chunked_from
+              and F.memory_chunked_fits(d, dv, at, proj.shape[1])):
+            y = F.memory_chunked(*core, self.norm_w, self.norm_eps, *steps, ctx.max_q_len)
+        else:  # few tokens a sequence, other sizes, and 32-bit runs (whose numbers do not depend on how a prompt is cut)
+            o, den = F.memory_scan(*core, *steps)
+            y = F.group_norm_gate(o.view(ctx.n_tokens, H * dv), dv, self.norm_w, proj, at.g, self.norm_eps, ctx.dtype, divisor=den)
         return linear(y, self.w_o)
 
 
