@@ -14,7 +14,8 @@ Weights are random (written as a model folder by the library's random-weights mo
 from there), token ids are seeded uniform-random: there is no network for checkpoints or data.
 The library runs on one GPU; with --gpus N > 1 a line says so and the exit code is 2.
 
-``--compare pofadra`` and ``--compare rezulorn`` do the same for the Pofadra and the Rezulorn decoders; ``--compare zasorax`` puts the Zasorax decoder beside the Rezulorn decoder.  ``--compare dasusun`` runs another workload instead and prints its own JSON line: the Dasusun decoder beside the transformer
+``--compare pofadra`` and ``--compare rezulorn`` do the same for the Pofadra and the Rezulorn decoders; ``--compare zasorax`` puts the Zasorax decoder beside the Rezulorn decoder,
+``--compare topezen`` the Topezen decoder beside the Pofadra decoder.  ``--compare dasusun`` runs another workload instead and prints its own JSON line: the Dasusun decoder beside the transformer
 at equal layer sizes (prefill and decode throughput of both, and the new design's kernels one by one against their rooflines).
 """
 
@@ -1486,6 +1487,254 @@ def run_compare_zasorax(args) -> dict:
             "results": results}
 
 
+# --compare topezen: the Topezen decoder (two gated branches a layer; matrix memories, one scored attention with capped
+# scores and one latent attention in four layers; PolyNorm and routed feed-forwards with a shared expert) beside the
+# Pofadra decoder (recurrent layers, one attention in four, routed experts) at equal width and about equal bytes of weights
+# read per token, and its kernels one by one beside the like kernels of the models that were here.
+def _topezen_config(width, layers, heads, dim, vdim, cap, a_heads, a_kv, a_dim, window, keep, softcap, l_heads, l_dim, l_rot, l_vdim, q_rank,
+                    kv_rank, ff, experts, top, groups, group_keep, expert_ff, shared_ff, vocab):
+    memory = {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": cap}
+    scored = {"heads": a_heads, "kv_heads": a_kv, "dim": a_dim, "vdim": a_dim, "scale": a_dim ** -0.5, "softcap": softcap,
+              "mask": {"size": window, "keep_first": keep}}
+    latent = {"heads": l_heads, "dim": l_dim, "rot_dim": l_rot, "vdim": l_vdim, "q_rank": q_rank, "kv_rank": kv_rank,
+              "scale": (l_dim + l_rot) ** -0.5, "rot": {"base": 500000.0, "dims": l_rot}}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff},
+           "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": group_keep}}}
+    kinds = [("mlstm", memory, dense), ("mlstm", memory, moe), ("attention", scored, moe), ("latent_attention", latent, moe)]
+    stack = [dict(zip(("type", "mixer", "mlp"), kinds[i % 4])) for i in range(layers)]
+    return {"architecture": "Topezen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
+            "layers": stack, "initializer_range": 0.02, "max_position_embeddings": 4096}
+
+
+TOPEZEN_SIZES = {
+    # name: (Topezen sizes, Pofadra sizes); 8 layers each, vocabulary 32,768; a routed layer's chosen and shared experts hold
+    # what the chosen experts of the other design hold, and so does a dense layer
+    "width1024": (dict(width=1024, layers=8, heads=8, dim=128, vdim=128, cap=15.0, a_heads=16, a_kv=4, a_dim=64, window=1024, keep=4,
+                       softcap=50.0, l_heads=16, l_dim=64, l_rot=32, l_vdim=64, q_rank=512, kv_rank=256, ff=4608, experts=32, top=3, groups=4,
+                       group_keep=2, expert_ff=768, shared_ff=768, vocab=32768),
+                  POFADRA_SIZES["width1024"][0]),
+    "width2048": (dict(width=2048, layers=8, heads=16, dim=128, vdim=128, cap=15.0, a_heads=16, a_kv=4, a_dim=128, window=1024, keep=4,
+                       softcap=50.0, l_heads=16, l_dim=128, l_rot=64, l_vdim=128, q_rank=768, kv_rank=512, ff=9216, experts=64, top=5, groups=8,
+                       group_keep=4, expert_ff=1024, shared_ff=1024, vocab=32768),
+                  POFADRA_SIZES["width2048"][0]),
+}
+
+
+def _topezen_prefill_flops(d: dict, tokens: int) -> float:
+    w = d["width"]
+    seen = sum(min(t + 1, d["window"]) + min(d["keep"], max(0, t + 1 - d["window"])) for t in range(tokens))
+    causal = tokens * (tokens + 1) // 2
+    gates = 4 * w * w
+    dense = 4 * w * d["ff"]
+    routed = 6 * w * (d["expert_ff"] * d["top"] + d["shared_ff"]) + 2 * w * d["experts"]
+    memory = 2 * w * (2 * d["heads"] * d["dim"] + 3 * d["heads"] * d["vdim"] + 2 * d["heads"]) + 4 * d["heads"] * d["dim"] * d["vdim"]
+    scored = 2 * w * (2 * d["a_heads"] + 2 * d["a_kv"]) * d["a_dim"]
+    lh, ld, lr, lv, r = d["l_heads"], d["l_dim"], d["l_rot"], d["l_vdim"], d["kv_rank"]
+    latent = 2 * (w * (d["q_rank"] + r + lr + 2 * lh * lv) + d["q_rank"] * lh * (ld + lr) + lh * ld * r + lh * r * lv)
+    total = 0.0
+    for i in range(d["layers"]):
+        mixer = (memory, memory, scored, latent)[i % 4]
+        attention = (0, 0, 4 * d["a_heads"] * d["a_dim"] * seen, lh * causal * (4 * r + 2 * lr))[i % 4]
+        total += (gates + mixer + (dense if i % 4 == 0 else routed)) * tokens + attention
+    return total + 2 * w * d["vocab"]
+
+
+def _topezen_kernel_table(d: dict, f: dict, peak: dict) -> dict:
+    """The new design's kernels alone and the like kernels of the models that were here (the Pofadra decoder's recurrence, norm,
+    gate and router, the Rezulorn decoder's chunked recurrence, scored attention and cache write, the transformer's residual add),
+    each with its share of its roofline."""
+    import torch
+
+    from gtar_kimik3_public_b200.ops import functional as F
+
+    dev = torch.device("cuda:0")
+    flush = torch.zeros(48 << 20, dtype=torch.float32, device=dev)  # 192 MB: larger than the 126 MB L2
+    hbm, tflops = peak["hbm_gbs"] * 1e9, peak["bf16_tflops"] * 1e12
+    out = {}
+
+    def record(name, ms, n_bytes, flops=0.0):
+        floor = max(n_bytes / hbm, flops / tflops) * 1e3
+        out[name] = {"us": round(ms * 1e3, 2), "roofline_us": round(floor * 1e3, 2), "frac": round(floor / ms, 4),
+                     "bound": "hbm" if n_bytes / hbm >= flops / tflops else "tensor"}
+
+    w, H, dk, dv, cap = d["width"], d["heads"], d["dim"], d["vdim"], d["cap"]
+    aq, ak, dim, window, keep = d["a_heads"], d["a_kv"], d["a_dim"], d["window"], d["keep"]
+    bf = torch.bfloat16
+    for label, tokens, n_seqs in (("prefill_2048", 2048, 1), ("decode_b8_ctx2048", 8, 8)):
+        each = tokens // n_seqs
+        inner = 1 if n_seqs == 1 else 20
+        past = 0 if n_seqs == 1 else 2047
+        length = past + each
+        pages_each = -(-length // 64)
+        table = torch.arange(n_seqs * pages_each, dtype=torch.int32, device=dev).view(n_seqs, pages_each)
+        tok_seq = torch.arange(n_seqs, dtype=torch.int32, device=dev).repeat_interleave(each)
+        tok_pos = (torch.arange(each, dtype=torch.int32, device=dev) + past).repeat(n_seqs)
+        cu_q = torch.arange(n_seqs + 1, dtype=torch.int32, device=dev) * each
+        slots = torch.arange(n_seqs, dtype=torch.int32, device=dev)
+        kv_len = torch.full((n_seqs,), length, dtype=torch.int32, device=dev)
+        timed = dict(flush=flush, inner=inner)
+        # ---- the stream
+        hs = torch.randn(tokens, w, device=dev)
+        branch = torch.randn(tokens, w, device=dev).to(bf)
+        wide_branch = torch.randn(tokens, w, device=dev)
+        z = torch.randn(tokens, 2 * w, device=dev).to(bf)
+        wn = torch.ones(w, device=dev)
+        ms = _event_ms(lambda: F.gated_merge(hs, bf, z=z, branch_1=branch, gate_gain_1=1.0, bias_1=wn, branch_2=wide_branch, gate_gain_2=1.0,
+                                             bias_2=wn, gain_1=1.0, gain_2=1.0, next_eps=1e-6), **timed)
+        record(f"topezen both gates, both adds, next norms, {label}", ms, tokens * w * (4 + 2 + 4 + 4 + 4 + 6))
+        ms = _event_ms(lambda: F.add_rmsnorm(hs, branch, wn, 1e-6, bf), **timed)
+        record(f"transformer residual add with next norm, {label}", ms, tokens * w * (4 + 2 + 4 + 2))
+        # ---- the dense feed-forward's activation
+        ff_in = torch.randn(tokens, d["ff"], device=dev).to(torch.float32 if tokens <= 16 else bf)
+        ms = _event_ms(lambda: F.poly_norm(ff_in, (0.5, 0.3, 0.2, 0.1), 1e-6, bf), **timed)
+        record(f"topezen PolyNorm, {label}", ms, tokens * d["ff"] * (ff_in.element_size() + 2))
+        ff_bf = ff_in.to(bf)
+        ms = _event_ms(lambda: F.xielu(ff_bf, 0.8, 1.2), **timed)
+        record(f"zasorax xIELU, {label}", ms, tokens * d["ff"] * 4)
+        # ---- routers
+        hb = torch.randn(tokens, w, device=dev).to(bf)
+        w_r, bias = torch.randn(d["experts"], w, device=dev) * 0.05, torch.randn(d["experts"], device=dev) * 0.01
+        route_bytes = tokens * w * 2 + d["experts"] * w * 4 + tokens * d["top"] * 8
+        ms = _event_ms(lambda: F.route_groups(hb, w_r, bias, d["top"], d["groups"], d["group_keep"], 1.0, softmax=True, best_of_group=True,
+                                              renormalise=True), **timed)
+        record(f"topezen router (softmax, best of a group, renormalised), {label}", ms, route_bytes)
+        ms = _event_ms(lambda: F.route_groups(hb, w_r, bias, d["top"], d["groups"], d["group_keep"], 1.0), **timed)
+        record(f"pofadra router (sigmoid scores, groups), {label}", ms, route_bytes)
+        # ---- the recurrences, each with the norm and gate behind it
+        at = F.MemoryColumns(0, H * dk, 2 * H * dk, 2 * H * dk + H * dv, 2 * H * dk + 2 * H * dv, 2 * H * dk + 2 * H * dv + H)
+        proj = torch.randn(tokens, -(-(at.f + H) // 8) * 8, device=dev).to(bf)
+        gate_bias = torch.cat([torch.zeros(H, device=dev), torch.full((H,), 3.0, device=dev)])
+        norm_w = torch.ones(H * dv, device=dev)
+        state, n_state = torch.zeros(n_seqs, H, dk + 1, dv, device=dev), torch.zeros(n_seqs, H, dk + 1, device=dev)
+        core = (proj, at, gate_bias, cap, state, n_state)
+        state_bytes = 8 * n_seqs * H * (dk + 1) * (dv + 1)
+        memory_bytes = 2 * tokens * (2 * H * dk + 2 * H * dv + 2 * H + H * dv) + state_bytes
+        memory_flops = tokens * H * 4 * dk * dv
+        if n_seqs == 1:
+            ms = _event_ms(lambda: F.memory_chunked(*core, norm_w, 1e-6, cu_q, slots, n_seqs, each), **timed)
+        else:
+            ms = _event_ms(lambda: F.memory_single(*core, norm_w, 1e-6, cu_q, slots, n_seqs), **timed)
+        record(f"topezen matrix memory with norm and gate, {label}", ms, memory_bytes, memory_flops)
+
+        wide_rows = proj.float()  # token by token is the way of 32-bit runs (and of short portions)
+
+        def token_by_token():
+            o, den = F.memory_scan(wide_rows, *core[1:], cu_q, slots, n_seqs)
+            return F.group_norm_gate(o.view(tokens, H * dv), dv, norm_w, wide_rows, at.g, 1e-6, torch.float32, divisor=den)
+
+        ms = _event_ms(token_by_token, repeats=3, **timed)
+        record(f"topezen matrix memory token by token, norm and gate (32-bit run), {label}", ms, 2 * memory_bytes - state_bytes)
+        fh, fk, fv = f["heads"], f["dim"], f["vdim"]
+        q, k = torch.randn(tokens, fh, fk, device=dev) * 0.1, torch.randn(tokens, fh, fk, device=dev) * 0.1
+        v, g, beta = torch.randn(tokens, fh, fv, device=dev), torch.rand(tokens, fh, fk, device=dev), torch.rand(tokens, fh, device=dev)
+        delta_state, low = torch.zeros(n_seqs, fh, fk, fv, device=dev), torch.randn(tokens, fh * fv, device=dev)
+        head_w = torch.ones(fv, device=dev)
+
+        def delta():
+            o = F.delta_scan(q, k, v, g, beta, delta_state, cu_q, slots, n_seqs)
+            return F.head_norm_gate(o, head_w, low, 0, 1e-6, bf)
+
+        ms = _event_ms(delta, **timed)
+        record(f"pofadra delta rule recurrence, norm and gate, {label}", ms,
+               4 * tokens * fh * (3 * fk + 2 * fv + 1) + 2 * tokens * fh * fv + 8 * n_seqs * fh * fk * fv, tokens * fh * 8 * fk * fv)
+        decay = torch.full((fh,), 0.97, device=dev)
+        if n_seqs == 1:
+            scan = lambda: F.decay_scan_chunked(q, k, v, decay, delta_state, cu_q, slots, n_seqs, each)
+        else:
+            scan = lambda: F.decay_scan(q, k, v, decay, delta_state, cu_q, slots, n_seqs)
+        ms = _event_ms(lambda: F.group_norm_gate(scan().view(tokens, fh * fv), fv, head_w, low, 0, 1e-6, bf), **timed)
+        record(f"rezulorn recurrence with a fixed decay, norm and gate, {label}", ms,
+               4 * tokens * fh * (2 * fk + 2 * fv) + 2 * tokens * fh * fv + 8 * n_seqs * fh * fk * fv, tokens * fh * 4 * fk * fv)
+        # ---- scored attention
+        kv = F.PagedKV(torch.randn(n_seqs * pages_each, ak, 64, dim, device=dev).to(bf) * 0.1,
+                       torch.randn(n_seqs * pages_each, ak, 64, dim, device=dev).to(bf) * 0.1, table, F.DecodeWork(dev))
+        wide = torch.randn(tokens, (aq + 2 * ak) * dim, device=dev).to(bf)
+        wq, wk = torch.ones(dim, device=dev), torch.ones(dim, device=dev)
+        prep_bytes = tokens * 2 * ((aq + 2 * ak) * dim + aq * dim + 2 * ak * dim)
+        place = (wide, 0, aq * dim, (aq + ak) * dim, aq, ak, dim, dim, tok_pos, tok_seq, slots)
+        ms = _event_ms(lambda: F.heads_prepare(*place, unit_eps=1e-6, w_q=wq, w_k=wk, kv=kv, max_position=length - 1), **timed)
+        record(f"topezen norm per head and cache write, {label}", ms, prep_bytes)
+        angle = torch.arange(length, dtype=torch.float32, device=dev)[:, None] * torch.rand(dim // 2, device=dev)[None, :]
+        cos, sin = angle.cos().contiguous(), angle.sin().contiguous()
+        ms = _event_ms(lambda: F.heads_prepare(*place, rot=dim, cos=cos, sin=sin, unit_eps=1e-6, kv=kv, max_position=length - 1), **timed)
+        record(f"rezulorn rotation, unit q and k, cache write, {label}", ms, prep_bytes)
+        qa = torch.randn(tokens, aq, dim, device=dev).to(bf)
+        sink = torch.full((aq,), 0.5, device=dev)
+        seen = sum(min(p + 1, window) + min(keep, max(0, p + 1 - window)) for p in range(past, length)) * n_seqs
+        attn_bytes = 2 * (2 * tokens * aq * dim + 2 * n_seqs * min(length, window + keep + each) * ak * dim)
+        parts = F.scored_attention_parts(n_seqs, aq, ak, each, -(-(window + keep) // 64) + 2, F.sm_count(dev))
+        ms = _event_ms(lambda: F.attention_scored(qa, kv, cu_q, kv_len, slots, each, dim ** -0.5, window, keep, n_parts=parts, sink=sink,
+                                                  softcap=d["softcap"]), **timed)
+        record(f"topezen attention: capped scores, window {window} keeping {keep}, learned sink, {label}", ms, attn_bytes, 4 * aq * dim * seen)
+        r1, r2 = torch.full((aq,), 0.3, device=dev), torch.full((aq,), 0.5, device=dev)
+        ms = _event_ms(lambda: F.attention_scored(qa, kv, cu_q, kv_len, slots, each, dim ** -0.5, window, keep, r1, r2, None, "softmax", parts),
+                       **timed)
+        record(f"rezulorn attention: distance term, window {window} keeping {keep}, {label}", ms, attn_bytes, 4 * aq * dim * seen)
+        # ---- latent attention (the Dasusun decoder's kernels; no window here)
+        lh, ld, lr, r = d["l_heads"], d["l_dim"], d["l_rot"], d["kv_rank"]
+        rows = F.PagedRows(torch.randn(n_seqs * pages_each, 64, r + lr, device=dev).to(bf) * 0.1, table)
+        l_angle = torch.arange(length, dtype=torch.float32, device=dev)[:, None] * torch.rand(lr // 2, device=dev)[None, :]
+        l_cos, l_sin = l_angle.cos().contiguous(), l_angle.sin().contiguous()
+        carried, mixed = torch.randn(lh, tokens, r, device=dev).to(bf), torch.empty(lh, tokens, r, dtype=bf, device=dev)
+        q_raw = torch.randn(tokens, lh, ld + lr, device=dev).to(bf)
+        splits = 1 if n_seqs == 1 else F.latent_splits(n_seqs, lh, length, 0, F.sm_count(dev))
+        causal = sum(p + 1 for p in range(past, length)) * n_seqs
+        ms = _event_ms(lambda: F.attention_latent_tiled(carried.transpose(0, 1), q_raw, ld, lr, lr, l_cos, l_sin, rows, tok_pos, cu_q, slots,
+                                                        (ld + lr) ** -0.5, 0, mixed.transpose(0, 1), n_seqs, each, splits), **timed)
+        record(f"topezen latent attention (dasusun's kernel, no window), {label}", ms,
+               2 * (tokens * lh * (2 * r + ld + lr) + n_seqs * length * (r + lr)), lh * causal * (4 * r + 2 * lr))
+        flat, gate_src = torch.randn(tokens, lh * d["l_vdim"], device=dev).to(bf), torch.randn(tokens, lh * d["l_vdim"], device=dev).to(bf)
+        ms = _event_ms(lambda: F.sigmoid_gate(flat, gate_src, 0), **timed)
+        record(f"topezen output gate (pofadra's kernel), {label}", ms, tokens * lh * d["l_vdim"] * 6)
+    return out
+
+
+def run_compare_topezen(args) -> dict:
+    import gc
+
+    import torch
+
+    from gtar_kimik3_public_b200.ops.library import require_device
+
+    require_device(torch.device("cuda:0"))
+    peak, peak_source = peaks()
+    results = {}
+    for name, (d, f) in TOPEZEN_SIZES.items():
+        entry = {}
+        for arch, raw, flops in (("topezen", _topezen_config(**d), _topezen_prefill_flops(d, PREFILL_TOKENS)),
+                                 ("pofadra", _pofadra_config(**f), _pofadra_prefill_flops(f, PREFILL_TOKENS))):
+            model = _device_model(raw)
+            ms = _time_prefill_ms(model, PREFILL_TOKENS)
+            decode = time_decode(model, args.batch, min(args.steps, 64), args.warmup)
+            entry[arch] = {
+                "weight_bytes_per_step": model.weight_bytes_per_step(),
+                "prefill_tokens_per_s": round(PREFILL_TOKENS / (ms / 1e3), 1), "prefill_ms": round(ms, 3),
+                "prefill_frac_of_bf16_peak": round(flops / (ms / 1e3) / (peak["bf16_tflops"] * 1e12), 4),
+                "decode_tokens_per_s": round(decode["tokens_per_s"], 1), "decode_ms_per_step": round(decode["ms_per_step"], 4),
+                "decode_frac_of_hbm_peak": round(decode["bytes_per_step"] / (decode["ms_per_step"] / 1e3) / 1e9 / peak["hbm_gbs"], 4),
+                "decode_launches_per_step": decode["launches"] // max(1, min(args.steps, 64)),
+            }
+            # a step's weight bytes count the experts ONE token reads; a batch reads every distinct expert its tokens
+            # choose: with uniform choices E (1 - (1 - top / E)^batch) of them in every routed layer
+            sizes, expert_ff = (d, d["expert_ff"]) if arch == "topezen" else (f, f["ff"])
+            distinct = sizes["experts"] * (1.0 - (1.0 - sizes["top"] / sizes["experts"]) ** args.batch)
+            routed_layers = sum(1 for layer in raw["layers"] if layer["mlp"]["kind"] == "moe")
+            more = routed_layers * (distinct - sizes["top"]) * 3 * expert_ff * sizes["width"] * 2
+            entry[arch]["decode_expected_distinct_experts"] = round(distinct, 1)
+            entry[arch]["decode_frac_of_hbm_peak_with_distinct_experts"] = round(
+                (decode["bytes_per_step"] + more) / (decode["ms_per_step"] / 1e3) / 1e9 / peak["hbm_gbs"], 4)
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+        entry["kernels"] = _topezen_kernel_table(d, f, peak)
+        results[name] = {"sizes": {"topezen": d, "pofadra": f}, **entry}
+    return {"compare": "topezen beside pofadra at equal width", "batch": args.batch, "prompt_tokens": PROMPT_LEN,
+            "prefill_tokens": PREFILL_TOKENS, "dtype": "bf16", "data": "synthetic: random token ids, random weights drawn on the device",
+            "peaks": dict(peak, source=peak_source), "l2": "single kernels: a 192 MB buffer is written between the timed calls of the 2,048-token cases; the 8-token cases are 20 calls back to back from a CUDA graph",
+            "results": results}
+
+
 def main() -> int:
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -1495,13 +1744,13 @@ def main() -> int:
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--layers", type=int, default=None, help="fewer layers than the configuration (named in config)")
     parser.add_argument("--no-large", action="store_true", help="leave out the points at the 4B and 8B layer sizes")
-    parser.add_argument("--compare", default=None, choices=["dasusun", "pofadra", "rezulorn", "zasorax"],
+    parser.add_argument("--compare", default=None, choices=["dasusun", "pofadra", "rezulorn", "zasorax", "topezen"],
                         help="instead of the default workload: this architecture beside the transformer at equal layer sizes")
     args = parser.parse_args()
     if args.compare:
         if args.warmup < 3:
             args.warmup = 3
-        runner = {"pofadra": run_compare_pofadra, "rezulorn": run_compare_rezulorn, "zasorax": run_compare_zasorax, "dasusun": run_compare}[args.compare]
+        runner = {"pofadra": run_compare_pofadra, "rezulorn": run_compare_rezulorn, "zasorax": run_compare_zasorax, "topezen": run_compare_topezen, "dasusun": run_compare}[args.compare]
         print(json.dumps(runner(args)))
         return 0
     if args.impl == "reference":

@@ -9,7 +9,7 @@
 // The state in memory: C with one more row [slots, H, d + 1, dv] and n with one more entry [slots, H, d + 1]; the extra
 // row and entry hold m, a copy for every column, so blocks that own different columns never touch one another's numbers.
 //
-// memory_single is the step of one token a sequence with the norm of the head, its weight and the sigmoid gate in the same
+// memory_single is the bfloat16 step of one token a sequence with the norm of the head, its weight and the sigmoid gate in the same
 // kernel: a cluster of blocks per (sequence, head), 64 value columns a block, one exchange of the blocks' sums of squares.
 
 #include "matrix_memory.cuh"
@@ -21,29 +21,98 @@ using namespace memory;
 constexpr int LANES = 8;      // lanes that share a column of the state
 constexpr int MAX_COLS = 32;  // columns a block at most (256 threads)
 
-// A column's d entries are spread over eight adjacent lanes, R consecutive rows a lane; TB tokens are staged at a time.
-template <typename T, int R, int TB>
-__global__ void __launch_bounds__(LANES * MAX_COLS) memory_scan_kernel(
-    const T* __restrict__ proj, long long ld, Columns at, const float* __restrict__ gate_bias, float cap, float k_scale,
-    float* __restrict__ state, float* __restrict__ n_state, float* __restrict__ out, float* __restrict__ den,
-    const int* __restrict__ cu_q, const int* __restrict__ slots, int n_heads, int d, int dv) {
-    constexpr int PIECE = R == 4 ? 4 : R + 4, VEC = LANES * PIECE;  // a lane's piece starts a bank group apart from its neighbours'
-    __shared__ __align__(16) float sq[TB][VEC], sk[TB][VEC];
-    __shared__ float sv[TB][MAX_COLS];
-    __shared__ float s_old[TB], s_new[TB], s_top[TB];
+// The gates of a sequence's tokens, a warp per (sequence, head): gates [T, H] = (e^(f + m - m'), e^(i - m'), m', 0).  The running
+// maximum goes from token to token in order, so it does not depend on how a prompt is cut.
+template <typename T>
+__global__ void __launch_bounds__(32) memory_gates_kernel(const T* __restrict__ proj, long long ld, Columns at,
+                                                          const float* __restrict__ gate_bias, float cap, const float* __restrict__ n_state,
+                                                          float4* __restrict__ gates, const int* __restrict__ cu_q,
+                                                          const int* __restrict__ slots, int n_heads, int d) {
     pdl_launch_dependents();
-    const int n_threads = blockDim.x, n_cols = n_threads / LANES;
-    const int seq = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * n_cols;
-    const int sub = threadIdx.x % LANES, col = col0 + threadIdx.x / LANES;
-    const bool live = col <= dv;   // column dv is n
-    const bool is_n = col == dv;
-    for (int i = threadIdx.x; i < TB * VEC; i += n_threads) {  // the pieces beyond d stay zero
-        (&sq[0][0])[i] = 0.f;
-        (&sk[0][0])[i] = 0.f;
-    }
+    const int head = blockIdx.x, seq = blockIdx.y, lane = threadIdx.x;
     const float bias_i = gate_bias[head], bias_f = gate_bias[n_heads + head];
     pdl_wait();
     const int t0 = cu_q[seq], n = cu_q[seq + 1] - t0;
+    if (n <= 0) return;
+    float m = n_state[((size_t)slots[seq] * n_heads + head) * (d + 1) + d];
+    float z_i = 0.f, z_f = 0.f;
+    auto fetch = [&](int first) {
+        if (first + lane < n) {
+            const T* row = proj + (size_t)(t0 + first + lane) * ld;
+            z_i = to_float(row[at.i + head]);
+            z_f = to_float(row[at.f + head]);
+        }
+    };
+    fetch(0);
+    for (int first = 0; first < n; first += 32) {
+        const float i = log_input_gate(z_i + bias_i, cap), f = log_forget_gate(z_f + bias_f, cap);
+        if (first + 32 < n) fetch(first + 32);
+        const int count = min(32, n - first);
+        float before = 0.f, after = 0.f;
+#pragma unroll 8
+        for (int tt = 0; tt < count; ++tt) {
+            const float fi = __shfl_sync(0xffffffffu, f, tt), ii = __shfl_sync(0xffffffffu, i, tt);
+            const float m_new = fmaxf(fi + m, ii);
+            if (lane == tt) {
+                before = m;
+                after = m_new;
+            }
+            m = m_new;
+        }
+        if (lane < count) gates[(size_t)(t0 + first + lane) * n_heads + head] = make_float4(expf(f + before - after), expf(i - after), after, 0.f);
+    }
+}
+
+template <int BYTES>
+__device__ __forceinline__ void copy_async(void* smem, const void* gmem) {
+    if constexpr (BYTES == 16)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem));
+    else
+        asm volatile("cp.async.ca.shared.global [%0], [%1], %2;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem), "n"(BYTES));
+}
+
+// 16 bytes of a row in shared memory as 32-bit numbers
+__device__ __forceinline__ void row_piece(const float* p, float (&v)[4]) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x, v[1] = x.y, v[2] = x.z, v[3] = x.w;
+}
+__device__ __forceinline__ void row_piece(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+        const float2 x = __bfloat1622float2(h[c]);
+        v[2 * c] = x.x, v[2 * c + 1] = x.y;
+    }
+}
+
+// A column's d entries are spread over eight adjacent lanes, R consecutive rows a lane.  The step's tokens come through a
+// two-stage cp.async ring, TB at a time, in the projection's type (VEC: its rows and their parts are whole 16-byte pieces).
+template <typename T, int R, int TB, bool VEC>
+__global__ void __launch_bounds__(LANES * MAX_COLS) memory_scan_kernel(
+    const T* __restrict__ proj, long long ld, Columns at, const float4* __restrict__ gates, float k_scale, float* __restrict__ state,
+    float* __restrict__ n_state, float* __restrict__ out, float* __restrict__ den, const int* __restrict__ cu_q,
+    const int* __restrict__ slots, int n_heads, int d, int dv) {
+    constexpr int PER16 = 16 / sizeof(T);
+    constexpr int PIECE = R + PER16, ROW = LANES * PIECE;  // a lane's piece starts a bank group apart from its neighbours'
+    static_assert(R % PER16 == 0, "a lane's rows are whole pieces");
+    __shared__ __align__(16) T sq[2][TB][ROW], sk[2][TB][ROW];
+    __shared__ __align__(16) T sv[2][TB][MAX_COLS];
+    __shared__ float4 sg[2][TB];
+    pdl_launch_dependents();
+    const int n_threads = blockDim.x, n_cols = n_threads / LANES;
+    const int seq = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * n_cols;
+    const int sub = threadIdx.x % LANES, my_col = threadIdx.x / LANES, col = col0 + my_col;
+    const bool live = col <= dv;   // column dv is n
+    const bool is_n = col == dv;
+    for (int i = threadIdx.x; i < 2 * TB * ROW; i += n_threads) {  // the pieces beyond d stay zero
+        (&sq[0][0][0])[i] = from_float<T>(0.f);
+        (&sk[0][0][0])[i] = from_float<T>(0.f);
+    }
+    __syncthreads();
+    pdl_wait();
+    const int t0 = cu_q[seq], n = cu_q[seq + 1] - t0;
+    if (n <= 0) return;
     const size_t slot_head = (size_t)slots[seq] * n_heads + head;
     float* column = is_n ? n_state + slot_head * (d + 1) : state + slot_head * (d + 1) * dv + col;
     const size_t stride = is_n ? 1 : dv;
@@ -53,58 +122,63 @@ __global__ void __launch_bounds__(LANES * MAX_COLS) memory_scan_kernel(
         const int row = sub * R + r;
         S[r] = (live && row < d) ? column[(size_t)row * stride] : 0.f;
     }
-    float top = live ? column[(size_t)d * stride] : 0.f;  // the same number in every column
-    for (int first = 0; first < n; first += TB) {
+    auto stage = [&](int buf, int first) {
         const int count = min(TB, n - first);
-        __syncthreads();  // the tokens of before are done with
-        for (int i = threadIdx.x; i < count * d; i += n_threads) {
-            const int tt = i / d, c = i - tt * d;
-            const int to = (c / R) * PIECE + c % R;
-            const T* row = proj + (size_t)(t0 + first + tt) * ld;
-            sq[tt][to] = to_float(row[at.q + head * d + c]);
-            sk[tt][to] = to_float(row[at.k + head * d + c]) * k_scale;
-        }
-        for (int i = threadIdx.x; i < count * n_cols; i += n_threads) {
-            const int tt = i / n_cols, cc = i - tt * n_cols;
-            const int vc = col0 + cc;
-            sv[tt][cc] = vc < dv ? to_float(proj[(size_t)(t0 + first + tt) * ld + at.v + head * dv + vc]) : vc == dv ? 1.f : 0.f;
-        }
-        for (int tt = threadIdx.x; tt < count; tt += n_threads) {
-            const T* row = proj + (size_t)(t0 + first + tt) * ld;
-            s_new[tt] = log_input_gate(to_float(row[at.i + head]) + bias_i, cap);
-            s_old[tt] = log_forget_gate(to_float(row[at.f + head]) + bias_f, cap);
-        }
-        __syncthreads();
-        if (threadIdx.x == 0) {  // the running maximum, one token after another
-            float m = top;
-            for (int tt = 0; tt < count; ++tt) {
-                const float f = s_old[tt], i = s_new[tt], m_new = fmaxf(f + m, i);
-                s_old[tt] = f + m - m_new;
-                s_new[tt] = i - m_new;
-                s_top[tt] = m = m_new;
+        const T* row0 = proj + (size_t)(t0 + first) * ld + head * d;
+        const T* v0 = proj + (size_t)(t0 + first) * ld + at.v + head * dv + col0;
+        if constexpr (VEC) {
+            const int pieces = d / PER16;
+            for (int i = threadIdx.x; i < count * pieces; i += n_threads) {
+                const int tt = i / pieces, c = (i - tt * pieces) * PER16, to = (c / R) * PIECE + c % R;
+                copy_async<16>(&sq[buf][tt][to], row0 + (size_t)tt * ld + at.q + c);
+                copy_async<16>(&sk[buf][tt][to], row0 + (size_t)tt * ld + at.k + c);
+            }
+            const int quads = n_cols / 4;
+            for (int i = threadIdx.x; i < count * quads; i += n_threads) {
+                const int tt = i / quads, c = (i - tt * quads) * 4;
+                if (col0 + c < dv) copy_async<4 * sizeof(T)>(&sv[buf][tt][c], v0 + (size_t)tt * ld + c);
+            }
+        } else {
+            for (int i = threadIdx.x; i < count * d; i += n_threads) {
+                const int tt = i / d, c = i - tt * d, to = (c / R) * PIECE + c % R;
+                sq[buf][tt][to] = row0[(size_t)tt * ld + at.q + c];
+                sk[buf][tt][to] = row0[(size_t)tt * ld + at.k + c];
+            }
+            for (int i = threadIdx.x; i < count * n_cols; i += n_threads) {
+                const int tt = i / n_cols, c = i - tt * n_cols;
+                if (col0 + c < dv) sv[buf][tt][c] = v0[(size_t)tt * ld + c];
             }
         }
-        __syncthreads();
-        for (int tt = threadIdx.x; tt < 2 * count; tt += n_threads) {
-            if (tt < count) s_old[tt] = expf(s_old[tt]);
-            else s_new[tt - count] = expf(s_new[tt - count]);
+        for (int tt = threadIdx.x; tt < count; tt += n_threads) copy_async<16>(&sg[buf][tt], gates + (size_t)(t0 + first + tt) * n_heads + head);
+        asm volatile("cp.async.commit_group;\n" ::);
+    };
+    stage(0, 0);
+    float top = 0.f;
+    int buf = 0;
+    for (int first = 0; first < n; first += TB, buf ^= 1) {
+        if (first + TB < n) {
+            stage(buf ^ 1, first + TB);
+            asm volatile("cp.async.wait_group 1;\n" ::);
+        } else {
+            asm volatile("cp.async.wait_group 0;\n" ::);
         }
         __syncthreads();
-        top = s_top[count - 1];
-        const float4* pq = reinterpret_cast<const float4*>(&sq[0][sub * PIECE]);
-        const float4* pk = reinterpret_cast<const float4*>(&sk[0][sub * PIECE]);
-        for (int tt = 0; tt < count; ++tt, pq += VEC / 4, pk += VEC / 4) {
-            const float keep = s_old[tt], vv = s_new[tt] * sv[tt][threadIdx.x / LANES];
-            float b4[4] = {0.f, 0.f, 0.f, 0.f};
+        const int count = min(TB, n - first);
+#pragma unroll 2
+        for (int tt = 0; tt < count; ++tt) {
+            const float4 g = sg[buf][tt];
+            const float v = is_n ? 1.f : live ? to_float(sv[buf][tt][my_col]) : 0.f;
+            const float vv = g.y * k_scale * v;
+            float b4[4] = {0.f, 0.f, 0.f, 0.f};  // four partial sums: chains of R / 4 dependent operations
 #pragma unroll
-            for (int r4 = 0; r4 < R / 4; ++r4) {
-                const float4 k4 = pk[r4], q4 = pq[r4];
-                const float ks[4] = {k4.x, k4.y, k4.z, k4.w}, qs[4] = {q4.x, q4.y, q4.z, q4.w};
+            for (int r0 = 0; r0 < R; r0 += PER16) {
+                float ks[PER16], qs[PER16];
+                row_piece(&sk[buf][tt][sub * PIECE + r0], ks);
+                row_piece(&sq[buf][tt][sub * PIECE + r0], qs);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int r = 4 * r4 + e;
-                    S[r] = fmaf(ks[e], vv, keep * S[r]);
-                    b4[e] = fmaf(S[r], qs[e], b4[e]);
+                for (int e = 0; e < PER16; ++e) {
+                    S[r0 + e] = fmaf(ks[e], vv, g.x * S[r0 + e]);
+                    b4[e & 3] = fmaf(S[r0 + e], qs[e], b4[e & 3]);
                 }
             }
             float b = (b4[0] + b4[1]) + (b4[2] + b4[3]);
@@ -112,10 +186,12 @@ __global__ void __launch_bounds__(LANES * MAX_COLS) memory_scan_kernel(
             for (int o = 1; o < LANES; o <<= 1) b += __shfl_xor_sync(0xffffffffu, b, o);
             if (live && sub == 0) {
                 const size_t row = (size_t)(t0 + first + tt) * n_heads + head;
-                if (is_n) den[row] = fmaxf(fabsf(b), expf(-s_top[tt])) + DEN_ADD;
+                if (is_n) den[row] = fmaxf(fabsf(b), expf(-g.z)) + DEN_ADD;
                 else out[row * dv + col] = b;
             }
+            top = g.z;
         }
+        __syncthreads();  // the stage is free for the load after next
     }
 #pragma unroll
     for (int r = 0; r < R; ++r) {
@@ -130,10 +206,10 @@ constexpr int ONE_THREADS = 256, ONE_COLS = 64, ONE_LANES = ONE_COLS / 4, ONE_GR
 // Sixteen threads side by side own four columns each, sixteen groups of them every sixteenth row (R rows a group): a thread
 // has all its rows' loads in flight at once.  n is updated by every block for itself, written by the cluster's first block once
 // all of them have read it.
-template <typename T, int R>
+template <int R>
 __global__ void __launch_bounds__(ONE_THREADS) memory_single_kernel(
-    const T* __restrict__ proj, long long ld, Columns at, int g_at, const float* __restrict__ gate_bias, float cap, float k_scale,
-    float* __restrict__ state, float* __restrict__ n_state, const float* __restrict__ norm_w, float eps, T* __restrict__ y,
+    const __nv_bfloat16* __restrict__ proj, long long ld, Columns at, int g_at, const float* __restrict__ gate_bias, float cap, float k_scale,
+    float* __restrict__ state, float* __restrict__ n_state, const float* __restrict__ norm_w, float eps, __nv_bfloat16* __restrict__ y,
     const int* __restrict__ cu_q, const int* __restrict__ slots, int n_heads, int d, int dv) {
     constexpr int D = R * ONE_GROUPS, PER = (D + ONE_THREADS - 1) / ONE_THREADS;
     __shared__ float sq[D], sk[D];
@@ -158,7 +234,7 @@ __global__ void __launch_bounds__(ONE_THREADS) memory_single_kernel(
         const int row = grp + r * ONE_GROUPS;
         S[r] = live && row < d ? *reinterpret_cast<const float4*>(own + (size_t)row * dv) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    const T* row = proj + (size_t)t * ld;
+    const __nv_bfloat16* row = proj + (size_t)t * ld;
     float n_new[PER];
     const float m = own_n[d];
     const float i = log_input_gate(to_float(row[at.i + head]) + bias_i, cap);
@@ -180,7 +256,7 @@ __global__ void __launch_bounds__(ONE_THREADS) memory_single_kernel(
     }
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (live) {
-        const T* vr = row + at.v + head * dv + col;
+        const __nv_bfloat16* vr = row + at.v + head * dv + col;
         v = make_float4(to_float(vr[0]), to_float(vr[1]), to_float(vr[2]), to_float(vr[3]));
     }
     dot = block_sum(dot, scratch);  // its barriers also publish sq and sk
@@ -226,18 +302,17 @@ __global__ void __launch_bounds__(ONE_THREADS) memory_single_kernel(
         for (int w = 0; w < tiles; ++w) total += squares[w];
         const float r = 1.f / sqrtf(total / (float)dv + eps);
         const float z = to_float(row[g_at + head * dv + mine]);
-        y[(size_t)t * n_heads * dv + head * dv + mine] = from_float<T>(num * r * norm_w[head * dv + mine] / (1.f + expf(-z)));
+        y[(size_t)t * n_heads * dv + head * dv + mine] = __float2bfloat16_rn(num * r * norm_w[head * dv + mine] / (1.f + expf(-z)));
         state[slot_head * (size_t)(d + 1) * dv + (size_t)d * dv + mine] = m_new;
     }
 }
 
 }  // namespace
 
-// One token a sequence: the recurrence, the heads' norm and the gate.  y [n_tokens, H dv] in the run's type.
-GK_EXPORT int gk_memory_single(const void* proj, int dtype, long long ld, int q_at, int k_at, int v_at, int g_at, int i_at, int f_at,
+// One token a sequence: the recurrence, the heads' norm and the gate, bfloat16 rows; y [n_tokens, H dv].
+GK_EXPORT int gk_memory_single(const void* proj, long long ld, int q_at, int k_at, int v_at, int g_at, int i_at, int f_at,
                                const float* gate_bias, float cap, float* state, float* n_state, const float* norm_w, float eps, void* y,
                                const int* cu_q, const int* slots, int n_seqs, int n_heads, int d, int dv, void* stream) {
-    GK_REQUIRE(GK_VALID_DTYPE(dtype), "memory_single: bad dtype %d", dtype);
     GK_REQUIRE(n_heads > 0 && n_heads <= 65535 && n_seqs >= 0 && n_seqs <= 65535, "memory_single: bad counts");
     GK_REQUIRE(d > 0 && d <= 512 && dv > 0 && dv % 4 == 0 && dv <= 8 * ONE_COLS, "memory_single: heads of %d / %d do not fit", d, dv);
     GK_REQUIRE(cap > 0.f && eps > 0.f, "memory_single: cap and eps must be positive");
@@ -247,26 +322,25 @@ GK_EXPORT int gk_memory_single(const void* proj, int dtype, long long ld, int q_
     const float k_scale = 1.f / sqrtf((float)d);
     cudaStream_t s = (cudaStream_t)stream;
 #define GK_ONE(R)                                                                                                                    \
-    gk_launch_cluster(memory_single_kernel<T, R>, dim3(tiles, n_heads, n_seqs), dim3(ONE_THREADS), 0, s, dim3(tiles, 1, 1), (const T*)proj, \
-                      ld, at, g_at, gate_bias, cap, k_scale, state, n_state, norm_w, eps, (T*)y, cu_q, slots, n_heads, d, dv)
-    GK_DISPATCH_DTYPE(dtype, T, {
-        if (d <= 64) GK_ONE(4);
-        else if (d <= 128) GK_ONE(8);
-        else if (d <= 256) GK_ONE(16);
-        else GK_ONE(32);
-    })
+    gk_launch_cluster(memory_single_kernel<R>, dim3(tiles, n_heads, n_seqs), dim3(ONE_THREADS), 0, s, dim3(tiles, 1, 1), (const __nv_bfloat16*)proj, \
+                      ld, at, g_at, gate_bias, cap, k_scale, state, n_state, norm_w, eps, (__nv_bfloat16*)y, cu_q, slots, n_heads, d, dv)
+    if (d <= 64) GK_ONE(4);
+    else if (d <= 128) GK_ONE(8);
+    else if (d <= 256) GK_ONE(16);
+    else GK_ONE(32);
 #undef GK_ONE
     GK_CHECK_LAUNCH("memory_single");
     return GK_OK;
 }
 
+// `gates` holds n_tokens * H * 4 floats.
 GK_EXPORT int gk_memory_scan(const void* proj, int dtype, long long ld, int q_at, int k_at, int v_at, int i_at, int f_at,
-                             const float* gate_bias, float cap, float* state, float* n_state, float* out, float* den, const int* cu_q,
-                             const int* slots, int n_seqs, int n_heads, int d, int dv, void* stream) {
+                             const float* gate_bias, float cap, float* state, float* n_state, float* gates, float* out, float* den,
+                             const int* cu_q, const int* slots, int n_seqs, int n_heads, int d, int dv, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(dtype), "memory_scan: bad dtype %d", dtype);
     GK_REQUIRE(n_heads > 0 && n_heads <= 65535 && n_seqs >= 0 && n_seqs <= 65535, "memory_scan: bad counts");
     GK_REQUIRE(d > 0 && d <= 512 && dv > 0, "memory_scan: key size %d must be at most 512, value size %d positive", d, dv);
-    GK_REQUIRE(cap > 0.f, "memory_scan: the gates' cap must be positive");
+    GK_REQUIRE(cap > 0.f && reinterpret_cast<uintptr_t>(gates) % 16 == 0, "memory_scan: the gates' cap must be positive, their array aligned");
     if (n_seqs == 0) return GK_OK;
     const int sms = memory::sm_count();
     // fewer columns a block while the blocks do not fill the device twice: a column's sums do not depend on the block's shape
@@ -275,13 +349,24 @@ GK_EXPORT int gk_memory_scan(const void* proj, int dtype, long long ld, int q_at
     const dim3 grid((dv + cols) / cols, n_heads, n_seqs), block(cols * LANES);  // dv + 1 columns, rounded up
     const memory::Columns at = {q_at, k_at, v_at, i_at, f_at};
     const float k_scale = 1.f / sqrtf((float)d);
+    const int per16 = dtype == GK_F32 ? 4 : 8;
+    const bool vec = d % per16 == 0 && dv % 4 == 0 && ld % per16 == 0 && q_at % per16 == 0 && k_at % per16 == 0 && v_at % 4 == 0 &&
+                     reinterpret_cast<uintptr_t>(proj) % 16 == 0;
     cudaStream_t s = (cudaStream_t)stream;
 #define GK_SCAN(R, TB)                                                                                                               \
-    gk_launch(memory_scan_kernel<T, R, TB>, grid, block, 0, s, (const T*)proj, ld, at, gate_bias, cap, k_scale, state, n_state, out, den, \
-              cu_q, slots, n_heads, d, dv)
+    do {                                                                                                                             \
+        if (vec)                                                                                                                     \
+            gk_launch(memory_scan_kernel<T, R, TB, true>, grid, block, 0, s, (const T*)proj, ld, at, (const float4*)gates, k_scale,  \
+                      state, n_state, out, den, cu_q, slots, n_heads, d, dv);                                                        \
+        else                                                                                                                         \
+            gk_launch(memory_scan_kernel<T, R, TB, false>, grid, block, 0, s, (const T*)proj, ld, at, (const float4*)gates, k_scale, \
+                      state, n_state, out, den, cu_q, slots, n_heads, d, dv);                                                        \
+    } while (0)
     GK_DISPATCH_DTYPE(dtype, T, {
-        if (d <= 32) GK_SCAN(4, 16);
-        else if (d <= 64) GK_SCAN(8, 16);
+        gk_launch(memory_gates_kernel<T>, dim3(n_heads, n_seqs), dim3(32), 0, s, (const T*)proj, ld, at, gate_bias, cap, (const float*)n_state,
+                  (float4*)gates, cu_q, slots, n_heads, d);
+        GK_CHECK_LAUNCH("memory_gates");
+        if (d <= 64) GK_SCAN(8, 16);
         else if (d <= 128) GK_SCAN(16, 16);
         else if (d <= 256) GK_SCAN(32, 8);
         else GK_SCAN(64, 4);

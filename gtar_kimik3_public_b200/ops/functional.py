@@ -1975,8 +1975,9 @@ def memory_scan(proj: torch.Tensor, at: MemoryColumns, gate_bias: torch.Tensor, 
     T = proj.shape[0]
     out = torch.empty((T, H, dv), dtype=torch.float32, device=proj.device)
     den = torch.empty((T, H), dtype=torch.float32, device=proj.device)
+    gates = torch.empty((T, H, 4), dtype=torch.float32, device=proj.device)
     call("gk_memory_scan", ptr(proj), dtype_code(proj.dtype), proj.shape[1], at.q, at.k, at.v, at.i, at.f, ptr(gate_bias), float(cap),
-         ptr(state), ptr(n_state), ptr(out), ptr(den), ptr(cu_q), ptr(slots), int(n_seqs), H, d, dv, stream_ptr())
+         ptr(state), ptr(n_state), ptr(gates), ptr(out), ptr(den), ptr(cu_q), ptr(slots), int(n_seqs), H, d, dv, stream_ptr())
     return out, den
 
 
@@ -1993,15 +1994,16 @@ def _check_memory_norm(norm_w: torch.Tensor, H: int, dv: int) -> None:
 
 def memory_single(proj: torch.Tensor, at: MemoryColumns, gate_bias: torch.Tensor, cap: float, state: torch.Tensor, n_state: torch.Tensor,
                   norm_w: torch.Tensor, eps: float, cu_q: torch.Tensor, slots: torch.Tensor, n_seqs: int) -> torch.Tensor:
-    """:func:`memory_scan` for steps of one token a sequence, with the division, the norm of every head, ``norm_w [H dv]`` and the
-    sigmoid of the gate's columns in the same kernel.  Returns ``[T, H dv]`` in the projection's type."""
+    """:func:`memory_scan` for bfloat16 steps of one token a sequence, with the division, the norm of every head, ``norm_w [H dv]`` and the
+    sigmoid of the gate's columns in the same kernel.  Returns ``[T, H dv]`` in bfloat16."""
     require_device(proj.device)
     H, d, dv = _check_memory(proj, at, gate_bias, state, n_state)
+    _check(proj, "proj", torch.bfloat16, 2)
     _check_memory_norm(norm_w, H, dv)
     if not memory_single_fits(d, dv) or proj.shape[0] != n_seqs:
         raise KernelError(f"memory_single: {proj.shape[0]} tokens of {n_seqs} sequences, heads of {d} / {dv}")
     y = torch.empty((proj.shape[0], H * dv), dtype=proj.dtype, device=proj.device)
-    call("gk_memory_single", ptr(proj), dtype_code(proj.dtype), proj.shape[1], at.q, at.k, at.v, at.g, at.i, at.f, ptr(gate_bias),
+    call("gk_memory_single", ptr(proj), proj.shape[1], at.q, at.k, at.v, at.g, at.i, at.f, ptr(gate_bias),
          float(cap), ptr(state), ptr(n_state), ptr(norm_w), float(eps), ptr(y), ptr(cu_q), ptr(slots), int(n_seqs), H, d, dv, stream_ptr())
     return y
 

@@ -94,9 +94,9 @@ _SIGNATURES: dict[str, list] = {
     "gk_attention_scored_exact": [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, P, P, I, P, F, P],
     "gk_gated_merge": [P, I, P, L, P, P, I, P, P, F, F, P, P, P, F, F, F, I, I, P],
     "gk_poly_norm": [P, I, P, I, I, I, F, F, F, F, F, P],
-    "gk_memory_single": [P, I, L, I, I, I, I, I, I, P, F, P, P, P, F, P, P, P, I, I, I, I, P],
+    "gk_memory_single": [P, L, I, I, I, I, I, I, P, F, P, P, P, F, P, P, P, I, I, I, I, P],
     "gk_memory_chunked": [P, L, I, I, I, I, I, I, P, F, P, P, P, F, P, P, P, P, P, P, I, I, I, I, I, I, P],
-    "gk_memory_scan": [P, I, L, I, I, I, I, I, P, F, P, P, P, P, P, P, I, I, I, I, P],
+    "gk_memory_scan": [P, I, L, I, I, I, I, I, P, F, P, P, P, P, P, P, P, I, I, I, I, P],
     "gk_attention_scored_bf16": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, I, P, P, I, P, F, P],
 }
 

@@ -20,9 +20,10 @@ entry, ``[heads, d + 1]``.  The last row and entry hold ``m``: a copy for every 
 blocks that own different columns of one head read and write nothing of one another's.
 
 A step's kernels: the packed projection q | k | v | g | i | f; the recurrence, which reads it as it is; norm and gate; the
-output projection.  In steps of one token a sequence the recurrence, norm and gate are one kernel.  In bfloat16 steps of many
-tokens the recurrence runs in chunks of 64 tokens whose inner work is matrix products; short portions and 32-bit runs go
-token by token (in a 32-bit run a token's sums have the same order however a prompt is cut).
+output projection.  In bfloat16 steps of one token a sequence the recurrence, norm and gate are one kernel, and in bfloat16
+steps of many tokens the recurrence runs in chunks of 64 tokens whose inner work is matrix products, with norm and gate in
+its last kernel; short portions and 32-bit runs go token by token (in a 32-bit run a token's sums have the same order
+however a prompt is cut).
 """
 
 from __future__ import annotations
@@ -86,10 +87,10 @@ class MatrixMemory(Mixer):
         at = F.MemoryColumns(q=0, k=H * d, v=2 * H * d, g=2 * H * d + H * dv, i=2 * H * d + 2 * H * dv, f=2 * H * d + 2 * H * dv + H)
         core = (proj, at, self.gate_bias, self.gate_cap, state, n_state)
         steps = (ctx.cu_q, ctx.slots, ctx.n_seqs)
-        if ctx.all_single and F.memory_single_fits(d, dv):
+        half = ctx.dtype == torch.bfloat16 and proj.dtype == torch.bfloat16
+        if half and ctx.all_single and F.memory_single_fits(d, dv):
             y = F.memory_single(*core, self.norm_w, self.norm_eps, *steps)
-        elif (ctx.dtype == torch.bfloat16 and proj.dtype == torch.bfloat16 and ctx.max_q_len >= self.chunked_from
-              and F.memory_chunked_fits(d, dv, at, proj.shape[1])):
+        elif half and ctx.max_q_len >= self.chunked_from and F.memory_chunked_fits(d, dv, at, proj.shape[1]):
             y = F.memory_chunked(*core, self.norm_w, self.norm_eps, *steps, ctx.max_q_len)
         else:  # few tokens a sequence, other sizes, and 32-bit runs (whose numbers do not depend on how a prompt is cut)
             o, den = F.memory_scan(*core, *steps)

@@ -159,7 +159,7 @@ def route(h: torch.Tensor, w: dict, p: str, r: dict, calls: list | None = None):
     seen = kept(h)  # the router may read the rounding that the experts read
     s = torch.softmax(seen @ w[p + "router"].T, -1)
     choice = s + w[p + "correction"]
-    spread = choice.std(-1)
+    spread = choice.std(-1, correction=0)
     margin = torch.full_like(spread, math.inf)
     groups = r.get("groups")
     if groups and groups["keep"] < groups["count"]:
