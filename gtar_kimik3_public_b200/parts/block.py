@@ -262,7 +262,8 @@ class GatedParallelBlock(Block):
             raise ValueError("a feed-forward comes with the norm before it, or not at all")
         self.width = int(width)
         self.norm_1, self.mixer, self.norm_2, self.feed_forward = norm_1, mixer, norm_2, feed_forward
-        self.names = {"mixer": "mix.", "feed_forward": "mlp.", "gate_1": "rg1", "gate_2": "rg2", **(names or {})}
+        self.names = {"mixer": "mix.", "feed_forward": "mlp.", "gate_1": "rg1", "gate_2": "rg2", "norm_2": "norm2",
+                      **(names or {})}
         self.next_block: GatedParallelBlock | None = None
         self.w_gates = self.bias_1 = self.bias_2 = None
 
@@ -282,6 +283,11 @@ class GatedParallelBlock(Block):
         for name in self._gate_names():
             specs[name] = TensorSpec((self.width, self.width))
             specs[name + ".b"] = TensorSpec((self.width,), "vector", init=(0.0, 0.5))
+        if self.feed_forward is None:  # a file may carry the absent branch's norm and gate all the same: nothing reads them
+            gate = self.names["gate_2"]
+            specs[self.names["norm_2"]] = TensorSpec((), "vector", optional=True)
+            specs[gate] = TensorSpec((self.width, self.width), optional=True)
+            specs[gate + ".b"] = TensorSpec((self.width,), "vector", optional=True)
         return specs
 
     def load(self, tensors):

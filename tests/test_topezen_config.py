@@ -26,7 +26,7 @@ def test_configurations_are_read_and_give_their_tensors(tag):
     raw = TPZ_CONFIGS[tag]
     W = raw["width"]
     model = _model(raw)
-    specs = {name: spec.shape for name, spec in model.tensor_specs().items()}
+    specs = {name: spec.shape for name, spec in model.tensor_specs().items() if not spec.optional}
     want = {"embed": (raw["vocab"], W), "head": (raw["vocab"], W), "final.norm": ()}
     for i, layer in enumerate(raw["layers"]):
         m, mlp = layer["mixer"], layer["mlp"]
@@ -56,6 +56,20 @@ def test_configurations_are_read_and_give_their_tensors(tag):
             want.update({p + "router": (mlp["router"]["experts"], W), p + "correction": (mlp["router"]["experts"],)})
     assert specs == want
     assert model.graph_safe()
+
+
+def test_a_layer_without_feed_forward_may_carry_the_absent_branchs_tensors(tmp_path):
+    """A file whose layer has no feed-forward loads with and without the second norm and gate; other names are refused."""
+    from gtar_kimik3_public_b200.weights.loader import WeightsError, check_tensors
+
+    specs = _model(TPZ_D).tensor_specs()
+    have = {name: tuple(spec.shape) for name, spec in specs.items() if not spec.optional}
+    assert "l0.rg2" not in have and "l1.rg2" in have
+    check_tensors(tmp_path, specs, have, {})
+    check_tensors(tmp_path, specs, {**have, "l0.norm2": (), "l0.rg2": (42, 42), "l0.rg2.b": (42,)}, {})
+    for extra in ("l0.norm3", "l0.mlp.up", "l1.mlp.shared.up"):
+        with pytest.raises(WeightsError):
+            check_tensors(tmp_path, specs, {**have, extra: (4,)}, {})
 
 
 def test_cache_requests():
