@@ -250,7 +250,7 @@ class Memory:
 MEMORIES = [
     # H, d, dv, lengths, cap, size of the gates' numbers
     (2, 16, 16, [5, 1, 33], 5.0, 1.0),
-    (3, 48, 80, [70, 17], 12.0, 4.0),
+    (3, 48, 80, [70, 17], 11.0, 4.0),
     (1, 128, 144, [130], 15.0, 2.0),
     (3, 10, 7, [40, 2], 3.0, 2.0),       # no multiple of 4
     (2, 20, 12, [65], 8.0, 8.0),         # gates that open and shut from token to token
@@ -287,7 +287,7 @@ def test_memory_token_by_token_whole_and_in_portions(dtype, H, d, dv, lengths, c
 
 
 @pytest.mark.parametrize("H,d,dv,lengths,cap,gate_size", [
-    (2, 16, 16, [64], 5.0, 1.0), (3, 48, 64, [300, 64, 1, 65], 12.0, 4.0), (2, 128, 128, [200, 129], 15.0, 1.0), (1, 64, 256, [128, 63], 15.0, 8.0),
+    (2, 16, 16, [64], 5.0, 1.0), (3, 48, 96, [300, 64, 1, 65], 11.0, 4.0), (2, 128, 128, [200, 129], 15.0, 1.0), (1, 64, 256, [128, 63], 15.0, 8.0),
     (1, 256, 512, [190], 15.0, 2.0), (2, 32, 80, [191, 2], 3.0, 2.0), (1, 16, 272, [100], 1.0, 3.0), (4, 80, 48, [65, 127, 128], 20.0, 12.0)])
 def test_memory_in_chunks(H, d, dv, lengths, cap, gate_size):
     """Chunks of 64 tokens against the plain read-outs and, closer than bfloat16 can show, against the states that the
@@ -321,7 +321,7 @@ def test_memory_in_waves_of_chunks(monkeypatch):
     assert torch.equal(whole, waves) and torch.equal(one[0], two[0]) and torch.equal(one[1], two[1])
 
 
-@pytest.mark.parametrize("H,d,dv,lengths,cap,gate_size", [(2, 16, 16, [9, 4, 1], 5.0, 1.0), (3, 48, 64, [40, 17], 12.0, 4.0), (2, 128, 144, [20, 30], 15.0, 2.0),
+@pytest.mark.parametrize("H,d,dv,lengths,cap,gate_size", [(2, 16, 16, [9, 4, 1], 5.0, 1.0), (3, 48, 96, [40, 17], 11.0, 4.0), (2, 128, 144, [20, 30], 15.0, 2.0),
                                                           (1, 256, 512, [6], 15.0, 2.0), (2, 20, 12, [40], 3.0, 8.0), (1, 300, 320, [5, 2], 4.0, 1.0)])
 def test_memory_single_tokens(H, d, dv, lengths, cap, gate_size):
     """One token of every sequence a step, the shorter ones leaving: read-outs and states as token by token."""

@@ -87,7 +87,7 @@ TPZ_D = model(120, 42, 1e-4, 6.3, [
 ])
 
 # one mixer alone and nothing else, with the layer's gates and norms
-TPZ_MEMORY = model(97, 48, 1e-6, 2.0, [layer(memory(2, 48, 64, 5.0), None)])
+TPZ_MEMORY = model(97, 48, 1e-6, 2.0, [layer(memory(2, 48, 32, 5.0), None)])
 TPZ_LATENT = model(101, 56, 1e-6, 1.0, [layer(latent(3, 24, 16, 24, 32, 64, 0.3, 300.0), None)])
 TPZ_SCORED = model(89, 40, 1e-6, 4.0, [layer(scored(4, 1, 64, 64, 0.3, softcap=6.0, window=33, keep=5), None)])
 
