@@ -75,7 +75,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_scored_kernel(
     const int* __restrict__ block_table, int n_tokens, int n_q, int n_kv, int d, int dv, int max_pages, int page_size,
     float scale, int window, int keep_first, const float* __restrict__ r1, const float* __restrict__ r2,
     const float* __restrict__ head_bias, int chunk, const float* __restrict__ temp, const float* __restrict__ dist_bias,
-    int n_dist, const float* __restrict__ sink, float softcap) {
+    int n_dist, const float* __restrict__ sink, float softcap, long long ld_out, float out_scale) {
     extern __shared__ float q_smem[];  // WARPS * d
     pdl_launch_dependents();
     pdl_wait();
@@ -150,28 +150,30 @@ __global__ void __launch_bounds__(WARPS * 32) attention_scored_kernel(
             }
         }
     }
-    T* orow = out + ((size_t)t * n_q + hq) * dv;
-    const float inv = SIGMOID ? 1.f : 1.f / l;
+    T* orow = out + (size_t)t * ld_out + (size_t)hq * dv;
+    const float inv = SIGMOID ? out_scale : out_scale / l;
 #pragma unroll
     for (int c = 0; c < MAX_ACC; ++c) {
         const int dim = lane + 32 * c;
-        if (c < n_acc && dim < dv) orow[dim] = from_float<T>(SIGMOID ? acc[c] : acc[c] * inv);
+        if (c < n_acc && dim < dv) orow[dim] = from_float<T>(acc[c] * inv);
     }
 }
 
 }  // namespace
 
 // weights: 0 softmax, 1 sigmoid.  r1, r2 (per query head, both or neither) and head_bias (per query head) may be null.
+// A token's read-outs, times out_scale, are the first n_q * dv entries of its row of `out`, rows ld_out apart.
 GK_EXPORT int gk_attention_scored_exact(const void* q, const void* k_pages, const void* v_pages, void* out, int dtype,
                                         const int* tok_pos, const int* tok_seq, const int* slots, const int* block_table,
                                         int n_tokens, int n_q, int n_kv, int d, int dv, int max_pages, int page_size, float scale,
                                         int window, int keep_first, const float* r1, const float* r2, const float* head_bias,
                                         int weights, int chunk, const float* temp, const float* dist_bias, int n_dist,
-                                        const float* sink, float softcap, void* stream) {
+                                        const float* sink, float softcap, long long ld_out, float out_scale, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(dtype), "attention_scored: bad dtype %d", dtype);
     GK_REQUIRE(n_tokens >= 0 && n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_scored: bad head counts %d/%d", n_q, n_kv);
     GK_REQUIRE(d > 0 && dv > 0 && dv <= 32 * MAX_ACC, "attention_scored: keys of %d must be positive, values of %d at most %d", d, dv,
                32 * MAX_ACC);
+    GK_REQUIRE(ld_out >= (long long)n_q * dv, "attention_scored: output rows of %lld for %d heads of %d", ld_out, n_q, dv);
     GK_REQUIRE(page_size > 0 && page_size % 32 == 0, "attention_scored: page_size %d must be a multiple of 32", page_size);
     GK_REQUIRE(window >= 0 && keep_first >= 0, "attention_scored: window and kept first keys must be >= 0 (0 = none)");
     GK_REQUIRE((r1 == nullptr) == (r2 == nullptr), "attention_scored: the distance term needs both of its numbers");
@@ -189,11 +191,11 @@ GK_EXPORT int gk_attention_scored_exact(const void* q, const void* k_pages, cons
         if (weights == 1)
             gk_launch(attention_scored_kernel<T, true>, dim3((unsigned)blocks), dim3(WARPS * 32), smem, s, (const T*)q, (const T*)k_pages,
                       (const T*)v_pages, (T*)out, tok_pos, tok_seq, slots, block_table, n_tokens, n_q, n_kv, d, dv, max_pages, page_size,
-                      scale, window, keep_first, r1, r2, head_bias, chunk, temp, dist_bias, n_dist, sink, softcap);
+                      scale, window, keep_first, r1, r2, head_bias, chunk, temp, dist_bias, n_dist, sink, softcap, ld_out, out_scale);
         else
             gk_launch(attention_scored_kernel<T, false>, dim3((unsigned)blocks), dim3(WARPS * 32), smem, s, (const T*)q, (const T*)k_pages,
                       (const T*)v_pages, (T*)out, tok_pos, tok_seq, slots, block_table, n_tokens, n_q, n_kv, d, dv, max_pages, page_size,
-                      scale, window, keep_first, r1, r2, head_bias, chunk, temp, dist_bias, n_dist, sink, softcap);
+                      scale, window, keep_first, r1, r2, head_bias, chunk, temp, dist_bias, n_dist, sink, softcap, ld_out, out_scale);
     })
     GK_CHECK_LAUNCH("attention_scored");
     return GK_OK;

@@ -1,5 +1,7 @@
-// Scored attention on the tensor cores (bfloat16, keys and values of 64 or 128 entries): the same rules as the exact
-// kernel of this family, for the new tokens of every sequence of a step over the paged cache.
+// Scored attention on the tensor cores (bfloat16): the same rules as the exact kernel of this family, for the new tokens of
+// every sequence of a step over the paged cache.  Keys and values of 64 or of 128 entries both have kernels of their own;
+// other sizes that are multiples of 8, keys of up to 128 and values of up to 256 entries, are padded with zeros in shared
+// memory to the next of 64, 128 (keys) and 64, 128, 256 (values), the cache's rows keeping their own length.
 //
 //   visible:  j <= i  and  (window = 0  or  i - j < window  or  j < keep_first)
 //   s_j = (q . k_j) * scale - r1_h * ln(1 + r2_h * (i - j))          (the second term only where r1, r2 are given)
@@ -30,14 +32,32 @@ using namespace attn;
 
 constexpr int SC_WARPS = 4;
 constexpr int SC_ROWS = SC_WARPS * 16;
-constexpr int SC_STAGES = 3;
 constexpr float LOG2E = 1.4426950408889634f;
 
-template <int D>
+template <int DV>
+constexpr int STAGES = DV > 128 ? 2 : 3;  // values of 256: two blocks a multiprocessor instead of a third stage
+
+template <int D, int DV>
 struct ScoredSmem {
-    __nv_bfloat16 k[SC_STAGES][PAGE * D];
-    __nv_bfloat16 v[SC_STAGES][PAGE * D];
+    __nv_bfloat16 k[STAGES<DV>][PAGE * D];
+    __nv_bfloat16 v[STAGES<DV>][PAGE * DV];
 };
+
+// A page whose rows have `d` entries (a multiple of 8, at most D) into a swizzled tile with rows of D: the entries from d on
+// and the rows from valid_rows on become zero.
+template <int D, int N_THREADS>
+__device__ __forceinline__ void load_page_padded(__nv_bfloat16* tile, const __nv_bfloat16* src, int d, int valid_rows, int tid) {
+    constexpr int CHUNKS = D / 8, ROWS_A_PASS = N_THREADS / CHUNKS;
+    const int row0 = tid / CHUNKS, chunk = tid % CHUNKS;
+    const bool in = chunk * 8 < d;
+    const __nv_bfloat16* g = src + (size_t)row0 * d + chunk * 8;
+#pragma unroll
+    for (int i = 0; i < PAGE / ROWS_A_PASS; ++i) {
+        const int row = row0 + i * ROWS_A_PASS;
+        const bool valid = in && row < valid_rows;
+        cp_async_16(reinterpret_cast<uint4*>(tile) + swz<D>(row, chunk), valid ? g + (size_t)i * ROWS_A_PASS * d : src, valid);
+    }
+}
 
 __device__ __forceinline__ float lg2_fast(float x) {
     float y;
@@ -55,17 +75,21 @@ __device__ __forceinline__ float soft_limit2(float t2, float two_by_cap, float c
 // CAP: the cap on the scores is compiled in.  MORE: which of the further rules are: 0 none, 1 the sink alone, 2 the chunk,
 // the head temperature, the distance table and the sink.  Without them the kernel is the windowed one alone and keeps its registers (a third block
 // a multiprocessor at heads of 64); the sink alone costs none.
-template <int D, bool SIGMOID, int MORE, bool CAP>
-__global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0) attention_scored_mma_kernel(
+// PADDED: the rows' lengths d <= D and dv <= DV are the arguments; else they are D and DV.
+template <int D, int DV, bool PADDED, bool SIGMOID, int MORE, bool CAP>
+__global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64 && !PADDED) ? 3 : 0) attention_scored_mma_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages, const __nv_bfloat16* __restrict__ v_pages,
     __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ cu_q,
     const int* __restrict__ kv_len, const int* __restrict__ slots, const int* __restrict__ block_table, int n_tokens, int n_q,
     int n_kv, int max_pages, float sl2, int window, int keep_first, const float* __restrict__ r1, const float* __restrict__ r2,
     const float* __restrict__ head_bias, int n_split, int chunk, const float* __restrict__ temp,
-    const float* __restrict__ dist_bias, int n_dist, const float* __restrict__ sink, float two_by_cap, float cap2) {
+    const float* __restrict__ dist_bias, int n_dist, const float* __restrict__ sink, float two_by_cap, float cap2, int d_arg,
+    int dv_arg, long long ld_out, float out_scale) {
     constexpr bool RULES = MORE == 2;
+    constexpr int SC_STAGES = STAGES<DV>;
+    const int d = PADDED ? d_arg : D, dv = PADDED ? dv_arg : DV;
     extern __shared__ __align__(128) unsigned char smem_raw[];
-    ScoredSmem<D>& sm = *reinterpret_cast<ScoredSmem<D>*>(smem_raw);
+    ScoredSmem<D, DV>& sm = *reinterpret_cast<ScoredSmem<D, DV>*>(smem_raw);
     pdl_launch_dependents();
     pdl_wait();
     const int seq = blockIdx.z, hk = blockIdx.y;
@@ -104,11 +128,11 @@ __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0)
         const int c0 = (lane & 3) * 2;
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-            const __nv_bfloat16* qrow = q + ((size_t)(q_begin + tok[h]) * n_q + head[h]) * D;
+            const __nv_bfloat16* qrow = q + ((size_t)(q_begin + tok[h]) * n_q + head[h]) * d;
 #pragma unroll
             for (int ks = 0; ks < D / 16; ++ks) {
-                qf[ks][h] = row_ok[h] ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + c0) : 0u;
-                qf[ks][h + 2] = row_ok[h] ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + c0 + 8) : 0u;
+                qf[ks][h] = row_ok[h] && (!PADDED || ks * 16 < d) ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + c0) : 0u;
+                qf[ks][h + 2] = row_ok[h] && (!PADDED || ks * 16 + 8 < d) ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + c0 + 8) : 0u;
             }
         }
     }
@@ -140,10 +164,15 @@ __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0)
             const int p = page_index(it);
             const int page = pages[p];
             const int valid = min(PAGE, len - p * PAGE);
-            const size_t base = ((size_t)page * n_kv + hk) * PAGE * D;
+            const size_t base = ((size_t)page * n_kv + hk) * PAGE;
             const int stage = (it - it0) % SC_STAGES;
-            load_page_async<D, SC_WARPS * 32>(sm.k[stage], k_pages + base, valid, tid);
-            load_page_async<D, SC_WARPS * 32>(sm.v[stage], v_pages + base, valid, tid);
+            if constexpr (PADDED) {
+                load_page_padded<D, SC_WARPS * 32>(sm.k[stage], k_pages + base * d, d, valid, tid);
+                load_page_padded<DV, SC_WARPS * 32>(sm.v[stage], v_pages + base * dv, dv, valid, tid);
+            } else {
+                load_page_async<D, SC_WARPS * 32>(sm.k[stage], k_pages + base * D, valid, tid);
+                load_page_async<DV, SC_WARPS * 32>(sm.v[stage], v_pages + base * DV, valid, tid);
+            }
         }
         cp_async_commit();
     };
@@ -157,9 +186,9 @@ __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0)
             l[h] = 1.f;
         }
     }
-    float o[D / 8][4];
+    float o[DV / 8][4];
 #pragma unroll
-    for (int j = 0; j < D / 8; ++j)
+    for (int j = 0; j < DV / 8; ++j)
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
 
@@ -206,9 +235,9 @@ __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0)
                     p[g][3] = pack_bf16(s[2 * g + 1][2], s[2 * g + 1][3]);
                 }
             } else {
-                softmax_page<D>(s, m, l, o, p, 1.0f);
+                softmax_page<DV>(s, m, l, o, p, 1.0f);
             }
-            pv_page<D, false>(o, p, sm.v[stage], n16, lane);
+            pv_page<DV, false>(o, p, sm.v[stage], n16, lane);
         }
     }
     cp_async_wait<0>();
@@ -218,11 +247,11 @@ __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0)
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
             if (!row_ok[h]) continue;
-            const float inv = SIGMOID ? 1.f : 1.0f / l[h];
-            __nv_bfloat16* orow = out + ((size_t)(q_begin + tok[h]) * n_q + head[h]) * D;
+            const float inv = SIGMOID ? out_scale : out_scale / l[h];
+            __nv_bfloat16* orow = out + (size_t)(q_begin + tok[h]) * ld_out + (size_t)head[h] * dv;
 #pragma unroll
-            for (int j = 0; j < D / 8; ++j)
-                *reinterpret_cast<uint32_t*>(orow + j * 8 + c0) = pack_bf16(o[j][2 * h] * inv, o[j][2 * h + 1] * inv);
+            for (int j = 0; j < DV / 8; ++j)
+                if (!PADDED || j * 8 < dv) *reinterpret_cast<uint32_t*>(orow + j * 8 + c0) = pack_bf16(o[j][2 * h] * inv, o[j][2 * h + 1] * inv);
         }
         return;
     }
@@ -230,17 +259,19 @@ __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64) ? 3 : 0)
     for (int h = 0; h < 2; ++h) {
         if (!row_ok[h]) continue;
         const size_t item = ((size_t)split * n_tokens + q_begin + tok[h]) * n_q + head[h];
-        float* orow = part_o + item * D;
+        float* orow = part_o + item * dv;
 #pragma unroll
-        for (int j = 0; j < D / 8; ++j) *reinterpret_cast<float2*>(orow + j * 8 + c0) = make_float2(o[j][2 * h], o[j][2 * h + 1]);
+        for (int j = 0; j < DV / 8; ++j)
+            if (!PADDED || j * 8 < dv) *reinterpret_cast<float2*>(orow + j * 8 + c0) = make_float2(o[j][2 * h], o[j][2 * h + 1]);
         if (!SIGMOID && (lane & 3) == 0) *reinterpret_cast<float2*>(part_ml + item * 2) = make_float2(m[h], l[h]);
     }
 }
 
 // One warp per (token, query head): the parts' sums brought to one maximum and added.
-template <int D, bool SIGMOID>
+template <int DV, bool SIGMOID>
 __global__ void __launch_bounds__(128) attention_scored_join_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                                                    __nv_bfloat16* __restrict__ out, long long n_items, int n_split) {
+                                                                    __nv_bfloat16* __restrict__ out, long long n_items, int n_split,
+                                                                    int n_q, int dv, long long ld_out, float out_scale) {
     pdl_launch_dependents();
     pdl_wait();
     const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -249,9 +280,9 @@ __global__ void __launch_bounds__(128) attention_scored_join_kernel(const float*
     float top = -INFINITY;
     if (!SIGMOID)
         for (int s = 0; s < n_split; ++s) top = fmaxf(top, part_ml[((size_t)s * n_items + item) * 2]);
-    float acc[D / 32], denom = 0.f;
+    float acc[DV / 32], denom = 0.f;
 #pragma unroll
-    for (int c = 0; c < D / 32; ++c) acc[c] = 0.f;
+    for (int c = 0; c < DV / 32; ++c) acc[c] = 0.f;
     for (int s = 0; s < n_split; ++s) {
         float w = 1.f;
         if (!SIGMOID) {
@@ -259,40 +290,44 @@ __global__ void __launch_bounds__(128) attention_scored_join_kernel(const float*
             w = ml.x == -INFINITY ? 0.f : exp2_fast(ml.x - top);
             denom = fmaf(ml.y, w, denom);
         }
-        const float* src = part_o + ((size_t)s * n_items + item) * D;
+        const float* src = part_o + ((size_t)s * n_items + item) * dv;
 #pragma unroll
-        for (int c = 0; c < D / 32; ++c) acc[c] = fmaf(src[lane + 32 * c], w, acc[c]);
+        for (int c = 0; c < DV / 32; ++c)
+            if (lane + 32 * c < dv) acc[c] = fmaf(src[lane + 32 * c], w, acc[c]);
     }
-    const float inv = SIGMOID ? 1.f : 1.f / denom;
+    const float inv = SIGMOID ? out_scale : out_scale / denom;
+    __nv_bfloat16* orow = out + (size_t)(item / n_q) * ld_out + (size_t)(item % n_q) * dv;
 #pragma unroll
-    for (int c = 0; c < D / 32; ++c) out[(size_t)item * D + lane + 32 * c] = __float2bfloat16(acc[c] * inv);
+    for (int c = 0; c < DV / 32; ++c)
+        if (lane + 32 * c < dv) orow[lane + 32 * c] = __float2bfloat16(acc[c] * inv);
 }
 
-template <int D, bool SIGMOID, int MORE, bool CAP>
+template <int D, int DV, bool PADDED, bool SIGMOID, int MORE, bool CAP>
 int launch_scored(const void* q, const void* k_pages, const void* v_pages, void* out, float* part_o, float* part_ml, const int* cu_q,
                   const int* kv_len, const int* slots, const int* block_table, int n_seqs, int max_q_len, int n_tokens, int n_q,
                   int n_kv, int max_pages, float scale, int window, int keep_first, const float* r1, const float* r2,
                   const float* head_bias, int n_split, int chunk, const float* temp, const float* dist_bias, int n_dist,
-                  const float* sink, float softcap, cudaStream_t stream) {
-    const size_t smem = sizeof(ScoredSmem<D>);
+                  const float* sink, float softcap, int d, int dv, long long ld_out, float out_scale, cudaStream_t stream) {
+    const size_t smem = sizeof(ScoredSmem<D, DV>);
     static bool configured = false;
     if (!configured) {
-        cudaError_t err = cudaFuncSetAttribute(attention_scored_mma_kernel<D, SIGMOID, MORE, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t err = cudaFuncSetAttribute(attention_scored_mma_kernel<D, DV, PADDED, SIGMOID, MORE, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (err != cudaSuccess) return gk_fail(GK_CUDA_ERROR, "attention_scored_mma: %s", cudaGetErrorString(err));
         configured = true;
     }
     const int group = n_q / n_kv;
     const long long blocks = (((long long)max_q_len * group + SC_ROWS - 1) / SC_ROWS) * n_split;
     GK_REQUIRE(blocks <= 2147483647LL, "attention_scored_mma: too many rows");
-    gk_launch(attention_scored_mma_kernel<D, SIGMOID, MORE, CAP>, dim3((unsigned)blocks, n_kv, n_seqs), dim3(SC_WARPS * 32), smem, stream,
+    gk_launch(attention_scored_mma_kernel<D, DV, PADDED, SIGMOID, MORE, CAP>, dim3((unsigned)blocks, n_kv, n_seqs), dim3(SC_WARPS * 32), smem, stream,
               (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, (__nv_bfloat16*)out, part_o, part_ml,
               cu_q, kv_len, slots, block_table, n_tokens, n_q, n_kv, max_pages, scale * LOG2E, window, keep_first, r1, r2, head_bias,
-              n_split, chunk, temp, dist_bias, n_dist, sink, CAP ? 2.f / softcap : 0.f, softcap * LOG2E);
+              n_split, chunk, temp, dist_bias, n_dist, sink, CAP ? 2.f / softcap : 0.f, softcap * LOG2E, d, dv, ld_out,
+              out_scale);
     GK_CHECK_LAUNCH("attention_scored_mma");
     if (n_split > 1) {
         const long long items = (long long)n_tokens * n_q;
-        gk_launch(attention_scored_join_kernel<D, SIGMOID>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, (const float*)part_o,
-                  (const float*)part_ml, (__nv_bfloat16*)out, items, n_split);
+        gk_launch(attention_scored_join_kernel<DV, SIGMOID>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, (const float*)part_o,
+                  (const float*)part_ml, (__nv_bfloat16*)out, items, n_split, n_q, dv, ld_out, out_scale);
         GK_CHECK_LAUNCH("attention_scored_join");
     }
     return GK_OK;
@@ -300,19 +335,25 @@ int launch_scored(const void* q, const void* k_pages, const void* v_pages, void*
 
 }  // namespace
 
-// q, out: [n_tokens, n_q, head_dim] bfloat16 packed by sequence (cu_q[i] = first token of sequence i); kv_len[i] counts
+// q: [n_tokens, n_q, d] bfloat16 packed by sequence (cu_q[i] = first token of sequence i); a token's read-outs, times
+// out_scale, are the first n_q * dv entries of its row of `out`, rows ld_out apart; kv_len[i] counts
 // the sequence's cached tokens including this step's; max_q_len = the longest part of the step.  weights: 0 softmax,
 // 1 sigmoid.  r1, r2 (both or neither) and head_bias, a number per query head, may be null.  With n_split > 1,
-// part_o [n_split, n_tokens, n_q, head_dim] and (softmax) part_ml [n_split, n_tokens, n_q, 2] are 32-bit workspaces.
+// part_o [n_split, n_tokens, n_q, dv] and (softmax) part_ml [n_split, n_tokens, n_q, 2] are 32-bit workspaces.
 GK_EXPORT int gk_attention_scored_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, float* part_o,
                                        float* part_ml, const int* cu_q, const int* kv_len, const int* slots, const int* block_table,
-                                       int n_seqs, int max_q_len, int n_tokens, int n_q, int n_kv, int head_dim, int max_pages,
+                                       int n_seqs, int max_q_len, int n_tokens, int n_q, int n_kv, int d, int dv, int max_pages,
                                        int page_size, float scale, int window, int keep_first, const float* r1, const float* r2,
                                        const float* head_bias, int weights, int n_split, int chunk, const float* temp,
-                                       const float* dist_bias, int n_dist, const float* sink, float softcap, void* stream) {
+                                       const float* dist_bias, int n_dist, const float* sink, float softcap, long long ld_out,
+                                       float out_scale, void* stream) {
     GK_REQUIRE(n_seqs >= 0 && n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_scored_mma: bad head counts %d/%d", n_q, n_kv);
     GK_REQUIRE(page_size == attn::PAGE, "attention_scored_mma: page_size must be %d, got %d", attn::PAGE, page_size);
-    GK_REQUIRE(head_dim == 64 || head_dim == 128, "attention_scored_mma: head size %d is not 64 or 128 (use the exact kernel)", head_dim);
+    const bool own_size = d == dv && (d == 64 || d == 128);
+    GK_REQUIRE(own_size || (d > 0 && d <= 128 && d % 8 == 0 && dv > 0 && dv <= 256 && dv % 8 == 0 && softcap == 0.f),
+               "attention_scored_mma: keys of %d and values of %d are no multiples of 8 up to 128 and 256, or a cap comes with sizes other "
+               "than 64 and 128 (use the exact kernel)", d, dv);
+    GK_REQUIRE(ld_out >= (long long)n_q * dv && ld_out % 2 == 0 && ((uintptr_t)out & 3) == 0, "attention_scored_mma: bad output rows");
     GK_REQUIRE(n_kv <= 65535 && n_seqs <= 65535, "attention_scored_mma: grid too large");
     GK_REQUIRE(window >= 0 && keep_first >= 0 && max_q_len >= 0, "attention_scored_mma: bad window, kept keys or length");
     GK_REQUIRE((r1 == nullptr) == (r2 == nullptr), "attention_scored_mma: the distance term needs both of its numbers");
@@ -325,31 +366,44 @@ GK_EXPORT int gk_attention_scored_bf16(const void* q, const void* k_pages, const
     if (n_seqs == 0 || max_q_len == 0 || n_tokens == 0) return GK_OK;
     cudaStream_t s = (cudaStream_t)stream;
     const int more = (chunk > 0 || temp != nullptr || dist_bias != nullptr) ? 2 : sink != nullptr ? 1 : 0;
-#define GK_SCORED_AS(D, SIG, MORE, CAP)                                                                                              \
-    return launch_scored<D, SIG, MORE, CAP>(q, k_pages, v_pages, out, part_o, part_ml, cu_q, kv_len, slots, block_table, n_seqs,     \
-                                            max_q_len, n_tokens, n_q, n_kv, max_pages, scale, window, keep_first, r1, r2, head_bias, \
-                                            n_split, chunk, temp, dist_bias, n_dist, sink, softcap, s)
-#define GK_SCORED(D, SIG)                              \
-    do {                                               \
-        if (more == 2) GK_SCORED_AS(D, SIG, 2, false); \
-        if (more == 1) GK_SCORED_AS(D, SIG, 1, false); \
-        GK_SCORED_AS(D, SIG, 0, false);                \
+#define GK_SCORED_AS(D, DV, PADDED, SIG, MORE, CAP)                                                                                    \
+    return launch_scored<D, DV, PADDED, SIG, MORE, CAP>(q, k_pages, v_pages, out, part_o, part_ml, cu_q, kv_len, slots, block_table, \
+                                                        n_seqs, max_q_len, n_tokens, n_q, n_kv, max_pages, scale, window, keep_first, \
+                                                        r1, r2, head_bias, n_split, chunk, temp, dist_bias, n_dist, sink, softcap, d, \
+                                                        dv, ld_out, out_scale, s)
+#define GK_SCORED(D, SIG)                                        \
+    do {                                                         \
+        if (more == 2) GK_SCORED_AS(D, D, false, SIG, 2, false); \
+        if (more == 1) GK_SCORED_AS(D, D, false, SIG, 1, false); \
+        GK_SCORED_AS(D, D, false, SIG, 0, false);                \
     } while (0)
-#define GK_CAPPED(D)                                    \
-    do {                                                \
-        if (more == 2) GK_SCORED_AS(D, false, 2, true); \
-        GK_SCORED_AS(D, false, 1, true);                \
+#define GK_CAPPED(D)                                              \
+    do {                                                          \
+        if (more == 2) GK_SCORED_AS(D, D, false, false, 2, true); \
+        GK_SCORED_AS(D, D, false, false, 1, true);                \
     } while (0)
+#define GK_PADDED(D, DV)                                              \
+    do {                                                              \
+        if (weights == 1) GK_SCORED_AS(D, DV, true, true, 2, false);  \
+        GK_SCORED_AS(D, DV, true, false, 2, false);                   \
+    } while (0)
+    if (!own_size) {  // the kernel with all rules
+        if (d <= 64 && dv <= 64) GK_PADDED(64, 64);
+        if (d <= 64 && dv <= 128) GK_PADDED(64, 128);
+        if (dv <= 128) GK_PADDED(128, 128);
+        GK_PADDED(128, 256);
+    }
     if (softcap > 0.f) {
-        if (head_dim == 64) GK_CAPPED(64);
+        if (d == 64) GK_CAPPED(64);
         GK_CAPPED(128);
     }
-    if (head_dim == 64) {
+    if (d == 64) {
         if (weights == 1) GK_SCORED(64, true);
         GK_SCORED(64, false);
     }
     if (weights == 1) GK_SCORED(128, true);
     GK_SCORED(128, false);
+#undef GK_PADDED
 #undef GK_CAPPED
 #undef GK_SCORED
 #undef GK_SCORED_AS

@@ -1,5 +1,6 @@
 // The gated delta rule with a decay per head and key channel, as a recurrent mixer: what stands between its
-// input projections and its output projection.
+// input projections and its output projection.  (The recurrence also takes one decay per head; what else that form needs
+// is in delta_head.cu.)
 //
 // Per sequence and head, with a state S [d, dv] of 32-bit floats that starts at zero:
 //     S <- diag(g_t) S ;  u_t = beta_t (v_t - S^T k_t) ;  S <- S + k_t u_t^T ;  o_t = S^T q_t
@@ -149,14 +150,15 @@ __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_gr
 // at lane * PIECE floats, padded so that the 16-byte loads of the lanes fall into different banks.  A token's step is
 // one chain of dependent instructions of a warp (it showed as 209 instructions a token at three cycles each with eight
 // lanes a column and sixteen rows a lane): more lanes a column shorten the chain and lengthen the exchange.
-template <int R, int TB, int LPC>
+// HEAD: one decay per token and head (g [T, H]) instead of one per key channel (g [T, H, d]).
+template <int R, int TB, int LPC, bool HEAD>
 __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
     const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, const float* __restrict__ g,
     const float* __restrict__ beta, float* __restrict__ state /* [slots, H, d, dv] */, float* __restrict__ out /* [T, H, dv] */,
     const int* __restrict__ cu_q, const int* __restrict__ slots, int n_heads, int n_kv, int d, int dv) {
     constexpr int PIECE = R == 4 ? 4 : R + 4, VEC = LPC * PIECE;
-    __shared__ __align__(16) float sq[2][TB][VEC], sk[2][TB][VEC], sg[2][TB][VEC];
-    __shared__ __align__(16) float sv[2][TB][SCAN_COLS], sb[2][TB];
+    __shared__ __align__(16) float sq[2][TB][VEC], sk[2][TB][VEC], sg[2][HEAD ? 1 : TB][VEC];
+    __shared__ __align__(16) float sv[2][TB][SCAN_COLS], sb[2][TB], sh[2][TB];
     pdl_launch_dependents();
     const int n_threads = blockDim.x, n_cols = n_threads / LPC;  // columns of this block
     const int seq = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * n_cols;
@@ -167,7 +169,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
     for (int i = threadIdx.x; i < 2 * TB * VEC; i += n_threads) {
         (&sq[0][0][0])[i] = 0.f;
         (&sk[0][0][0])[i] = 0.f;
-        (&sg[0][0][0])[i] = 0.f;
+        if (!HEAD) (&sg[0][0][0])[i] = 0.f;
     }
     __syncthreads();
     pdl_wait();
@@ -182,7 +184,15 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
     const int quads = d / 4;  // 16-byte pieces of a vector of this head
     auto stage = [&](int buf, int first) {
         const int count = min(TB, n - first);
-        if (n_threads % quads == 0) {  // a thread's piece of a vector is the same for every token it copies
+        if (HEAD && (d & 3)) {  // rows that do not start on 16 bytes: one entry a copy
+            for (int i = threadIdx.x; i < count * d; i += n_threads) {
+                const int tt = i / d, c = i - tt * d;
+                const int at = (c / R) * PIECE + c % R;
+                const size_t tok = (size_t)(t0 + first + tt);
+                cp_async4(&sq[buf][tt][at], q + (tok * n_kv + hk) * d + c);
+                cp_async4(&sk[buf][tt][at], k + (tok * n_kv + hk) * d + c);
+            }
+        } else if (n_threads % quads == 0) {  // a thread's piece of a vector is the same for every token it copies
             const int c4 = (threadIdx.x % quads) * 4, step = n_threads / quads;
             const int at = (c4 / R) * PIECE + c4 % R;
             const float* pq_ = q + ((size_t)(t0 + first) * n_kv + hk) * d + c4;
@@ -191,7 +201,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
             for (int tt = threadIdx.x / quads; tt < count; tt += step) {
                 cp_async16(&sq[buf][tt][at], pq_ + (size_t)tt * n_kv * d);
                 cp_async16(&sk[buf][tt][at], pk_ + (size_t)tt * n_kv * d);
-                cp_async16(&sg[buf][tt][at], pg_ + (size_t)tt * n_heads * d);
+                if (!HEAD) cp_async16(&sg[buf][HEAD ? 0 : tt][at], pg_ + (size_t)tt * n_heads * d);
             }
         } else {
             for (int i = threadIdx.x; i < count * quads; i += n_threads) {
@@ -201,14 +211,17 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
                 const size_t tok = (size_t)(t0 + first + tt);
                 cp_async16(&sq[buf][tt][at], q + (tok * n_kv + hk) * d + c4);
                 cp_async16(&sk[buf][tt][at], k + (tok * n_kv + hk) * d + c4);
-                cp_async16(&sg[buf][tt][at], g + (tok * n_heads + head) * d + c4);
+                if (!HEAD) cp_async16(&sg[buf][HEAD ? 0 : tt][at], g + (tok * n_heads + head) * d + c4);
             }
         }
         for (int i = threadIdx.x; i < count * n_cols; i += n_threads) {
             const int tt = i / n_cols, cc = i - tt * n_cols;
             if (col0 + cc < dv) cp_async4(&sv[buf][tt][cc], v + ((size_t)(t0 + first + tt) * n_heads + head) * dv + col0 + cc);
         }
-        if (threadIdx.x < count) cp_async4(&sb[buf][threadIdx.x], beta + (size_t)(t0 + first + threadIdx.x) * n_heads + head);
+        for (int i = threadIdx.x; i < count; i += n_threads) {
+            cp_async4(&sb[buf][i], beta + (size_t)(t0 + first + i) * n_heads + head);
+            if (HEAD) cp_async4(&sh[buf][i], g + (size_t)(t0 + first + i) * n_heads + head);
+        }
         cp_async_commit();
     };
     stage(0, 0);
@@ -231,13 +244,14 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
         const float4* pg = reinterpret_cast<const float4*>(&sg[buf][0][sub * PIECE]);
         const size_t out_step = (size_t)n_heads * dv;
 #pragma unroll 2
-        for (int tt = 0; tt < count; ++tt, out_at += out_step, v_at += SCAN_COLS, ++b_at, pq += VEC / 4, pk += VEC / 4, pg += VEC / 4) {
+        for (int tt = 0; tt < count; ++tt, out_at += out_step, v_at += SCAN_COLS, ++b_at, pq += VEC / 4, pk += VEC / 4, pg += HEAD ? 0 : VEC / 4) {
             float kk[R], qq[R];
+            const float gh = HEAD ? sh[buf][tt] : 0.f;
             // four partial sums each (one per place in a group of four rows): chains of R / 4 dependent operations
             float a4[4] = {0.f, 0.f, 0.f, 0.f}, b4[4] = {0.f, 0.f, 0.f, 0.f}, c4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int r4 = 0; r4 < R / 4; ++r4) {
-                const float4 g4 = pg[r4], k4 = pk[r4], q4 = pq[r4];
+                const float4 g4 = HEAD ? make_float4(gh, gh, gh, gh) : pg[r4], k4 = pk[r4], q4 = pq[r4];
                 const float gs[4] = {g4.x, g4.y, g4.z, g4.w};
                 kk[4 * r4] = k4.x; kk[4 * r4 + 1] = k4.y; kk[4 * r4 + 2] = k4.z; kk[4 * r4 + 3] = k4.w;
                 qq[4 * r4] = q4.x; qq[4 * r4 + 1] = q4.y; qq[4 * r4 + 2] = q4.z; qq[4 * r4 + 3] = q4.w;
@@ -332,11 +346,13 @@ GK_EXPORT int gk_conv_roll(const void* proj, int dtype, long long ld, float* sta
     return GK_OK;
 }
 
+// head_decay: g is [T, H] (one decay per token and head) instead of [T, H, d].
 GK_EXPORT int gk_delta_scan(const float* q, const float* k, const float* v, const float* g, const float* beta, float* state,
                             float* out, const int* cu_q, const int* slots, int n_seqs, int n_heads, int n_kv, int d, int dv,
-                            int lanes, int force_cols, void* stream) {
+                            int lanes, int force_cols, int head_decay, void* stream) {
     GK_REQUIRE(n_heads > 0 && n_kv > 0 && n_heads % n_kv == 0, "delta_scan: bad head counts %d/%d", n_heads, n_kv);
-    GK_REQUIRE(d > 0 && d % 4 == 0 && d <= 256, "delta_scan: key size %d must be a multiple of 4, at most 256", d);
+    GK_REQUIRE(d > 0 && (head_decay ? d <= 512 : d % 4 == 0 && d <= 256),
+               "delta_scan: key size %d must be a multiple of 4, at most 256 (one decay per head: any size up to 512)", d);
     GK_REQUIRE(dv > 0 && n_seqs >= 0 && n_seqs <= 65535 && n_heads <= 65535, "delta_scan: bad sizes");
     if (n_seqs == 0) return GK_OK;
     // Few (sequence, head) pairs: fewer columns a block, so that the columns of a head spread over more SMs and a token's
@@ -356,13 +372,19 @@ GK_EXPORT int gk_delta_scan(const float* q, const float* k, const float* v, cons
     GK_REQUIRE(lanes == 8 || lanes == 16 || lanes == 32, "delta_scan: 8, 16 or 32 lanes a column, not %d", lanes);
     if (d <= 32) lanes = 8;
     else if (d <= 64 && lanes == 32) lanes = 16;
+    else if (d > 256) lanes = 16;
     int cols = SCAN_THREADS / lanes;
     while (cols > 2 && cols * lanes > 64 && (long long)n_seqs * n_heads * ((dv + cols - 1) / cols) < 2LL * sms) cols /= 2;
     if (force_cols > 0 && force_cols * lanes <= SCAN_THREADS && force_cols <= SCAN_COLS) cols = force_cols;
     const dim3 grid((dv + cols - 1) / cols, n_heads, n_seqs), block(cols * lanes);
     cudaStream_t s = (cudaStream_t)stream;
-#define GK_SCAN(R, TB, L)                                                                                                \
-    gk_launch(delta_scan_kernel<R, TB, L>, grid, block, 0, s, q, k, v, g, beta, state, out, cu_q, slots, n_heads, n_kv, d, dv)
+#define GK_SCAN(R, TB, L)                                                                                                              \
+    do {                                                                                                                               \
+        if (head_decay)                                                                                                                \
+            gk_launch(delta_scan_kernel<R, TB, L, true>, grid, block, 0, s, q, k, v, g, beta, state, out, cu_q, slots, n_heads, n_kv, d, dv); \
+        else                                                                                                                           \
+            gk_launch(delta_scan_kernel<R, TB, L, false>, grid, block, 0, s, q, k, v, g, beta, state, out, cu_q, slots, n_heads, n_kv, d, dv); \
+    } while (0)
     if (lanes == 8) {
         if (d <= 32) GK_SCAN(4, 16, 8);
         else if (d <= 64) GK_SCAN(8, 16, 8);
@@ -371,7 +393,9 @@ GK_EXPORT int gk_delta_scan(const float* q, const float* k, const float* v, cons
     } else if (lanes == 16) {
         if (d <= 64) GK_SCAN(4, 16, 16);
         else if (d <= 128) GK_SCAN(8, 8, 16);
-        else GK_SCAN(16, 4, 16);
+        else if (d <= 256) GK_SCAN(16, 4, 16);
+        else
+            gk_launch(delta_scan_kernel<32, 4, 16, true>, grid, block, 0, s, q, k, v, g, beta, state, out, cu_q, slots, n_heads, n_kv, d, dv);
     } else {
         if (d <= 128) GK_SCAN(4, 8, 32);
         else GK_SCAN(8, 4, 32);

@@ -1,13 +1,19 @@
-// Layer norm with a weight and no bias on the 32-bit residual stream, fused with the add of a branch output that
-// has not been added yet:
+// Layer norm with a weight and an optional bias on the 32-bit residual stream, fused with the add of a branch output
+// that has not been added yet:
 //
 //   h += delta_scale * delta            (in place; skipped when there is no delta)
-//   out = (h - mean(h)) / sqrt(mean((h - mean(h))^2) + eps) * w
+//   out = (h - mean(h)) / sqrt(mean((h - mean(h))^2) + eps) * w + b
 //
 // The variance is the mean of the squared deviations, formed in a second pass over the row (kept in shared
 // memory), not from the mean of squares.  With `rows` only those rows are normed and the stream is not written.
 // One block of a fixed size per row: the order of a row's sums depends on nothing but the row.  All arithmetic
 // is 32-bit; the branch output may be bfloat16, the result bfloat16 or float32.
+//
+// layernorm_merge is the same norm around a branch on both sides, with the adds that may stand between two layers:
+//
+//   v = x + LN(y; w_y, b_y)             (y added as it is where it comes without weights; left out where there is none)
+//   v = v + first + step                (each only where given: a row a token; one vector for all tokens)
+//   x_out = v ;  z = LN(v; w_z, b_z)    (the second only where a next norm is given)
 
 #include "common.cuh"
 
@@ -18,7 +24,7 @@ constexpr int LN_THREADS = 256;
 template <typename TD, typename TW, typename TO>
 __global__ void __launch_bounds__(LN_THREADS) add_layernorm_kernel(float* __restrict__ h, const TD* __restrict__ delta,
                                                                    float delta_scale, const TW* __restrict__ w,
-                                                                   TO* __restrict__ out, const int* __restrict__ rows,
+                                                                   const TW* __restrict__ bias, TO* __restrict__ out, const int* __restrict__ rows,
                                                                    int hidden, float eps) {
     extern __shared__ float row[];  // hidden floats
     __shared__ float scratch[33];
@@ -45,7 +51,163 @@ __global__ void __launch_bounds__(LN_THREADS) add_layernorm_kernel(float* __rest
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
     TO* orow = out + (size_t)blockIdx.x * hidden;
-    for (int i = threadIdx.x; i < hidden; i += LN_THREADS) orow[i] = from_float<TO>((row[i] - mean) * inv * to_float(w[i]));
+    for (int i = threadIdx.x; i < hidden; i += LN_THREADS) {
+        float v = (row[i] - mean) * inv * to_float(w[i]);
+        if (bias != nullptr) v += to_float(bias[i]);
+        orow[i] = from_float<TO>(v);
+    }
+}
+
+// The sum of a row over the block with one barrier: every thread adds the warps' parts in their order.  Each call of a
+// kernel has a `parts` of its own.
+__device__ __forceinline__ float row_sum(float v, float* parts) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) parts[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int i = 0; i < LN_THREADS / 32; ++i) total += parts[i];
+    return total;
+}
+
+template <typename T, int VEC>
+__device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4 && sizeof(T) == 4) {
+        const float4 a = *reinterpret_cast<const float4*>(p);
+        v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w;
+    } else if constexpr (VEC == 4) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        v[0] = lo.x, v[1] = lo.y, v[2] = hi.x, v[3] = hi.y;
+    } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = to_float(p[e]);
+    }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 4 && sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    } else if constexpr (VEC == 4) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        uint2 raw;
+        raw.x = *reinterpret_cast<uint32_t*>(&lo);
+        raw.y = *reinterpret_cast<uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(p) = raw;
+    } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) p[e] = from_float<T>(v[e]);
+    }
+}
+
+// A row a block, held in registers: N pieces of VEC neighbouring entries a thread.
+template <typename TY, typename TZ, int VEC, int N>
+__global__ void __launch_bounds__(LN_THREADS) layernorm_merge_kernel(
+    const float* x, const TY* __restrict__ y, const float* __restrict__ w_y, const float* __restrict__ b_y, float eps_y,
+    const float* first, const float* __restrict__ step, float* x_out, const float* __restrict__ w_z,
+    const float* __restrict__ b_z, float eps_z, TZ* __restrict__ z, int width) {
+    __shared__ float parts[4][LN_THREADS / 32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t at = (size_t)blockIdx.x * width;
+    float v[N][VEC];
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int i = (n * LN_THREADS + (int)threadIdx.x) * VEC;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[n][e] = 0.f;
+        if (i < width) load_vec<float, VEC>(x + at + i, v[n]);
+    }
+    if (y != nullptr) {
+        float b[N][VEC], sum = 0.f;
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+            const int i = (n * LN_THREADS + (int)threadIdx.x) * VEC;
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) b[n][e] = 0.f;
+            if (i < width) load_vec<TY, VEC>(y + at + i, b[n]);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) sum += b[n][e];
+        }
+        if (w_y != nullptr) {
+            const float mean = row_sum(sum, parts[0]) / (float)width;
+            float ss = 0.f;
+#pragma unroll
+            for (int n = 0; n < N; ++n) {
+                const int i = (n * LN_THREADS + (int)threadIdx.x) * VEC;
+                if (i < width)
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        b[n][e] -= mean;
+                        ss = fmaf(b[n][e], b[n][e], ss);
+                    }
+            }
+            const float inv = 1.0f / sqrtf(row_sum(ss, parts[1]) / (float)width + eps_y);
+#pragma unroll
+            for (int n = 0; n < N; ++n) {
+                const int i = (n * LN_THREADS + (int)threadIdx.x) * VEC;
+                if (i < width) {
+                    float w[VEC], bias[VEC];
+                    load_vec<float, VEC>(w_y + i, w);
+                    load_vec<float, VEC>(b_y + i, bias);
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) b[n][e] = fmaf(b[n][e] * inv, w[e], bias[e]);
+                }
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < N; ++n)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[n][e] += b[n][e];
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int i = (n * LN_THREADS + (int)threadIdx.x) * VEC;
+        if (i < width) {
+            float more[VEC];
+            if (first != nullptr) {
+                load_vec<float, VEC>(first + at + i, more);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[n][e] += more[e];
+            }
+            if (step != nullptr) {
+                load_vec<float, VEC>(step + i, more);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[n][e] += more[e];
+            }
+            store_vec<float, VEC>(x_out + at + i, v[n]);
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) sum += v[n][e];
+    }
+    if (z == nullptr) return;
+    const float mean = row_sum(sum, parts[2]) / (float)width;
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int i = (n * LN_THREADS + (int)threadIdx.x) * VEC;
+        if (i < width)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                v[n][e] -= mean;
+                ss = fmaf(v[n][e], v[n][e], ss);
+            }
+    }
+    const float inv = 1.0f / sqrtf(row_sum(ss, parts[3]) / (float)width + eps_z);
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int i = (n * LN_THREADS + (int)threadIdx.x) * VEC;
+        if (i < width) {
+            float w[VEC], bias[VEC];
+            load_vec<float, VEC>(w_z + i, w);
+            load_vec<float, VEC>(b_z + i, bias);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[n][e] = fmaf(v[n][e] * inv, w[e], bias[e]);
+            store_vec<TZ, VEC>(z + at + i, v[n]);
+        }
+    }
 }
 
 // Steps in which every sequence brings ONE token: the add, the layer norm and the short convolution over time that
@@ -206,7 +368,7 @@ __global__ void xielu_bf16x8_kernel(const uint4* __restrict__ in, uint4* __restr
 
 }  // namespace
 
-GK_EXPORT int gk_add_layernorm(float* h, const void* delta, int delta_dtype, float delta_scale, const void* weight,
+GK_EXPORT int gk_add_layernorm(float* h, const void* delta, int delta_dtype, float delta_scale, const void* weight, const void* bias,
                                int weight_dtype, void* out, int out_dtype, const int* rows, int n_out_rows, int hidden,
                                float eps, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(delta_dtype) && GK_VALID_DTYPE(weight_dtype) && GK_VALID_DTYPE(out_dtype), "add_layernorm: bad dtype code");
@@ -222,11 +384,50 @@ GK_EXPORT int gk_add_layernorm(float* h, const void* delta, int delta_dtype, flo
                 if (smem > 48 * 1024)
                     cudaFuncSetAttribute(add_layernorm_kernel<TD, TW, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
                 gk_launch(add_layernorm_kernel<TD, TW, TO>, dim3(n_out_rows), dim3(LN_THREADS), smem, s, h, (const TD*)delta,
-                          delta_scale, (const TW*)weight, (TO*)out, rows, hidden, eps);
+                          delta_scale, (const TW*)weight, (const TW*)bias, (TO*)out, rows, hidden, eps);
             })
         })
     })
     GK_CHECK_LAUNCH("add_layernorm");
+    return GK_OK;
+}
+
+// x, first, x_out [n_rows, width] 32-bit (x_out may be x), step [width]; w_y, b_y, w_z, b_z [width] 32-bit, both of a norm or
+// neither.
+GK_EXPORT int gk_layernorm_merge(const float* x, const void* y, int y_dtype, const float* w_y, const float* b_y, float eps_y,
+                                 const float* first, const float* step, float* x_out, const float* w_z, const float* b_z, float eps_z,
+                                 void* z, int z_dtype, int n_rows, int width, void* stream) {
+    GK_REQUIRE(GK_VALID_DTYPE(y_dtype) && GK_VALID_DTYPE(z_dtype), "layernorm_merge: bad dtype code");
+    GK_REQUIRE(n_rows >= 0 && width > 0 && x != nullptr && x_out != nullptr, "layernorm_merge: bad sizes rows=%d width=%d", n_rows, width);
+    GK_REQUIRE((w_y == nullptr) == (b_y == nullptr) && (w_y == nullptr || (y != nullptr && eps_y > 0.f)),
+               "layernorm_merge: the branch's norm needs a branch, a weight, a bias and a positive eps");
+    GK_REQUIRE((w_z == nullptr) == (b_z == nullptr) && (w_z == nullptr) == (z == nullptr) && (z == nullptr || eps_z > 0.f),
+               "layernorm_merge: the next norm needs a weight, a bias, an output and a positive eps");
+    if (n_rows == 0) return GK_OK;
+    const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)w_y | (uintptr_t)b_y | (uintptr_t)first | (uintptr_t)step |
+                          (uintptr_t)x_out | (uintptr_t)w_z | (uintptr_t)b_z | (uintptr_t)z;
+    const bool vec = width % 4 == 0 && (all & 15) == 0;
+    GK_REQUIRE(width <= (vec ? 16384 : 8192), "layernorm_merge: rows of %d are longer than a block holds", width);
+    cudaStream_t s = (cudaStream_t)stream;
+#define GK_MERGE(VEC, N)                                                                                                          \
+    gk_launch(layernorm_merge_kernel<TY, TZ, VEC, N>, dim3(n_rows), dim3(LN_THREADS), 0, s, x, (const TY*)y, w_y, b_y, eps_y, first, step, \
+              x_out, w_z, b_z, eps_z, (TZ*)z, width)
+    GK_DISPATCH_DTYPE(y_dtype, TY, {
+        GK_DISPATCH_DTYPE(z_dtype, TZ, {
+            if (vec) {
+                if (width <= 1024) GK_MERGE(4, 1);
+                else if (width <= 2048) GK_MERGE(4, 2);
+                else if (width <= 4096) GK_MERGE(4, 4);
+                else GK_MERGE(4, 16);
+            } else {
+                if (width <= 512) GK_MERGE(1, 2);
+                else if (width <= 2048) GK_MERGE(1, 8);
+                else GK_MERGE(1, 32);
+            }
+        })
+    })
+#undef GK_MERGE
+    GK_CHECK_LAUNCH("layernorm_merge");
     return GK_OK;
 }
 

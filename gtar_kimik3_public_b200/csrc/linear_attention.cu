@@ -1,7 +1,8 @@
 // Linear attention with a fixed decay per head, and what stands between the projections and it.
 //
-//   heads_prepare:  a warp per (token, head) of the packed projection q | k | v: optional SiLU (on q and k, on v),
-//                   rotation by position of the first `rot` entries of a q or k head (entry i paired with i + rot/2;
+//   heads_prepare:  a warp per (token, head) of the packed projection q | k | v: an optional bias per column, optional
+//                   SiLU (on q and k, on v), rotation by position of the first `rot` entries of a q or k head (entry i
+//                   paired with i + rot/2, or with flag 16 entry 2i with 2i + 1;
 //                   cosines and sines from tables of rot/2 angles a position), then optional division of a q or k
 //                   head by its root mean square (eps inside the root; times a weight per entry that all query heads or all
 //                   key heads share, where one is given), then a constant on k.  With flag 8
@@ -14,7 +15,8 @@
 //                   single tokens take the same path; a token's sums have the same order in all of them.
 //   group_norm_gate: rows cut into groups (a head, or all heads together), each first divided by a number of its own
 //                   where one is given, that are divided by their root mean square, multiplied by an optional weight (one
-//                   for all groups of a row, or one for the whole row) and by sigmoid or SiLU of a gate.
+//                   for all groups of a row, or one for the whole row), by a constant, and by sigmoid or SiLU of a gate;
+//                   the result's rows may be columns of wider rows.
 //
 // Everything is 32-bit except the projection that is read and the activations that are handed on.
 
@@ -28,10 +30,11 @@ __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); 
 constexpr int PREP_WARPS = 8;
 constexpr int PREP_MAX = 16;  // heads of up to 512 entries
 
-// flags: 1 SiLU on q and k, 2 SiLU on v, 4 unit root mean square of q and k, 8 values turned by position
+// flags: 1 SiLU on q and k, 2 SiLU on v, 4 unit root mean square of q and k, 8 values turned by position, 16 neighbours
+// turn together.  `bias` holds a number for every column from `bias_at` on (null: none).
 template <typename T, typename TQ>
 __global__ void __launch_bounds__(PREP_WARPS * 32) heads_prepare_kernel(
-    const T* __restrict__ proj, long long ld, int q_at, int k_at, int v_at, int n_q, int n_k, int d, int dv, int flags,
+    const T* __restrict__ proj, const float* __restrict__ bias, int bias_at, long long ld, int q_at, int k_at, int v_at, int n_q, int n_k, int d, int dv, int flags,
     int rot, const float* __restrict__ cos_t, const float* __restrict__ sin_t, const float* __restrict__ v_cos,
     const float* __restrict__ v_sin, float unit_eps, const float* __restrict__ w_q, const float* __restrict__ w_k, float k_scale,
     const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ slots,
@@ -49,7 +52,8 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) heads_prepare_kernel(
     const int kind = head < n_q ? 0 : head < n_q + n_k ? 1 : 2;  // q, k, v
     head -= kind == 0 ? 0 : kind == 1 ? n_q : n_q + n_k;
     const int width = kind == 2 ? dv : d;
-    const T* src = proj + (size_t)t * ld + (kind == 0 ? q_at : kind == 1 ? k_at : v_at) + (size_t)head * width;
+    const int column = (kind == 0 ? q_at : kind == 1 ? k_at : v_at) + head * width;
+    const T* src = proj + (size_t)t * ld + column;
     const bool to_pages = k_pages != nullptr;
     if (to_pages && kind != 0 && !write_kv) return;
     float x[PREP_MAX];
@@ -60,6 +64,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) heads_prepare_kernel(
         x[c] = 0.f;
         if (i < width) {
             x[c] = to_float(src[i]);
+            if (bias != nullptr) x[c] += bias[column - bias_at + i];
             if (act) x[c] = silu_f(x[c]);
         }
     }
@@ -79,7 +84,12 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) heads_prepare_kernel(
 #pragma unroll
             for (int c = 0; c < PREP_MAX; ++c) {
                 const int i = lane + 32 * c;
-                if (i < half) x[c] = mine[i] * cs[i] - mine[i + half] * sn[i];
+                if (flags & 16) {
+                    if (i < rot) {
+                        const float cosine = cs[i >> 1], sine = sn[i >> 1];
+                        x[c] = (i & 1) ? mine[i] * cosine + mine[i - 1] * sine : mine[i] * cosine - mine[i + 1] * sine;
+                    }
+                } else if (i < half) x[c] = mine[i] * cs[i] - mine[i + half] * sn[i];
                 else if (i < rot) x[c] = mine[i] * cs[i - half] + mine[i - half] * sn[i - half];
             }
         }
@@ -268,8 +278,8 @@ __global__ void __launch_bounds__(SCAN_LANES * SCAN_MAX_COLS) decay_scan_kernel(
 template <typename T, typename TG>
 __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ divisor,
                                                               const float* __restrict__ weight, int row_weight,
-                                                              const TG* __restrict__ gate, long long ld_gate, T* __restrict__ out,
-                                                              long long n_rows, int n_groups, int size, float eps, int gate_kind) {
+                                                              const TG* __restrict__ gate, long long ld_gate, T* __restrict__ out, long long ld_out,
+                                                              float out_scale, long long n_rows, int n_groups, int size, float eps, int gate_kind) {
     pdl_launch_dependents();
     pdl_wait();
     const long long row = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -283,14 +293,15 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
     ss = warp_sum(ss);
     // a group divided by c first: x / c has the mean square ss / c^2
     const float c = divisor != nullptr ? 1.f / divisor[row] : 1.f;
-    const float r = c / sqrtf(ss * c * c / (float)size + eps);
+    const float r = out_scale * (c / sqrtf(ss * c * c / (float)size + eps));
+    T* orow = out + (size_t)t * ld_out + (size_t)g * size;
     if (weight != nullptr && row_weight) weight += (size_t)g * size;
     const TG* gt = gate + (size_t)t * ld_gate + (size_t)g * size;
     for (int i = lane; i < size; i += 32) {
         const float z = to_float(gt[i]);
         float y = xr[i] * r;
         if (weight != nullptr) y *= weight[i];
-        out[(size_t)row * size + i] = from_float<T>(y * (gate_kind == 0 ? sigmoid_f(z) : silu_f(z)));
+        orow[i] = from_float<T>(y * (gate_kind == 0 ? sigmoid_f(z) : silu_f(z)));
     }
 }
 
@@ -299,7 +310,7 @@ template <typename T, typename TG>
 __global__ void __launch_bounds__(256) group_norm_gate_wide_kernel(const float* __restrict__ x, const float* __restrict__ divisor,
                                                                    const float* __restrict__ weight, int row_weight,
                                                                    const TG* __restrict__ gate, long long ld_gate, T* __restrict__ out,
-                                                                   int n_groups, int size, float eps, int gate_kind) {
+                                                                   long long ld_out, float out_scale, int n_groups, int size, float eps, int gate_kind) {
     __shared__ float scratch[33];
     pdl_launch_dependents();
     pdl_wait();
@@ -312,20 +323,21 @@ __global__ void __launch_bounds__(256) group_norm_gate_wide_kernel(const float* 
     ss = block_sum(ss, scratch);
     // a group divided by c first: x / c has the mean square ss / c^2
     const float c = divisor != nullptr ? 1.f / divisor[row] : 1.f;
-    const float r = c / sqrtf(ss * c * c / (float)size + eps);
+    const float r = out_scale * (c / sqrtf(ss * c * c / (float)size + eps));
+    T* orow = out + (size_t)t * ld_out + (size_t)g * size;
     if (weight != nullptr && row_weight) weight += (size_t)g * size;
     const TG* gt = gate + (size_t)t * ld_gate + (size_t)g * size;
     for (int i = threadIdx.x; i < size; i += 256) {
         const float z = to_float(gt[i]);
         float y = xr[i] * r;
         if (weight != nullptr) y *= weight[i];
-        out[(size_t)row * size + i] = from_float<T>(y * (gate_kind == 0 ? sigmoid_f(z) : silu_f(z)));
+        orow[i] = from_float<T>(y * (gate_kind == 0 ? sigmoid_f(z) : silu_f(z)));
     }
 }
 
 }  // namespace
 
-GK_EXPORT int gk_heads_prepare(const void* proj, int dtype, long long ld, int q_at, int k_at, int v_at, int n_q, int n_k, int d,
+GK_EXPORT int gk_heads_prepare(const void* proj, int dtype, const float* bias, int bias_at, long long ld, int q_at, int k_at, int v_at, int n_q, int n_k, int d,
                                int dv, int flags, int rot, const float* cos_t, const float* sin_t, const float* v_cos,
                                const float* v_sin, float unit_eps, const float* w_q, const float* w_k, float k_scale, const int* tok_pos, const int* tok_seq, const int* slots, void* q_out, int q_dtype, float* k_out,
                                float* v_out, void* k_pages, void* v_pages, const int* block_table, int max_pages, int page_size,
@@ -351,11 +363,11 @@ GK_EXPORT int gk_heads_prepare(const void* proj, int dtype, long long ld, int q_
     cudaStream_t s = (cudaStream_t)stream;
     GK_DISPATCH_DTYPE(dtype, T, {
         if (to_pages) {
-            gk_launch(heads_prepare_kernel<T, T>, dim3((unsigned)blocks), dim3(PREP_WARPS * 32), smem, s, (const T*)proj, ld, q_at,
+            gk_launch(heads_prepare_kernel<T, T>, dim3((unsigned)blocks), dim3(PREP_WARPS * 32), smem, s, (const T*)proj, bias, bias_at, ld, q_at,
                       k_at, v_at, n_q, n_k, d, dv, flags, rot, cos_t, sin_t, v_cos, v_sin, unit_eps, w_q, w_k, k_scale, tok_pos, tok_seq, slots, (T*)q_out,
                       (float*)nullptr, (float*)nullptr, (T*)k_pages, (T*)v_pages, block_table, max_pages, page_size, write_kv, items);
         } else {
-            gk_launch(heads_prepare_kernel<T, float>, dim3((unsigned)blocks), dim3(PREP_WARPS * 32), smem, s, (const T*)proj, ld,
+            gk_launch(heads_prepare_kernel<T, float>, dim3((unsigned)blocks), dim3(PREP_WARPS * 32), smem, s, (const T*)proj, bias, bias_at, ld,
                       q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot, cos_t, sin_t, v_cos, v_sin, unit_eps, w_q, w_k, k_scale, tok_pos, tok_seq, slots,
                       (float*)q_out, k_out, v_out, (T*)nullptr, (T*)nullptr, block_table, max_pages, page_size, write_kv, items);
         }
@@ -394,7 +406,7 @@ GK_EXPORT int gk_decay_scan(const float* q, const float* k, const float* v, cons
 }
 
 GK_EXPORT int gk_group_norm_gate(const float* x, const float* divisor, const float* weight, int row_weight, const void* gate, int gate_dtype, long long ld_gate, void* out,
-                                 int out_dtype, long long n_tokens, int n_groups, int size, float eps, int gate_kind, void* stream) {
+                                 long long ld_out, float out_scale, int out_dtype, long long n_tokens, int n_groups, int size, float eps, int gate_kind, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(gate_dtype) && GK_VALID_DTYPE(out_dtype), "group_norm_gate: bad dtype");
     GK_REQUIRE(n_groups > 0 && size > 0 && eps > 0.f && (gate_kind == 0 || gate_kind == 1), "group_norm_gate: bad sizes");
     if (n_tokens == 0) return GK_OK;
@@ -407,10 +419,10 @@ GK_EXPORT int gk_group_norm_gate(const float* x, const float* divisor, const flo
         GK_DISPATCH_DTYPE(gate_dtype, TG, {
             if (wide)
                 gk_launch(group_norm_gate_wide_kernel<T, TG>, dim3((unsigned)rows), dim3(256), 0, s, x, divisor, weight, row_weight, (const TG*)gate, ld_gate,
-                          (T*)out, n_groups, size, eps, gate_kind);
+                          (T*)out, ld_out, out_scale, n_groups, size, eps, gate_kind);
             else
                 gk_launch(group_norm_gate_kernel<T, TG>, dim3((unsigned)blocks), dim3(256), 0, s, x, divisor, weight, row_weight, (const TG*)gate, ld_gate,
-                          (T*)out, rows, n_groups, size, eps, gate_kind);
+                          (T*)out, ld_out, out_scale, rows, n_groups, size, eps, gate_kind);
         })
     })
     GK_CHECK_LAUNCH("group_norm_gate");

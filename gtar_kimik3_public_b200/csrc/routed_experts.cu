@@ -9,8 +9,11 @@
 //                and the chosen experts' weights are the softmax over the chosen scores alone, times the constant.
 //                Further rules (flags): s = softmax(z) over all experts; a group's score is its largest choice score; the
 //                chosen experts' s are divided by their sum (plus 1e-20) before the constant.
+//                A shared expert that every token runs, weighted by the sigmoid of a number of its own: that number's row
+//                stands behind the router's rows (z has E + 1 entries), and the sigmoid is either the weight of one more
+//                pair (token, expert E) behind the token's chosen ones, or an output of its own.
 //   experts_up   act[pair] = silu(W_gate[e] h_t) * (W_up[e] h_t) for every pair (token, chosen expert)
-//   experts_down out_t = add_t + sum over the token's pairs, in the order they were chosen, of weight * W_down[e] act[pair]
+//   experts_down out_t = add_t (times a number per token, where one is given) + sum over the token's pairs, in the order they were chosen, of weight * W_down[e] act[pair]
 //                (32-bit result: it is what goes into the residual stream)
 //
 // The two expert kernels take a pair at a time, one warp per output row: the path of single-token steps, of 32-bit
@@ -71,10 +74,12 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_scores_kernel(const T*
 
 enum RouteFlags : int { ROUTE_LOGITS = 1, ROUTE_SOFTMAX = 2, ROUTE_GROUP_BEST = 4, ROUTE_RENORMALISE = 8 };
 
-// The choice from the scores: one warp per token.
+// The choice from the scores: one warp per token.  z has n_scores = n_experts or n_experts + 1 entries a token; ids and
+// weights have ld_pairs.
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_choose_kernel(
     const float* __restrict__ z, const float* __restrict__ correction, int* __restrict__ ids, float* __restrict__ weights,
-    int n_tokens, int n_experts, int top, int n_groups, int keep, float scale, int flags) {
+    int n_tokens, int n_experts, int top, int n_groups, int keep, float scale, int flags, int n_scores, int ld_pairs,
+    float* __restrict__ shared_weight) {
     extern __shared__ float route_smem[];  // per warp: s [E] | choice [E] | group score [n_groups]
     pdl_launch_dependents();
     pdl_wait();
@@ -87,16 +92,24 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_choose_kernel(
     const bool logits = (flags & ROUTE_LOGITS) != 0, softmax = (flags & ROUTE_SOFTMAX) != 0;
     float largest_z = -INFINITY, denom = 0.f;
     if (softmax) {
-        for (int e = lane; e < n_experts; e += 32) largest_z = fmaxf(largest_z, z[(size_t)t * n_experts + e]);
+        for (int e = lane; e < n_experts; e += 32) largest_z = fmaxf(largest_z, z[(size_t)t * n_scores + e]);
         largest_z = warp_max(largest_z);
-        for (int e = lane; e < n_experts; e += 32) denom += expf(z[(size_t)t * n_experts + e] - largest_z);
+        for (int e = lane; e < n_experts; e += 32) denom += expf(z[(size_t)t * n_scores + e] - largest_z);
         denom = warp_sum(denom);
     }
     for (int e = lane; e < n_experts; e += 32) {
-        const float ze = z[(size_t)t * n_experts + e];
+        const float ze = z[(size_t)t * n_scores + e];
         const float sg = logits ? ze + correction[e] : softmax ? expf(ze - largest_z) / denom : 1.f / (1.f + expf(-ze));
         s[e] = sg;
         choice[e] = logits ? sg : sg + correction[e];
+    }
+    if (n_scores > n_experts && lane == 0) {
+        const float share = 1.f / (1.f + expf(-z[(size_t)t * n_scores + n_experts]));
+        if (shared_weight != nullptr) shared_weight[t] = share;
+        else {
+            ids[(size_t)t * ld_pairs + top] = n_experts;
+            weights[(size_t)t * ld_pairs + top] = share;
+        }
     }
     __syncwarp();
     const int per = n_experts / n_groups;
@@ -136,21 +149,21 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_choose_kernel(
         }
         if (arg == 0x7fffffff) arg = 0;  // nothing left to choose from: cannot happen when top <= allowed experts
         if (lane == 0) {
-            ids[(size_t)t * top + pick] = arg;
-            weights[(size_t)t * top + pick] = logits || (flags & ROUTE_RENORMALISE) ? s[arg] : s[arg] * scale;
+            ids[(size_t)t * ld_pairs + pick] = arg;
+            weights[(size_t)t * ld_pairs + pick] = logits || (flags & ROUTE_RENORMALISE) ? s[arg] : s[arg] * scale;
             choice[arg] = -INFINITY;
         }
         __syncwarp();
     }
     if ((flags & ROUTE_RENORMALISE) && lane == 0) {
-        float* w = weights + (size_t)t * top;
+        float* w = weights + (size_t)t * ld_pairs;
         float sum = 0.f;
         for (int pick = 0; pick < top; ++pick) sum += w[pick];
         for (int pick = 0; pick < top; ++pick) w[pick] = w[pick] / (sum + 1e-20f) * scale;
     }
     if (logits && lane == 0) {
         // softmax over the chosen scores, in the order they were chosen (the first is the largest)
-        float* w = weights + (size_t)t * top;
+        float* w = weights + (size_t)t * ld_pairs;
         const float largest = w[0];
         float sum = 0.f;
         for (int pick = 0; pick < top; ++pick) sum += expf(w[pick] - largest);
@@ -279,7 +292,8 @@ __global__ void __launch_bounds__(UP_WARPS * 32) experts_up_kernel(
 template <typename T, typename TW>
 __global__ void __launch_bounds__(UP_WARPS * 32) experts_down_kernel(
     const T* __restrict__ act, const TW* __restrict__ w_down, const int* __restrict__ ids, const float* __restrict__ weights,
-    const T* __restrict__ add, float* __restrict__ out, int width, int ff, int top, int rows_per_block) {
+    const T* __restrict__ add, const float* __restrict__ add_weight, float* __restrict__ out, int width, int ff, int top,
+    int rows_per_block) {
     extern __shared__ __align__(16) float as[];  // top * ff
     pdl_launch_dependents();
     pdl_wait();
@@ -290,6 +304,7 @@ __global__ void __launch_bounds__(UP_WARPS * 32) experts_down_kernel(
     const int c0 = blockIdx.y * rows_per_block;
     for (int c = c0 + warp; c < min(width, c0 + rows_per_block); c += UP_WARPS) {
         float acc = add != nullptr ? to_float(add[(size_t)t * width + c]) : 0.f;
+        if (add_weight != nullptr) acc *= add_weight[t];
         int kk = 0;
         for (; kk + 1 < top; kk += 2) {  // two experts' rows in flight; the sum still takes them in the order they were chosen
             const int e0 = ids[(size_t)t * top + kk], e1 = ids[(size_t)t * top + kk + 1];
@@ -360,12 +375,14 @@ __global__ void gather_rows_kernel(const T* __restrict__ x, const int* __restric
 // out_t = add_t + sum_k weights[t, k] * y[place_of[t, k]] in the order the experts were chosen (32-bit)
 template <typename T>
 __global__ void experts_combine_kernel(const T* __restrict__ y, const int* __restrict__ place_of, const float* __restrict__ weights,
-                                       const T* __restrict__ add, float* __restrict__ out, int width, int top) {
+                                       const T* __restrict__ add, const float* __restrict__ add_weight, float* __restrict__ out,
+                                       int width, int top) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t t = blockIdx.x;
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         float acc = add != nullptr ? to_float(add[t * width + c]) : 0.f;
+        if (add_weight != nullptr) acc *= add_weight[t];
         for (int kk = 0; kk < top; ++kk)
             acc = fmaf(weights[t * top + kk], to_float(y[(size_t)place_of[t * top + kk] * width + c]), acc);
         out[t * width + c] = acc;
@@ -392,21 +409,23 @@ GK_EXPORT int gk_gather_rows(const void* x, int dtype, const int* pair_at, void*
     return GK_OK;
 }
 
-GK_EXPORT int gk_experts_combine(const void* y, int dtype, const int* place_of, const float* weights, const void* add, float* out,
-                                 int n_tokens, int width, int top, void* stream) {
-    GK_REQUIRE(GK_VALID_DTYPE(dtype) && width > 0 && top > 0, "experts_combine: bad arguments");
+GK_EXPORT int gk_experts_combine(const void* y, int dtype, const int* place_of, const float* weights, const void* add,
+                                 const float* add_weight, float* out, int n_tokens, int width, int top, void* stream) {
+    GK_REQUIRE(GK_VALID_DTYPE(dtype) && width > 0 && top > 0 && (add != nullptr || add_weight == nullptr), "experts_combine: bad arguments");
     if (n_tokens == 0) return GK_OK;
     GK_DISPATCH_DTYPE(dtype, T, {
         gk_launch(experts_combine_kernel<T>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, (const T*)y, place_of, weights,
-                  (const T*)add, out, width, top);
+                  (const T*)add, add_weight, out, width, top);
     })
     GK_CHECK_LAUNCH("experts_combine");
     return GK_OK;
 }
 
+// shared: w_router and z have one row more, the shared expert's number; its sigmoid goes to shared_weight [T] or, where that is
+// null, to one more pair a token (ids and weights [T, top + 1]).
 GK_EXPORT int gk_route_groups(const void* h, int dtype, const float* w_router, const float* correction, float* z, int* ids,
                               float* weights, int n_tokens, int width, int n_experts, int top, int n_groups, int keep, float scale, int flags,
-                              void* stream) {
+                              int shared, float* shared_weight, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(dtype), "route_groups: bad dtype %d", dtype);
     GK_REQUIRE(n_experts > 0 && top > 0 && top <= n_experts, "route_groups: %d of %d experts", top, n_experts);
     GK_REQUIRE(n_groups >= 1 && n_experts % n_groups == 0 && keep >= 1 && keep <= n_groups, "route_groups: %d groups, %d kept, %d experts",
@@ -421,18 +440,19 @@ GK_EXPORT int gk_route_groups(const void* h, int dtype, const float* w_router, c
     const bool many = (long long)((n_tokens + 7) / 8) * ((n_experts + 7) / 8) >= 512;
     const int per_warp = many ? 8 : 2;
     const int token_groups = (n_tokens + 3) / 4;
-    const long long units = (long long)token_groups * ((n_experts + per_warp - 1) / per_warp);
+    const int n_scores = n_experts + (shared ? 1 : 0), ld_pairs = top + (shared && shared_weight == nullptr ? 1 : 0);
+    const long long units = (long long)token_groups * ((n_scores + per_warp - 1) / per_warp);
     GK_REQUIRE(units / ROUTE_WARPS < 2147483647LL, "route_groups: too many tokens");
     const dim3 score_grid((unsigned)((units + ROUTE_WARPS - 1) / ROUTE_WARPS));
     GK_DISPATCH_DTYPE(dtype, T, {
         if (per_warp == 8)
-            gk_launch(route_scores_kernel<T, 8, 4>, score_grid, dim3(ROUTE_WARPS * 32), 0, s, (const T*)h, w_router, z, n_tokens, width, n_experts);
+            gk_launch(route_scores_kernel<T, 8, 4>, score_grid, dim3(ROUTE_WARPS * 32), 0, s, (const T*)h, w_router, z, n_tokens, width, n_scores);
         else
-            gk_launch(route_scores_kernel<T, 2, 4>, score_grid, dim3(ROUTE_WARPS * 32), 0, s, (const T*)h, w_router, z, n_tokens, width, n_experts);
+            gk_launch(route_scores_kernel<T, 2, 4>, score_grid, dim3(ROUTE_WARPS * 32), 0, s, (const T*)h, w_router, z, n_tokens, width, n_scores);
     })
     GK_CHECK_LAUNCH("route_scores");
     gk_launch(route_choose_kernel, dim3((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, s, (const float*)z,
-              correction, ids, weights, n_tokens, n_experts, top, n_groups, keep, scale, flags);
+              correction, ids, weights, n_tokens, n_experts, top, n_groups, keep, scale, flags, n_scores, ld_pairs, shared_weight);
     GK_CHECK_LAUNCH("route_groups");
     return GK_OK;
 }
@@ -463,9 +483,9 @@ GK_EXPORT int gk_experts_up(const void* h, int dtype, const void* w_gate_up, int
 }
 
 GK_EXPORT int gk_experts_down(const void* act, int dtype, const void* w_down, int w_dtype, const int* ids, const float* weights,
-                              const void* add, float* out, int n_tokens, int width, int ff, int top, void* stream) {
+                              const void* add, const float* add_weight, float* out, int n_tokens, int width, int ff, int top, void* stream) {
     GK_REQUIRE(GK_VALID_DTYPE(dtype) && GK_VALID_DTYPE(w_dtype), "experts_down: bad dtype");
-    GK_REQUIRE(width > 0 && ff > 0 && top > 0, "experts_down: bad sizes");
+    GK_REQUIRE(width > 0 && ff > 0 && top > 0 && (add != nullptr || add_weight == nullptr), "experts_down: bad sizes");
     if (n_tokens == 0) return GK_OK;
     const size_t smem = (size_t)top * ff * sizeof(float);
     GK_REQUIRE(smem <= 200 * 1024, "experts_down: %d experts of %d are more than the kernel stages", top, ff);
@@ -477,7 +497,7 @@ GK_EXPORT int gk_experts_down(const void* act, int dtype, const void* w_down, in
         GK_DISPATCH_DTYPE(w_dtype, TW, {
             if (smem > 48 * 1024) cudaFuncSetAttribute(experts_down_kernel<T, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
             gk_launch(experts_down_kernel<T, TW>, dim3(n_tokens, (width + rows - 1) / rows), dim3(UP_WARPS * 32), smem, s, (const T*)act,
-                      (const TW*)w_down, ids, weights, (const T*)add, out, width, ff, top, rows);
+                      (const TW*)w_down, ids, weights, (const T*)add, add_weight, out, width, ff, top, rows);
         })
     })
     GK_CHECK_LAUNCH("experts_down");

@@ -19,12 +19,52 @@ from ..parts.base import Block, Norm, Part, PositionEncoding, StepContext, Tenso
 from ..parts.embedding import OutputHead, TokenEmbedding
 
 
+@dataclass(frozen=True)
+class Enter:
+    """What is added to the stream right before an entry of the run list: the embedding output (the stream as it was before the
+    first entry), and a row of the plan's table of steps."""
+
+    embedding: bool = False
+    step: int | None = None
+
+
 @dataclass
 class RunEntry:
-    """One step of the run list: which layer runs, and whose storage it uses (None: its own)."""
+    """One step of the run list: which layer runs, whose storage it uses (None: its own), and what is added before it."""
 
     layer: int
     cache_of: int | None = None  # index of an earlier run-list entry
+    enter: Enter | None = None
+
+
+class StepTable(Part):
+    """Vectors that are added to the stream at entries of the run list (``Enter.step`` is a row)."""
+
+    graph_safe = True
+
+    def __init__(self, rows: int, size: int, weight_name: str = "step"):
+        self.rows, self.size, self.weight_name = int(rows), int(size), weight_name
+        self.table: torch.Tensor | None = None
+
+    def tensor_specs(self):
+        return {self.weight_name: TensorSpec((self.rows, self.size), "vector", init=(0.0, 0.5))}
+
+    def load(self, tensors):
+        self.table = tensors[self.weight_name].float().contiguous()
+
+
+def looped_run_list(n_layers: int, start: int, stop: int, times: int, steps: bool = False) -> list[RunEntry]:
+    """The run list of ``n_layers`` layers of which ``start .. stop - 1`` run ``times`` times in a row with the same weights, every
+    pass with storage of its own.  Before each pass but the first the embedding output is added, and with ``steps`` before each
+    pass the row of the step table with the pass's number."""
+    if not 0 <= start < stop <= n_layers or times < 1:
+        raise ValueError(f"layers {start} .. {stop - 1} of {n_layers} cannot run {times} times")
+    entries = [RunEntry(i) for i in range(start)]
+    for t in range(times):
+        for i in range(start, stop):
+            enter = Enter(embedding=t > 0, step=t if steps else None) if i == start and (t > 0 or steps) else None
+            entries.append(RunEntry(i, enter=enter))
+    return entries + [RunEntry(i) for i in range(stop, n_layers)]
 
 
 @dataclass
@@ -42,6 +82,8 @@ class ModelPlan:
     # Layers that mix the results of earlier layers into their stream need those kept for the length of a step:
     # how many streams a step keeps (the embedding output and every layer's result), 0 for none.
     keep_streams: int = 0
+    steps: StepTable | None = None  # what the run list's ``Enter.step`` name
+    steps_prefix: str = "loop."
 
 
 class Model:
@@ -54,6 +96,8 @@ class Model:
                 raise ValueError(f"run-list entry {position} names layer {entry.layer}; there are {len(plan.layers)}")
             if entry.cache_of is not None and not 0 <= entry.cache_of < position:
                 raise ValueError(f"run-list entry {position} may only read the storage of an earlier entry")
+            if entry.enter is not None and entry.enter.step is not None and (plan.steps is None or not 0 <= entry.enter.step < plan.steps.rows):
+                raise ValueError(f"run-list entry {position} names row {entry.enter.step} of the step table, which has no such row")
         self.vocab_size = plan.head.vocab_size
 
     # ------------------------------------------------------------------ weights
@@ -62,6 +106,8 @@ class Model:
         parts: list[tuple[str, Part]] = [(plan.embedding_prefix, plan.embedding)]
         parts += [(plan.layer_prefix.format(i), layer) for i, layer in enumerate(plan.layers)]
         parts += [(plan.final_norm_prefix, plan.final_norm), (plan.head_prefix, plan.head)]
+        if plan.steps is not None:
+            parts.insert(1, (plan.steps_prefix, plan.steps))
         return parts
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
@@ -114,6 +160,13 @@ class Model:
         for position in self.plan.positions:
             position.prepare(max_position, self.device)
 
+    def _enter(self, entry: RunEntry, first: torch.Tensor | None) -> tuple | None:
+        """(embedding output or None, step vector or None) that is added to the stream before the entry, or None."""
+        if entry.enter is None:
+            return None
+        row = None if entry.enter.step is None else self.plan.steps.table[entry.enter.step]
+        return (first if entry.enter.embedding else None, row)
+
     def step(self, ctx: StepContext, cache: Cache) -> torch.Tensor:
         """Runs the step's tokens through the run list and returns float32 logits ``[n_want, vocab]``
         at ``ctx.want_rows``."""
@@ -131,9 +184,24 @@ class Model:
         if persistent is not None:
             persistent.run(h, ctx)  # every layer of the run list in one kernel; the stream is complete afterwards
         else:
-            for index, entry in enumerate(plan.run_list):
+            first = stream = None
+            if any(entry.enter is not None and entry.enter.embedding for entry in plan.run_list):
+                first, stream = h, torch.empty_like(h)  # the embedding output stays as it is; the layers' sums go to the stream
+            ctx.extras["stream"] = stream
+            enters = [self._enter(entry, first) for entry in plan.run_list]
+            blocks = [plan.layers[entry.layer] for entry in plan.run_list]
+            for index, block in enumerate(blocks):
                 ctx.extras["cache_read_only"] = cache.is_shared(index)
-                h, pending = plan.layers[entry.layer].forward(h, pending, ctx, cache.view(index))
+                if block.hands_on:
+                    ctx.extras["enter"] = enters[index]
+                    follows = index + 1 < len(blocks) and blocks[index + 1].hands_on
+                    ctx.extras["follower"] = (blocks[index + 1], enters[index + 1]) if follows else None
+                elif enters[index] is not None:
+                    h, _ = F.layernorm_merge(h, pending, first=enters[index][0], step=enters[index][1], x_out=h if stream is None else stream)
+                    pending = None
+                elif first is not None and h.data_ptr() == first.data_ptr():
+                    h = stream.copy_(h)
+                h, pending = block.forward(h, pending, ctx, cache.view(index))
         if ctx.want_rows.numel() == 0:
             # nothing asked for: still fold the last branch into the stream so the step is whole
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=self.device)

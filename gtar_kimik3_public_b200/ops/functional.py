@@ -12,7 +12,7 @@ from dataclasses import dataclass
 
 import torch
 
-from .library import KernelError, call, dtype_code, ptr, require_device, stream_ptr
+from .library import KernelError, call, dtype_code, library, ptr, require_device, stream_ptr
 
 
 def _check(tensor: torch.Tensor, name: str, dtype=None, dims: int | None = None) -> None:
@@ -1318,19 +1318,21 @@ DELTA_SCAN_COLS = int(__import__("os").environ.get("GTAR_B200_SCAN_COLS", "0")) 
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
                cu_q: torch.Tensor, slots: torch.Tensor, n_seqs: int) -> torch.Tensor:
     """The recurrence ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` over the step's tokens of every
-    sequence, from and to ``state [slots, n_heads, d, dv]`` (32-bit).  Returns ``o [T, n_heads, dv]`` (32-bit)."""
+    sequence, from and to ``state [slots, n_heads, d, dv]`` (32-bit).  ``g``: a decay per key channel ``[T, n_heads, d]`` or one
+    per head ``[T, n_heads]``.  Returns ``o [T, n_heads, dv]`` (32-bit)."""
     require_device(q.device)
-    for name, t in (("q", q), ("k", k), ("v", v), ("g", g)):
+    for name, t in (("q", q), ("k", k), ("v", v)):
         _check(t, name, torch.float32, 3)
+    _check(g, "g", torch.float32, 2 if g.dim() == 2 else 3)
     _check(beta, "beta", torch.float32, 2)
     _check(state, "state", torch.float32, 4)
     T, n_kv, d = q.shape
     n_heads, dv = v.shape[1], v.shape[2]
-    if tuple(state.shape[1:]) != (n_heads, d, dv) or tuple(g.shape) != (T, n_heads, d) or k.shape != q.shape:
+    if tuple(state.shape[1:]) != (n_heads, d, dv) or tuple(g.shape) not in ((T, n_heads, d), (T, n_heads)) or k.shape != q.shape:
         raise KernelError("delta_scan: the state or the inputs have other sizes than the heads")
     out = torch.empty((T, n_heads, dv), dtype=torch.float32, device=q.device)
     call("gk_delta_scan", ptr(q), ptr(k), ptr(v), ptr(g), ptr(beta), ptr(state), ptr(out), ptr(cu_q), ptr(slots), n_seqs, n_heads,
-         n_kv, d, dv, DELTA_SCAN_LANES, DELTA_SCAN_COLS, stream_ptr())
+         n_kv, d, dv, DELTA_SCAN_LANES, DELTA_SCAN_COLS, int(g.dim() == 2), stream_ptr())
     return out
 
 
@@ -1349,36 +1351,168 @@ def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, ga
     return out
 
 
+# ------------------------------------------------------------------ the delta rule with one decay per head
+@dataclass(frozen=True)
+class DeltaHeads:
+    """Sizes of a delta rule with one decay per head, and where its columns start in the rows of a packed projection:
+    q (n_kv d) | k (n_kv d) | v (n_heads dv) | b (n_heads) | a (n_heads) | gate (n_heads dv)."""
+
+    n_heads: int
+    n_kv: int
+    d: int
+    dv: int
+    taps: int
+
+    @property
+    def channels(self) -> int:
+        return 2 * self.n_kv * self.d + self.n_heads * self.dv
+
+    @property
+    def gate_at(self) -> int:
+        return self.channels + 2 * self.n_heads
+
+    @property
+    def columns(self) -> int:
+        return self.gate_at + self.n_heads * self.dv
+
+    def state_shape(self) -> tuple[int, int, int]:
+        return (self.n_heads, self.d, self.dv)
+
+    def ring_shape(self) -> tuple[int, int]:
+        return (self.taps, self.channels)
+
+
+def _check_delta_head(proj: torch.Tensor, at: int, hd: DeltaHeads, conv_w: torch.Tensor, ring: torch.Tensor | None, a_log: torch.Tensor,
+                      dt_bias: torch.Tensor) -> None:
+    require_device(proj.device)
+    _check(proj, "proj", dims=2)
+    if at < 0 or proj.shape[1] < at + hd.columns:
+        raise KernelError(f"a projection of {proj.shape[1]} columns is too narrow for {hd} from column {at}")
+    _check(conv_w, "conv_w", torch.float32, 2)
+    if tuple(conv_w.shape) != (hd.taps, hd.channels):
+        raise KernelError(f"conv_w is {tuple(conv_w.shape)}, expected {(hd.taps, hd.channels)}")
+    if hd.taps > 1:
+        _check(ring, "ring", torch.float32, 3)
+        if tuple(ring.shape[1:]) != hd.ring_shape():
+            raise KernelError(f"the convolution state is {tuple(ring.shape)}, expected [slots, {hd.taps}, {hd.channels}]")
+    for name, t in (("a_log", a_log), ("dt_bias", dt_bias)):
+        _check(t, name, torch.float32, 1)
+        if t.shape[0] != hd.n_heads:
+            raise KernelError(f"{name} has {t.shape[0]} entries for {hd.n_heads} heads")
+
+
+@dataclass
+class DeltaInputs:
+    """What a recurrence reads.  32-bit: unit q, k ``[T, n_kv, d]``, v ``[T, n_heads, dv]``, ``g`` the decay factors.  ``rounded``:
+    q, k, v in bfloat16, ``q_unit``, ``k_unit [T, n_kv]`` the factors that make q and k unit vectors (q's with ``d ** -0.5``),
+    ``g`` the decays' logarithms.  ``g``, ``beta`` ``[T, n_heads]``, always 32-bit."""
+
+    q: torch.Tensor
+    k: torch.Tensor
+    v: torch.Tensor
+    g: torch.Tensor
+    beta: torch.Tensor
+    q_unit: torch.Tensor | None = None
+    k_unit: torch.Tensor | None = None
+
+
+def delta_head_prepare(proj: torch.Tensor, at: int, hd: DeltaHeads, conv_w: torch.Tensor, ring: torch.Tensor | None, a_log: torch.Tensor,
+                       dt_bias: torch.Tensor, tok_pos: torch.Tensor, tok_seq: torch.Tensor, cu_q: torch.Tensor, slots: torch.Tensor,
+                       rounded: bool = False) -> DeltaInputs:
+    """Everything between the packed projection and the recurrence, in 32-bit.  ``ring [slots, taps, channels]`` holds the
+    inputs before the step (the input at position ``p`` in row ``p % taps``) and is not written (``conv_ring`` follows)."""
+    _check_delta_head(proj, at, hd, conv_w, ring, a_log, dt_bias)
+    for name, t in (("tok_pos", tok_pos), ("tok_seq", tok_seq), ("cu_q", cu_q), ("slots", slots)):
+        _check(t, name, torch.int32, 1)
+    T, dev = proj.shape[0], proj.device
+    kind = torch.bfloat16 if rounded else torch.float32
+    out = DeltaInputs(q=torch.empty((T, hd.n_kv, hd.d), dtype=kind, device=dev), k=torch.empty((T, hd.n_kv, hd.d), dtype=kind, device=dev),
+                      v=torch.empty((T, hd.n_heads, hd.dv), dtype=kind, device=dev),
+                      g=torch.empty((T, hd.n_heads), dtype=torch.float32, device=dev),
+                      beta=torch.empty((T, hd.n_heads), dtype=torch.float32, device=dev))
+    if rounded:
+        out.q_unit = torch.empty((T, hd.n_kv), dtype=torch.float32, device=dev)
+        out.k_unit = torch.empty((T, hd.n_kv), dtype=torch.float32, device=dev)
+    call("gk_delta_head_prepare", proj.data_ptr() + at * proj.element_size(), dtype_code(proj.dtype), proj.shape[1], ptr(conv_w),
+         ptr(ring) if hd.taps > 1 else None, ptr(a_log), ptr(dt_bias), ptr(tok_pos), ptr(tok_seq), ptr(cu_q), ptr(slots), ptr(out.q),
+         ptr(out.k), ptr(out.v), ptr(out.q_unit), ptr(out.k_unit), ptr(out.g), ptr(out.beta), int(rounded), T, hd.n_heads, hd.n_kv,
+         hd.d, hd.dv, hd.taps, stream_ptr())
+    return out
+
+
+def conv_ring(proj: torch.Tensor, at: int, hd: DeltaHeads, ring: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
+              slots: torch.Tensor) -> None:
+    """Leaves every sequence's last inputs of the step in its ring.  ``kv_len``: the sequences' tokens including the step's."""
+    _check(ring, "ring", torch.float32, 3)
+    call("gk_conv_ring", proj.data_ptr() + at * proj.element_size(), dtype_code(proj.dtype), proj.shape[1], ptr(ring), ptr(cu_q),
+         ptr(kv_len), ptr(slots), kv_len.shape[0], hd.channels, hd.taps, stream_ptr())
+
+
+def delta_head_single_fits(d: int, dv: int) -> bool:
+    """Whether :func:`delta_head_single` takes heads of these sizes (a block holds a head's state in registers)."""
+    return bool(library().gk_delta_head_single_fits(int(d), int(dv)))
+
+
+def delta_head_single(proj: torch.Tensor, at: int, hd: DeltaHeads, conv_w: torch.Tensor, ring: torch.Tensor | None, a_log: torch.Tensor,
+                      dt_bias: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, tok_pos: torch.Tensor, tok_seq: torch.Tensor,
+                      slots: torch.Tensor, eps: float, out: torch.Tensor, out_at: int = 0, out_scale: float = 1.0) -> None:
+    """Steps of one token a sequence: convolutions, unit lengths, decay, the recurrence from and to ``state [slots, n_heads, d,
+    dv]``, the norm of every head's read-out, weight and silu(gate), in one kernel.  The result, times ``out_scale``, goes to
+    columns ``out_at ..`` of ``out [T, ...]``; state and ring are moved on."""
+    _check_delta_head(proj, at, hd, conv_w, ring, a_log, dt_bias)
+    _check(norm_w, "norm_w", torch.float32, 1)
+    _check(state, "state", torch.float32, 4)
+    _check(out, "out", proj.dtype, 2)
+    T = proj.shape[0]
+    if tuple(state.shape[1:]) != hd.state_shape() or norm_w.shape[0] != hd.dv:
+        raise KernelError("delta_head_single: the state or the norm's weight have other sizes than the heads")
+    if out.shape[0] != T or out.shape[1] < out_at + hd.n_heads * hd.dv:
+        raise KernelError(f"delta_head_single: results do not fit {tuple(out.shape)} from column {out_at}")
+    for name, t in (("tok_pos", tok_pos), ("tok_seq", tok_seq), ("slots", slots)):
+        _check(t, name, torch.int32, 1)
+    call("gk_delta_head_single", proj.data_ptr() + at * proj.element_size(), dtype_code(proj.dtype), proj.shape[1], ptr(conv_w),
+         ptr(ring) if hd.taps > 1 else None, ptr(a_log), ptr(dt_bias), ptr(norm_w), ptr(state), ptr(tok_pos), ptr(tok_seq), ptr(slots),
+         out.data_ptr() + out_at * out.element_size(), out.shape[1], float(out_scale), float(eps), T, hd.n_heads, hd.n_kv, hd.d, hd.dv,
+         hd.taps, stream_ptr())
+
+
 # ------------------------------------------------------------------ routed experts
 def route_groups(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor, top: int, n_groups: int, keep: int,
                  scale: float, logits: bool = False, softmax: bool = False, best_of_group: bool = False,
-                 renormalise: bool = False) -> tuple[torch.Tensor, torch.Tensor]:
+                 renormalise: bool = False, shared: str | None = None) -> tuple[torch.Tensor, ...]:
     """Chosen experts ``[T, top]`` (int32) and their weights (float32): sigmoid scores, choice by score plus
     ``correction`` among the experts of the best ``keep`` of ``n_groups`` groups, weight = score times ``scale``.
     ``logits``: the score is the logit plus ``correction`` (a bias), the choice goes by it, and the weights are the
     softmax over the chosen scores alone, times ``scale``.  ``softmax``: scores are the softmax of the logits over all experts;
     ``best_of_group``: a group's score is its largest choice score (else its two largest added); ``renormalise``: the chosen
-    scores are divided by their sum plus 1e-20 before ``scale``."""
+    scores are divided by their sum plus 1e-20 before ``scale``.  ``shared``: the last row of ``w_router`` is no expert's but gives
+    the number whose sigmoid weights a shared expert: ``"pair"``: every token gets one more pair, with the expert behind the last
+    one and that weight (the results are ``[T, top + 1]``); ``"weight"``: the weights ``[T]`` are a third result."""
     require_device(h.device)
     _check(h, "h", dims=2)
     _check(w_router, "w_router", torch.float32, 2)
     _check(correction, "correction", torch.float32, 1)
     T, width = h.shape
-    n_experts = w_router.shape[0]
+    n_scores = w_router.shape[0]
+    n_experts = n_scores - (1 if shared else 0)
     if w_router.shape[1] != width or correction.shape[0] != n_experts:
         raise KernelError("route_groups: router sizes do not fit")
-    ids = torch.empty((T, top), dtype=torch.int32, device=h.device)
-    weights = torch.empty((T, top), dtype=torch.float32, device=h.device)
-    z = torch.empty((T, n_experts), dtype=torch.float32, device=h.device)
+    pairs = top + (1 if shared == "pair" else 0)
+    ids = torch.empty((T, pairs), dtype=torch.int32, device=h.device)
+    weights = torch.empty((T, pairs), dtype=torch.float32, device=h.device)
+    z = torch.empty((T, n_scores), dtype=torch.float32, device=h.device)
+    share = torch.empty((T,), dtype=torch.float32, device=h.device) if shared == "weight" else None
     call("gk_route_groups", ptr(h), dtype_code(h.dtype), ptr(w_router), ptr(correction), ptr(z), ptr(ids), ptr(weights), T, width, n_experts,
-         top, n_groups, keep, float(scale), bool(logits) + 2 * bool(softmax) + 4 * bool(best_of_group) + 8 * bool(renormalise), stream_ptr())
-    return ids, weights
+         top, n_groups, keep, float(scale), bool(logits) + 2 * bool(softmax) + 4 * bool(best_of_group) + 8 * bool(renormalise), int(shared is not None), ptr(share),
+         stream_ptr())
+    return (ids, weights) if share is None else (ids, weights, share)
 
 
 def experts_pairwise(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                     add: torch.Tensor | None = None) -> torch.Tensor:
+                     add: torch.Tensor | None = None, add_weight: torch.Tensor | None = None) -> torch.Tensor:
     """``add + sum_k weights[t, k] * down_e(silu(gate_e h_t) * up_e h_t)`` with ``e = ids[t, k]``, a (token, expert) pair
-    at a time.  ``w_gate_up [E, 2, ff, width]``, ``w_down [E, width, ff]``.  Returns 32-bit ``[T, width]``."""
+    at a time (``add`` times ``add_weight [T]`` where given).  ``w_gate_up [E, 2, ff, width]``, ``w_down [E, width, ff]``.  Returns
+    32-bit ``[T, width]``."""
     require_device(h.device)
     _check(h, "h", dims=2)
     _check(w_gate_up, "w_gate_up", dims=4)
@@ -1397,7 +1531,7 @@ def experts_pairwise(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Ten
     call("gk_experts_up", ptr(h), dtype_code(h.dtype), ptr(w_gate_up), dtype_code(w_gate_up.dtype), ptr(ids), ptr(act), T, width, ff,
          top, stream_ptr())
     call("gk_experts_down", ptr(act), dtype_code(h.dtype), ptr(w_down), dtype_code(w_down.dtype), ptr(ids), ptr(weights), ptr(add),
-         ptr(out), T, width, ff, top, stream_ptr())
+         ptr(add_weight), ptr(out), T, width, ff, top, stream_ptr())
     return out
 
 
@@ -1530,8 +1664,9 @@ def gather_rows(x: torch.Tensor, pair_at: torch.Tensor, top: int) -> torch.Tenso
     return out
 
 
-def experts_combine(y: torch.Tensor, place_of: torch.Tensor, weights: torch.Tensor, add: torch.Tensor | None) -> torch.Tensor:
-    """``add[t] + sum_k weights[t, k] * y[place_of[t, k]]`` in the order of ``k``, 32-bit ``[T, width]``."""
+def experts_combine(y: torch.Tensor, place_of: torch.Tensor, weights: torch.Tensor, add: torch.Tensor | None,
+                    add_weight: torch.Tensor | None = None) -> torch.Tensor:
+    """``add[t]`` (times ``add_weight[t]`` where given) ``+ sum_k weights[t, k] * y[place_of[t, k]]`` in the order of ``k``, 32-bit ``[T, width]``."""
     _check(y, "y", dims=2)
     _check(place_of, "place_of", torch.int32, 2)
     _check(weights, "weights", torch.float32, 2)
@@ -1539,16 +1674,16 @@ def experts_combine(y: torch.Tensor, place_of: torch.Tensor, weights: torch.Tens
     if add is not None:
         _check(add, "add", y.dtype, 2)
     out = torch.empty((T, y.shape[1]), dtype=torch.float32, device=y.device)
-    call("gk_experts_combine", ptr(y), dtype_code(y.dtype), ptr(place_of), ptr(weights), ptr(add), ptr(out), T, y.shape[1], top,
-         stream_ptr())
+    call("gk_experts_combine", ptr(y), dtype_code(y.dtype), ptr(place_of), ptr(weights), ptr(add), ptr(add_weight), ptr(out), T,
+         y.shape[1], top, stream_ptr())
     return out
 
 
 # ------------------------------------------------------------------ layer norm, scored attention, linear attention with a fixed decay
 def add_layernorm(h: torch.Tensor, delta: torch.Tensor | None, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
-                  rows: torch.Tensor | None = None, delta_scale: float = 1.0) -> torch.Tensor:
+                  rows: torch.Tensor | None = None, delta_scale: float = 1.0, bias: torch.Tensor | None = None) -> torch.Tensor:
     """``h += delta_scale * delta`` (in place, skipped when ``delta`` is None), then the layer norm of ``h`` with a weight
-    and no bias: ``(h - mean) / sqrt(mean((h - mean)^2) + eps) * weight``.  With ``rows`` (int32 indices) only those rows
+    and an optional bias: ``(h - mean) / sqrt(mean((h - mean)^2) + eps) * weight + bias``.  With ``rows`` (int32 indices) only those rows
     are normed and ``h`` is not written."""
     require_device(h.device)
     _check(h, "h", torch.float32, 2)
@@ -1556,6 +1691,10 @@ def add_layernorm(h: torch.Tensor, delta: torch.Tensor | None, weight: torch.Ten
     hidden = h.shape[1]
     if weight.shape[0] != hidden:
         raise KernelError(f"norm weight has {weight.shape[0]} entries for rows of {hidden}")
+    if bias is not None:
+        _check(bias, "bias", weight.dtype, 1)
+        if bias.shape[0] != hidden:
+            raise KernelError(f"norm bias has {bias.shape[0]} entries for rows of {hidden}")
     delta_code = 0
     if delta is not None:
         _check(delta, "delta", dims=2)
@@ -1567,9 +1706,47 @@ def add_layernorm(h: torch.Tensor, delta: torch.Tensor | None, weight: torch.Ten
         _check(rows, "rows", torch.int32, 1)
         n_out = rows.shape[0]
     out = torch.empty((n_out, hidden), dtype=out_dtype, device=h.device)
-    call("gk_add_layernorm", ptr(h), ptr(delta), delta_code, float(delta_scale), ptr(weight), dtype_code(weight.dtype), ptr(out),
+    call("gk_add_layernorm", ptr(h), ptr(delta), delta_code, float(delta_scale), ptr(weight), ptr(bias), dtype_code(weight.dtype), ptr(out),
          dtype_code(out_dtype), ptr(rows), n_out, hidden, float(eps), stream_ptr())
     return out
+
+
+def layernorm_merge(x: torch.Tensor, y: torch.Tensor | None = None, norm_y: tuple | None = None, first: torch.Tensor | None = None,
+                    step: torch.Tensor | None = None, norm_z: tuple | None = None, z_dtype: torch.dtype = torch.float32,
+                    x_out: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """The sums that stand between two sublayers and the norms around them, in one kernel: ``v = x + LN(y)`` (``norm_y =
+    (weight, bias, eps)``; without it ``y`` is added as it is, without ``y`` nothing is), ``v += first`` (a row a token), ``v +=
+    step`` (one vector for all tokens), ``x_out = v`` (a new tensor unless given; it may be ``x``), ``z = LN(v)`` in ``z_dtype`` with
+    ``norm_z`` (None: no ``z``).  Returns ``(x_out, z)``."""
+    require_device(x.device)
+    _check(x, "x", torch.float32, 2)
+    rows, width = x.shape
+    if y is not None:
+        _check(y, "y", dims=2)
+    if first is not None:
+        _check(first, "first", torch.float32, 2)
+    for name, t in (("y", y), ("first", first), ("x_out", x_out)):
+        if t is not None and t.shape != x.shape:
+            raise KernelError(f"layernorm_merge: {name} {tuple(t.shape)} for a stream {tuple(x.shape)}")
+    if step is not None:
+        _check(step, "step", torch.float32, 1)
+    for norm in (norm_y, norm_z):
+        if norm is not None:
+            _check(norm[0], "norm weight", torch.float32, 1)
+            _check(norm[1], "norm bias", torch.float32, 1)
+    for t in [step] + [t for norm in (norm_y, norm_z) if norm is not None for t in norm[:2]]:
+        if t is not None and t.shape[0] != width:
+            raise KernelError(f"layernorm_merge: a vector of {t.shape[0]} entries for rows of {width}")
+    if x_out is None:
+        x_out = torch.empty_like(x)
+    else:
+        _check(x_out, "x_out", torch.float32, 2)
+    z = None if norm_z is None else torch.empty((rows, width), dtype=z_dtype, device=x.device)
+    w_y, b_y, eps_y = norm_y or (None, None, 0.0)
+    w_z, b_z, eps_z = norm_z or (None, None, 0.0)
+    call("gk_layernorm_merge", ptr(x), ptr(y), 0 if y is None else dtype_code(y.dtype), ptr(w_y), ptr(b_y), float(eps_y), ptr(first),
+         ptr(step), ptr(x_out), ptr(w_z), ptr(b_z), float(eps_z), ptr(z), dtype_code(z_dtype), rows, width, stream_ptr())
+    return x_out, z
 
 
 def add_layernorm_conv_single_fits(hidden: int, taps: int) -> bool:
@@ -1642,7 +1819,7 @@ def relu_squared(x: torch.Tensor) -> torch.Tensor:
     return out
 
 
-PREPARE_SILU_QK, PREPARE_SILU_V, PREPARE_UNIT_RMS, PREPARE_TURN_V = 1, 2, 4, 8
+PREPARE_SILU_QK, PREPARE_SILU_V, PREPARE_UNIT_RMS, PREPARE_TURN_V, PREPARE_NEIGHBOURS = 1, 2, 4, 8, 16
 
 
 def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int, n_k: int, d: int, dv: int, tok_pos: torch.Tensor,
@@ -1650,11 +1827,12 @@ def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int,
                   cos: torch.Tensor | None = None, sin: torch.Tensor | None = None, unit_eps: float | None = None,
                   k_scale: float = 1.0, kv: PagedKV | None = None, write_kv: bool = True, max_position: int | None = None,
                   v_cos: torch.Tensor | None = None, v_sin: torch.Tensor | None = None, w_q: torch.Tensor | None = None,
-                  w_k: torch.Tensor | None = None):
+                  w_k: torch.Tensor | None = None, bias: torch.Tensor | None = None, bias_at: int = 0, neighbours: bool = False):
     """What stands between a packed projection and a mixer's core.  ``proj [T, >= ...]`` holds ``n_q`` query heads of ``d``
     from column ``q_at``, ``n_k`` key heads of ``d`` from ``k_at`` and ``n_k`` value heads of ``dv`` from ``v_at``.  In this
-    order: SiLU (``silu_qk`` on q and k, ``silu_v`` on v); rotation of the first ``rot`` entries of every q and k head by
-    the token's position (entry ``i`` with ``i + rot/2``; ``cos``, ``sin`` ``[positions, rot/2]``); with ``unit_eps`` every q
+    order: ``bias`` (a number for every column from ``bias_at`` on); SiLU (``silu_qk`` on q and k, ``silu_v`` on v); rotation of the
+    first ``rot`` entries of every q and k head by the token's position (entry ``i`` with ``i + rot/2``, or ``2i`` with ``2i + 1``
+    where ``neighbours``; ``cos``, ``sin`` ``[positions, rot/2]``); with ``unit_eps`` every q
     and k head divided by its root mean square (and multiplied by ``w_q [d]`` or ``w_k [d]`` where given); ``k_scale`` on k; with ``v_cos``, ``v_sin`` ``[positions, dv/2]`` every
     value head turned by its token's position over all of its entries (entry ``m`` with ``m + dv/2``).  With ``kv`` the keys and values are written into the
     cache's pages and q ``[T, n_q, d]`` comes back in the projection's type; without, q, k ``[T, n, d]`` and v ``[T, n_k,
@@ -1679,7 +1857,12 @@ def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int,
             _check(t, name, torch.float32, 1)
             if t.shape[0] != d or unit_eps is None:
                 raise KernelError(f"heads_prepare: {name} has {t.shape[0]} entries for the norm of heads of {d}")
-    flags = (PREPARE_SILU_QK if silu_qk else 0) | (PREPARE_SILU_V if silu_v else 0) | (PREPARE_UNIT_RMS if unit_eps is not None else 0)
+    if bias is not None:
+        _check(bias, "bias", torch.float32, 1)
+        columns = max(q_at + n_q * d, (k_at + n_k * d) if reads_kv else 0, (v_at + n_k * dv) if reads_kv else 0)
+        if bias_at > min([q_at] + ([k_at, v_at] if reads_kv else [])) or bias.shape[0] < columns - bias_at:
+            raise KernelError(f"heads_prepare: {bias.shape[0]} biases from column {bias_at} on do not cover these heads")
+    flags = (PREPARE_NEIGHBOURS if neighbours else 0) | (PREPARE_SILU_QK if silu_qk else 0) | (PREPARE_SILU_V if silu_v else 0) | (PREPARE_UNIT_RMS if unit_eps is not None else 0)
     if v_cos is not None:
         _check(v_cos, "v_cos", torch.float32, 2)
         _check(v_sin, "v_sin", torch.float32, 2)
@@ -1695,7 +1878,7 @@ def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int,
         if tuple(kv.k.shape[1:]) != (n_k, kv.page_size, d) or tuple(kv.v.shape[1:]) != (n_k, kv.page_size, dv):
             raise KernelError(f"heads_prepare: pages {tuple(kv.k.shape)} / {tuple(kv.v.shape)} do not hold {n_k} heads of {d} / {dv}")
         q = torch.empty((T, n_q, d), dtype=proj.dtype, device=dev)
-        call("gk_heads_prepare", ptr(proj), dtype_code(proj.dtype), proj.shape[1], q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot,
+        call("gk_heads_prepare", ptr(proj), dtype_code(proj.dtype), ptr(bias), int(bias_at), proj.shape[1], q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot,
              ptr(cos) if rot else None, ptr(sin) if rot else None, ptr(v_cos), ptr(v_sin), float(unit_eps or 0.0), ptr(w_q), ptr(w_k), float(k_scale),
              ptr(tok_pos), ptr(tok_seq), ptr(slots), ptr(q), dtype_code(q.dtype), None, None, ptr(kv.k), ptr(kv.v), ptr(kv.block_table), kv.max_pages,
              kv.page_size, int(write_kv), T, stream_ptr())
@@ -1703,7 +1886,7 @@ def heads_prepare(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, n_q: int,
     q = torch.empty((T, n_q, d), dtype=torch.float32, device=dev)
     k = torch.empty((T, n_k, d), dtype=torch.float32, device=dev)
     v = torch.empty((T, n_k, dv), dtype=torch.float32, device=dev)
-    call("gk_heads_prepare", ptr(proj), dtype_code(proj.dtype), proj.shape[1], q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot,
+    call("gk_heads_prepare", ptr(proj), dtype_code(proj.dtype), ptr(bias), int(bias_at), proj.shape[1], q_at, k_at, v_at, n_q, n_k, d, dv, flags, rot,
          ptr(cos) if rot else None, ptr(sin) if rot else None, ptr(v_cos), ptr(v_sin), float(unit_eps or 0.0), ptr(w_q), ptr(w_k), float(k_scale),
          ptr(tok_pos), ptr(tok_seq), ptr(slots), ptr(q), dtype_code(q.dtype), ptr(k), ptr(v), None, None, None, 0, 0, 0, T, stream_ptr())
     return q, k, v
@@ -1764,11 +1947,13 @@ def decay_scan_chunked(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay:
 
 
 def group_norm_gate(x: torch.Tensor, group: int, weight: torch.Tensor | None, gate: torch.Tensor, gate_at: int, eps: float,
-                    out_dtype: torch.dtype, gate_kind: str = "sigmoid", divisor: torch.Tensor | None = None) -> torch.Tensor:
+                    out_dtype: torch.dtype, gate_kind: str = "sigmoid", divisor: torch.Tensor | None = None,
+                    out: torch.Tensor | None = None, out_at: int = 0, out_scale: float = 1.0) -> torch.Tensor:
     """Rows of ``x [T, width]`` (32-bit) cut into groups of ``group`` entries; every group divided by its root mean square
     (eps inside the root), multiplied by ``weight`` (if given: ``[group]`` for every group alike, or ``[width]``) and by sigmoid or
     SiLU of ``gate[:, gate_at : gate_at + width]``.  ``divisor [T, width / group]``: every group is divided by its own number
-    before its norm.  Returns ``[T, width]`` in ``out_dtype``."""
+    before its norm.  Returns ``[T, width]`` in ``out_dtype``, or writes columns ``out_at ..`` of ``out [T, ...]``; the result is
+    multiplied by ``out_scale``."""
     require_device(x.device)
     _check(x, "x", torch.float32, 2)
     _check(gate, "gate", dims=2)
@@ -1784,9 +1969,22 @@ def group_norm_gate(x: torch.Tensor, group: int, weight: torch.Tensor | None, ga
         if tuple(divisor.shape) != (T, width // group):
             raise KernelError(f"group_norm_gate: divisors {tuple(divisor.shape)} for {width // group} groups a row")
     kinds = {"sigmoid": 0, "silu": 1}
-    out = torch.empty((T, width), dtype=out_dtype, device=x.device)
+    out = _read_out_rows(out, out_at, T, width, out_dtype, x.device)
     call("gk_group_norm_gate", ptr(x), ptr(divisor), ptr(weight), int(weight is not None and weight.shape[0] == width), gate.data_ptr() + gate_at * gate.element_size(), dtype_code(gate.dtype),
-         gate.shape[1], ptr(out), dtype_code(out_dtype), T, width // group, group, float(eps), kinds[gate_kind], stream_ptr())
+         gate.shape[1], out.data_ptr() + out_at * out.element_size(), out.shape[1], float(out_scale), dtype_code(out_dtype), T, width // group,
+         group, float(eps), kinds[gate_kind], stream_ptr())
+    return out
+
+
+def _read_out_rows(out: torch.Tensor | None, out_at: int, rows: int, width: int, dtype: torch.dtype, device) -> torch.Tensor:
+    """``out``, checked to have room for ``width`` columns from ``out_at`` on, or a new ``[rows, width]``."""
+    if out is None:
+        if out_at:
+            raise KernelError("a first column belongs to a given output")
+        return torch.empty((rows, width), dtype=dtype, device=device)
+    _check(out, "out", dtype, 2)
+    if out.shape[0] != rows or out.shape[1] < out_at + width:
+        raise KernelError(f"results of {width} columns do not fit {tuple(out.shape)} from column {out_at}")
     return out
 
 
@@ -1795,14 +1993,15 @@ def attention_scored_exact(q: torch.Tensor, kv: PagedKV, tok_pos: torch.Tensor, 
                            r2: torch.Tensor | None = None, head_bias: torch.Tensor | None = None,
                            weights: str = "softmax", chunk: int = 0, temp: torch.Tensor | None = None,
                            dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None,
-                           softcap: float = 0.0) -> torch.Tensor:
+                           softcap: float = 0.0, out: torch.Tensor | None = None, out_at: int = 0, out_scale: float = 1.0) -> torch.Tensor:
     """Causal grouped-query attention of ``q [T, n_q, d]`` over pages of keys ``[.., d]`` and values ``[.., dv]`` (exact
     kernel): a key at ``j`` is seen from ``i`` if ``i - j < window`` or ``j < keep_first``; the score is ``q . k * scale -
     r1_h ln(1 + r2_h (i - j))``; the weights are the softmax over the seen keys, or ``sigmoid(score + head_bias_h)``
     without a sum that divides.  ``chunk``: only keys of the token's own chunk of that many positions are seen; ``temp``
     ``[n_q]`` multiplies the product per head; ``dist_bias [n_dist, n_q]`` is added by distance (the last row for
     every distance beyond); ``sink [n_q]`` joins the softmax's denominator as ``exp(sink_h)``; ``softcap > 0``: the product
-    becomes ``softcap * tanh(product / softcap)`` before any distance term.  Returns ``[T, n_q, dv]``."""
+    becomes ``softcap * tanh(product / softcap)`` before any distance term.  Returns ``[T, n_q, dv]``, or writes the read-outs
+    into columns ``out_at ..`` of ``out [T, ...]`` and returns that; ``out_scale`` multiplies them."""
     require_device(q.device)
     _check(q, "q", dims=3)
     n, n_q, d = q.shape
@@ -1819,12 +2018,12 @@ def attention_scored_exact(q: torch.Tensor, kv: PagedKV, tok_pos: torch.Tensor, 
             _check(t, name, torch.float32, 1)
             if t.shape[0] != n_q:
                 raise KernelError(f"{name} has {t.shape[0]} entries for {n_q} query heads")
-    out = torch.empty((n, n_q, dv), dtype=q.dtype, device=q.device)
-    call("gk_attention_scored_exact", ptr(q), ptr(kv.k), ptr(kv.v), ptr(out), dtype_code(q.dtype), ptr(tok_pos), ptr(tok_seq),
+    rows = _read_out_rows(out, out_at, n, n_q * dv, q.dtype, q.device)
+    call("gk_attention_scored_exact", ptr(q), ptr(kv.k), ptr(kv.v), rows.data_ptr() + out_at * rows.element_size(), dtype_code(q.dtype), ptr(tok_pos), ptr(tok_seq),
          ptr(slots), ptr(kv.block_table), n, n_q, n_kv, d, dv, kv.max_pages, kv.page_size, float(scale), int(window),
          int(keep_first), ptr(r1), ptr(r2), ptr(head_bias), {"softmax": 0, "sigmoid": 1}[weights], int(chunk), ptr(temp),
-         ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], ptr(sink), float(softcap), stream_ptr())
-    return out
+         ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], ptr(sink), float(softcap), rows.shape[1], float(out_scale), stream_ptr())
+    return rows.view(n, n_q, dv) if out is None else out
 
 
 def _check_score_rules(n_q: int, temp, dist_bias, sink) -> None:
@@ -1853,12 +2052,21 @@ def scored_attention_parts(n_seqs: int, n_q: int, n_kv: int, max_q_len: int, vis
     return max(1, min(wanted, visible_pages, 32))
 
 
+def attention_scored_fits(d: int, dv: int, softcap: float = 0.0) -> bool:
+    """Whether :func:`attention_scored` takes keys of ``d`` and values of ``dv`` entries: 64 or 128 both, or (without a cap)
+    multiples of 8 up to 128 and 256, which it pads in shared memory."""
+    if d == dv and d in (64, 128):
+        return True
+    return 0 < d <= 128 and d % 8 == 0 and 0 < dv <= 256 and dv % 8 == 0 and not softcap
+
+
 def attention_scored(q: torch.Tensor, kv: PagedKV, cu_q: torch.Tensor, kv_len: torch.Tensor, slots: torch.Tensor, max_q_len: int,
                      scale: float, window: int = 0, keep_first: int = 0, r1: torch.Tensor | None = None,
                      r2: torch.Tensor | None = None, head_bias: torch.Tensor | None = None, weights: str = "softmax",
                      n_parts: int = 1, chunk: int = 0, temp: torch.Tensor | None = None, dist_bias: torch.Tensor | None = None,
-                     sink: torch.Tensor | None = None, softcap: float = 0.0) -> torch.Tensor:
-    """:func:`attention_scored_exact` on the tensor cores: bfloat16, keys and values of 64 or 128 entries both, pages of 64
+                     sink: torch.Tensor | None = None, softcap: float = 0.0, out: torch.Tensor | None = None, out_at: int = 0,
+                     out_scale: float = 1.0) -> torch.Tensor:
+    """:func:`attention_scored_exact` on the tensor cores: bfloat16, sizes for which :func:`attention_scored_fits`, pages of 64
     keys.  The new tokens ``q [n_tokens, n_q, d]`` are packed by sequence (``cu_q``), ``kv_len`` counts each sequence's
     cached tokens including them.  ``n_parts`` > 1 cuts every block's keys into that many blocks whose sums a second
     kernel adds (steps of few tokens)."""
@@ -1867,8 +2075,9 @@ def attention_scored(q: torch.Tensor, kv: PagedKV, cu_q: torch.Tensor, kv_len: t
     n, n_q, d = q.shape
     _check(kv.k, "k pages", torch.bfloat16, 4)
     _check(kv.v, "v pages", torch.bfloat16, 4)
-    if kv.k.shape[3] != d or kv.v.shape[3] != d:
-        raise KernelError(f"attention_scored: pages of {kv.k.shape[3]} / {kv.v.shape[3]} for queries of {d} (use the exact kernel)")
+    dv = kv.v.shape[3]
+    if kv.k.shape[3] != d or not attention_scored_fits(d, dv, softcap):
+        raise KernelError(f"attention_scored: pages of {kv.k.shape[3]} / {dv} for queries of {d} (use the exact kernel)")
     for name, t in (("cu_q", cu_q), ("kv_len", kv_len), ("slots", slots)):
         _check(t, name, torch.int32, 1)
     n_seqs = kv_len.shape[0]
@@ -1881,17 +2090,18 @@ def attention_scored(q: torch.Tensor, kv: PagedKV, cu_q: torch.Tensor, kv_len: t
                 raise KernelError(f"{name} has {t.shape[0]} entries for {n_q} query heads")
     _check_score_rules(n_q, temp, dist_bias, sink)
     sigmoid = {"softmax": 0, "sigmoid": 1}[weights]
-    out = torch.empty_like(q)
+    rows = _read_out_rows(out, out_at, n, n_q * dv, q.dtype, q.device)
     part_o = part_ml = None
     if n_parts > 1:
-        part_o = torch.empty((n_parts, n, n_q, d), dtype=torch.float32, device=q.device)
+        part_o = torch.empty((n_parts, n, n_q, dv), dtype=torch.float32, device=q.device)
         if not sigmoid:
             part_ml = torch.empty((n_parts, n, n_q, 2), dtype=torch.float32, device=q.device)
-    call("gk_attention_scored_bf16", ptr(q), ptr(kv.k), ptr(kv.v), ptr(out), ptr(part_o), ptr(part_ml), ptr(cu_q), ptr(kv_len),
-         ptr(slots), ptr(kv.block_table), n_seqs, int(max_q_len), n, n_q, kv.k.shape[1], d, kv.max_pages, kv.page_size, float(scale),
+    call("gk_attention_scored_bf16", ptr(q), ptr(kv.k), ptr(kv.v), rows.data_ptr() + out_at * rows.element_size(), ptr(part_o), ptr(part_ml), ptr(cu_q), ptr(kv_len),
+         ptr(slots), ptr(kv.block_table), n_seqs, int(max_q_len), n, n_q, kv.k.shape[1], d, dv, kv.max_pages, kv.page_size, float(scale),
          int(window), int(keep_first), ptr(r1), ptr(r2), ptr(head_bias), sigmoid, int(n_parts), int(chunk), ptr(temp),
-         ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], ptr(sink), float(softcap), stream_ptr())
-    return out
+         ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], ptr(sink), float(softcap), rows.shape[1], float(out_scale),
+         stream_ptr())
+    return rows.view(n, n_q, dv) if out is None else out
 
 
 # ------------------------------------------------------------------ gated branches, PolyNorm, matrix memory

@@ -68,36 +68,41 @@ _SIGNATURES: dict[str, list] = {
     "gk_sample": [P, L, I, I, F, I, U, P, P, I, P, I, P, P],
     "gk_delta_prepare": [P, I, L, P, I, L, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
     "gk_conv_roll": [P, I, L, P, P, P, I, I, I, P],
-    "gk_delta_scan": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
+    "gk_delta_scan": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
+    "gk_delta_head_prepare": [P, I, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
+    "gk_conv_ring": [P, I, L, P, P, P, P, I, I, I, P],
+    "gk_delta_head_single": [P, I, L, P, P, P, P, P, P, P, P, P, P, L, F, F, I, I, I, I, I, I, P],
+    "gk_delta_head_single_fits": [I, I],
     "gk_head_norm_gate": [P, P, P, I, L, P, I, L, I, I, F, P],
-    "gk_route_groups": [P, I, P, P, P, P, P, I, I, I, I, I, I, F, I, P],
+    "gk_route_groups": [P, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P, P],
     "gk_experts_up": [P, I, P, I, P, P, I, I, I, I, P],
-    "gk_experts_down": [P, I, P, I, P, P, P, P, I, I, I, I, P],
+    "gk_experts_down": [P, I, P, I, P, P, P, P, P, I, I, I, I, P],
     "gk_experts_sort": [P, I, I, P, P, P, P],
     "gk_gather_rows": [P, I, P, P, I, I, I, P],
-    "gk_experts_combine": [P, I, P, P, P, P, I, I, I, P],
+    "gk_experts_combine": [P, I, P, P, P, P, P, I, I, I, P],
     "gk_wide_norm_rope_write": [P, I, L, P, P, P, P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, I, P],
     "gk_turn_back_gate": [P, P, P, I, I, P, P, L, P, I, L, I, I, P],
     "gk_xielu": [P, P, I, L, F, F, P],
     "gk_stream_cast": [P, P, I, L, P],
     "gk_sigmoid_gate": [P, P, L, P, I, L, I, P],
     "gk_softcap": [P, L, F, P],
-    "gk_add_layernorm": [P, P, I, F, P, I, P, I, P, I, I, F, P],
+    "gk_add_layernorm": [P, P, I, F, P, P, I, P, I, P, I, I, F, P],
+    "gk_layernorm_merge": [P, P, I, P, P, F, P, P, P, P, P, F, P, I, I, I, P],
     "gk_add_layernorm_conv_single": [P, P, I, F, P, P, P, P, P, P, P, I, I, I, I, F, I, P],
     "gk_scaled_sum": [P, F, P, F, I, P, L, P],
     "gk_relu_squared": [P, P, I, L, P],
     "gk_scale": [P, L, F, P],
-    "gk_heads_prepare": [P, I, L, I, I, I, I, I, I, I, I, I, P, P, P, P, F, P, P, F, P, P, P, P, I, P, P, P, P, P, I, I, I, I, P],
+    "gk_heads_prepare": [P, I, P, I, L, I, I, I, I, I, I, I, I, I, P, P, P, P, F, P, P, F, P, P, P, P, I, P, P, P, P, P, I, I, I, I, P],
     "gk_decay_scan": [P, P, P, P, P, P, P, P, I, I, I, I, P],
     "gk_decay_scan_chunked": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
-    "gk_group_norm_gate": [P, P, P, I, P, I, L, P, I, L, I, I, F, I, P],
-    "gk_attention_scored_exact": [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, P, P, I, P, F, P],
+    "gk_group_norm_gate": [P, P, P, I, P, I, L, P, L, F, I, L, I, I, F, I, P],
+    "gk_attention_scored_exact": [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, P, P, I, P, F, L, F, P],
     "gk_gated_merge": [P, I, P, L, P, P, I, P, P, F, F, P, P, P, F, F, F, I, I, P],
     "gk_poly_norm": [P, I, P, I, I, I, F, F, F, F, F, P],
     "gk_memory_single": [P, L, I, I, I, I, I, I, P, F, P, P, P, F, P, P, P, I, I, I, I, P],
     "gk_memory_chunked": [P, L, I, I, I, I, I, I, P, F, P, P, P, F, P, P, P, P, P, P, I, I, I, I, I, I, P],
     "gk_memory_scan": [P, I, L, I, I, I, I, I, P, F, P, P, P, P, P, P, P, I, I, I, I, P],
-    "gk_attention_scored_bf16": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, I, P, P, I, P, F, P],
+    "gk_attention_scored_bf16": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, I, P, P, I, P, F, L, F, P],
 }
 
 

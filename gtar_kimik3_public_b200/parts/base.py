@@ -148,6 +148,24 @@ class Mixer(Part):
         raise NotImplementedError
 
 
+class ProjectedMixer(Mixer):
+    """A mixer of one packed input product, a core that turns a row's columns into read-outs, and one output product.  What
+    stands around it may make both products for several such mixers at once (``side_by_side`` does)."""
+
+    w_in: torch.Tensor | None = None  # [columns, hidden], rows padded to a multiple of 8
+    w_o: torch.Tensor | None = None  # [hidden, out_columns]
+    packable = True  # whether ``core`` takes columns and leaves read-outs anywhere in wider rows
+
+    @property
+    def out_columns(self) -> int:
+        raise NotImplementedError
+
+    def core(self, proj: torch.Tensor, at: int, ctx: StepContext, cache: Any, out: torch.Tensor, out_at: int, out_scale: float) -> None:
+        """The mixer's columns begin at ``at`` in the rows of ``proj``; its read-outs, times ``out_scale``, go to the columns
+        ``out_at ..`` of ``out``."""
+        raise NotImplementedError
+
+
 class FeedForward(Part):
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
@@ -172,6 +190,10 @@ class Block(Part):
         return bool(parts) and all(part.graph_safe for _, part in parts)
 
     mixer: Mixer
+
+    # Whether the block itself adds what stands at its entry of the run list (``ctx.extras["enter"]``) and forms the rows that
+    # the next entry's block reads (``ctx.extras["follower"]``); for other blocks the model does the adds.
+    hands_on = False
 
     def forward(self, h: torch.Tensor, pending: torch.Tensor | None, ctx: StepContext,
                 cache: Any) -> tuple[torch.Tensor, torch.Tensor | None]:

@@ -2,7 +2,8 @@
 (src/models/transformer.py:47-48).  The adds are fused into the norm that follows them: the
 block hands its last branch output on as ``pending`` instead of adding it itself.  Beside it: the block with
 convolutions over time in front of its sublayers, the block whose branches share one norm, the block whose two gated branches
-have norms of their own, the block that norms every branch on both sides, and the block that norms every branch on its way OUT only."""
+have norms of their own, the block that norms every branch on both sides (with a convolution and the depth mix), the block that
+norms every branch on its way OUT only, and the block with a layer norm on both sides of every branch."""
 
 from __future__ import annotations
 
@@ -165,7 +166,7 @@ class ConvPreNormBlock(Block):
     def _normed_through_conv(self, norm, h, pending, weight, state, ctx: StepContext):
         """``norm(h + pending)`` through the convolution; one kernel where every sequence brings one token and the norm has
         that form, else the norm's kernel and the convolution's."""
-        if ctx.all_single and hasattr(norm, "forward_conv_single") and F.add_layernorm_conv_single_fits(h.shape[1], weight.shape[0]):
+        if ctx.all_single and hasattr(norm, "forward_conv_single") and getattr(norm, "bias", None) is None and F.add_layernorm_conv_single_fits(h.shape[1], weight.shape[0]):
             keep = state is not None and not ctx.extras.get("cache_read_only", False)
             return norm.forward_conv_single(h, pending, weight, state, ctx, keep)
         return self._through_conv(norm.forward(h, pending, torch.float32), weight, state, ctx)
@@ -517,3 +518,73 @@ class OutNormBlock(Block):
 
 
 register_part("block", "out_norm", OutNormBlock)
+
+
+class LayerNormBothSidesBlock(Block):
+    """A layer with a layer norm (weight and bias) before and after each of its branches:
+
+        x += norm_1b(mixer(norm_1(x)));   x += norm_2b(feed_forward(norm_2(x)))      (the second left out without feed-forward)
+
+    A branch's second norm, its add into the 32-bit stream and the norm of what reads the stream next are one kernel
+    (``layernorm_merge``).  What reads next may be the following entry of the run list (``follower``, given by the model): its
+    first norm, and whatever is added to the stream in front of it, are then formed here; only a block that nothing handed its
+    rows forms them with a launch of its own."""
+
+    hands_on = True
+
+    def __init__(self, norm_1: Norm, mixer: Mixer, norm_1b: Norm, norm_2: Norm | None, feed_forward: FeedForward | None,
+                 norm_2b: Norm | None, names: dict[str, str] | None = None, unused: tuple[Norm, ...] = ()):
+        """``unused``: norms whose tensors a file may carry although no branch reads them (a layer without feed-forward)."""
+        if (feed_forward is None) != (norm_2 is None) or (feed_forward is None) != (norm_2b is None):
+            raise ValueError("a feed-forward comes with the norms before and after it, or not at all")
+        self.norm_1, self.mixer, self.norm_1b = norm_1, mixer, norm_1b
+        self.norm_2, self.feed_forward, self.norm_2b = norm_2, feed_forward, norm_2b
+        self.unused = tuple(unused)
+        self.names = {"mixer": "mix.", "feed_forward": "mlp.", **(names or {})}
+
+    def children(self):
+        parts = [("", self.norm_1), (self.names["mixer"], self.mixer), ("", self.norm_1b)]
+        if self.feed_forward is not None:
+            parts += [("", self.norm_2), (self.names["feed_forward"], self.feed_forward), ("", self.norm_2b)]
+        return parts
+
+    def tensor_specs(self):
+        from dataclasses import replace
+
+        specs = {prefix + name: spec for prefix, part in self.children() for name, spec in part.tensor_specs().items()}
+        for part in self.unused:
+            specs.update({name: replace(spec, optional=True) for name, spec in part.tensor_specs().items()})
+        return specs
+
+    def load(self, tensors):
+        for prefix, part in self.children():
+            part.load({name: tensors[prefix + name] for name in part.tensor_specs() if prefix + name in tensors})
+
+    def weight_bytes(self):
+        return sum(part.weight_bytes() for _, part in self.children())
+
+    def forward(self, h, pending, ctx: StepContext, cache):
+        stream = ctx.extras.get("stream")
+        out = h if stream is None else stream
+        z = ctx.extras.pop("normed_rows", None)
+        if z is None:
+            first, step = ctx.extras.get("enter") or (None, None)
+            _, z = F.layernorm_merge(h, pending, first=first, step=step, norm_z=self.norm_1.rule(), z_dtype=ctx.dtype, x_out=out)
+            h = out
+        branch, norm = self.mixer.forward(z, ctx, cache), self.norm_1b
+        if self.feed_forward is not None:
+            _, z = F.layernorm_merge(h, branch, norm.rule(), norm_z=self.norm_2.rule(), z_dtype=ctx.dtype, x_out=out)
+            h = out
+            branch, norm = self.feed_forward.forward(z, ctx), self.norm_2b
+        follower = ctx.extras.get("follower")
+        if follower is None:
+            F.layernorm_merge(h, branch, norm.rule(), x_out=out)
+        else:
+            block, enter = follower
+            first, step = enter or (None, None)
+            _, z = F.layernorm_merge(h, branch, norm.rule(), first=first, step=step, norm_z=block.norm_1.rule(), z_dtype=ctx.dtype, x_out=out)
+            ctx.extras["normed_rows"] = z
+        return out, None
+
+
+register_part("block", "layernorm_both_sides", LayerNormBothSidesBlock)

@@ -1,4 +1,6 @@
-"""A recurrent mixer: the gated delta rule with a decay per head and key channel.
+"""Recurrent mixers: the gated delta rule with a decay per head and key channel, and the one with a decay per head.
+
+The first, ``channel_delta``:
 
 Per head a state ``S [d, dv]`` of 32-bit floats, zero at the start of a sequence, is carried from token to token:
 
@@ -18,6 +20,12 @@ A step's kernels: the packed projection q | k | v | b; the packed first halves o
 for their second halves (a block-diagonal matrix); one kernel for convolutions, activations, unit lengths, decays and
 beta; one that moves the convolution state on; the recurrence; norm and gate; the output projection.  Prompts,
 portions of prompts and single tokens take the same path.
+
+The second, ``head_delta``, has one decay number per head, ``g_t = exp(-exp(A_h) * softplus(W_a x + dt_bias_h))``, and its gate is
+``silu(W_g x)``; everything else is as above.  All of its input projections are one packed product q | k | v | b | a | gate.  A
+step of one token a sequence is one kernel between the two products; steps of more tokens prepare their vectors, move the
+convolution's ring on, run the recurrence (in chunks on the tensor cores for bfloat16, token by token in 32-bit runs and for
+head sizes that the chunks do not take) and norm and gate the read-outs.
 """
 
 from __future__ import annotations
@@ -26,7 +34,7 @@ import torch
 
 from ..ops import functional as F
 from ..ops.linear import linear
-from .base import Mixer, StateRequest, StepContext, TensorSpec, register_part
+from .base import Mixer, ProjectedMixer, StateRequest, StepContext, TensorSpec, register_part
 
 _NAMES = {"q": "q", "k": "k", "v": "v", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "b": "b", "a_log": "A_log",
           "norm": "norm", "a1": "a1", "a2": "a2", "dt_bias": "dt_bias", "g1": "g1", "g2": "g2", "o": "o"}
@@ -121,3 +129,88 @@ class ChannelDeltaRule(Mixer):
 
 
 register_part("mixer", "channel_delta", ChannelDeltaRule)
+
+
+_HEAD_NAMES = {"q": "q", "k": "k", "v": "v", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "b": "b", "a": "a",
+               "a_log": "A_log", "dt_bias": "dt_bias", "norm": "norm", "g": "g", "o": "o"}
+
+
+class HeadDeltaRule(ProjectedMixer):
+    graph_safe = True
+
+    def __init__(self, hidden_size: int, n_heads: int, n_kv_heads: int, key_dim: int, value_dim: int, conv_taps: int,
+                 norm_eps: float, names: dict[str, str] | None = None):
+        if n_heads % n_kv_heads:
+            raise ValueError("value heads must be a multiple of key heads")
+        self.hidden_size, self.norm_eps = int(hidden_size), float(norm_eps)
+        self.heads = F.DeltaHeads(int(n_heads), int(n_kv_heads), int(key_dim), int(value_dim), int(conv_taps))
+        if min(self.hidden_size, n_heads, n_kv_heads, key_dim, value_dim, conv_taps) <= 0:
+            raise ValueError("delta rule sizes must be positive")
+        self.names = {**_HEAD_NAMES, **(names or {})}
+        self.w_in = self.w_o = self.conv_w = self.a_log = self.dt_bias = self.norm_w = None
+
+    def tensor_specs(self):
+        n, W, hd = self.names, self.hidden_size, self.heads
+        H, G, d, dv, conv = hd.n_heads, hd.n_kv, hd.d, hd.dv, (0.0, 0.4)
+        return {
+            n["q"]: TensorSpec((G * d, W)), n["q_conv"]: TensorSpec((G * d, hd.taps), init=conv),
+            n["k"]: TensorSpec((G * d, W)), n["k_conv"]: TensorSpec((G * d, hd.taps), init=conv),
+            n["v"]: TensorSpec((H * dv, W)), n["v_conv"]: TensorSpec((H * dv, hd.taps), init=conv),
+            n["b"]: TensorSpec((H, W)),
+            n["a_log"]: TensorSpec((H,), "vector", init=(-1.0, 0.7)),
+            n["norm"]: TensorSpec((dv,), "vector"),
+            n["a"]: TensorSpec((H, W)),
+            n["dt_bias"]: TensorSpec((H,), "vector", init=(-1.0, 1.0)),
+            n["g"]: TensorSpec((H * dv, W)),
+            n["o"]: TensorSpec((W, H * dv)),
+        }
+
+    def load(self, tensors):
+        get = lambda key: tensors[self.names[key]]
+        mats = [get(key) for key in ("q", "k", "v", "b", "a", "g")]
+        if len({m.dtype for m in mats}) != 1:
+            mats = [m.float() for m in mats]
+        self.w_in = _pad_rows(torch.cat(mats, dim=0)).contiguous()
+        self.w_o = get("o").contiguous()
+        # [taps, channels]: the kernels read tap by tap
+        self.conv_w = torch.cat([get("q_conv"), get("k_conv"), get("v_conv")], dim=0).float().t().contiguous()
+        self.a_log, self.dt_bias, self.norm_w = (get(k).float().contiguous() for k in ("a_log", "dt_bias", "norm"))
+
+    def weight_bytes(self):
+        return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o, self.conv_w) if t is not None)
+
+    def cache_request(self):
+        requests = [StateRequest(self.heads.state_shape(), torch.float32)]
+        if self.heads.taps > 1:
+            requests.append(StateRequest(self.heads.ring_shape(), torch.float32))
+        return requests
+
+    @property
+    def out_columns(self) -> int:
+        return self.heads.n_heads * self.heads.dv
+
+    def core(self, proj, at: int, ctx: StepContext, cache, out, out_at: int, out_scale: float) -> None:
+        if ctx.extras.get("cache_read_only", False):
+            raise ValueError("a recurrent mixer advances its state at every step: it cannot run on another entry's storage")
+        hd, state = self.heads, cache[0]
+        ring = cache[1] if hd.taps > 1 else None
+        if ctx.all_single and F.delta_head_single_fits(hd.d, hd.dv):
+            F.delta_head_single(proj, at, hd, self.conv_w, ring, self.a_log, self.dt_bias, self.norm_w, state, ctx.tok_pos, ctx.tok_seq,
+                                ctx.slots, self.norm_eps, out, out_at, out_scale)
+            return
+        chunked = False
+        x = F.delta_head_prepare(proj, at, hd, self.conv_w, ring, self.a_log, self.dt_bias, ctx.tok_pos, ctx.tok_seq, ctx.cu_q, ctx.slots,
+                                 rounded=chunked)
+        if ring is not None:
+            F.conv_ring(proj, at, hd, ring, ctx.cu_q, ctx.kv_len, ctx.slots)
+        o = F.delta_scan(x.q, x.k, x.v, x.g, x.beta, state, ctx.cu_q, ctx.slots, ctx.n_seqs)
+        F.group_norm_gate(o.view(ctx.n_tokens, -1), hd.dv, self.norm_w, proj, at + hd.gate_at, self.norm_eps, ctx.dtype, "silu", out=out,
+                          out_at=out_at, out_scale=out_scale)
+
+    def forward(self, x, ctx: StepContext, cache) -> torch.Tensor:
+        out = torch.empty((ctx.n_tokens, self.out_columns), dtype=ctx.dtype, device=x.device)
+        self.core(linear(x, self.w_in), 0, ctx, cache, out, 0, 1.0)
+        return linear(out, self.w_o)
+
+
+register_part("mixer", "head_delta", HeadDeltaRule)

@@ -15,24 +15,22 @@ from .base import FeedForward, StepContext, TensorSpec, register_part
 class SwiGLUFeedForward(FeedForward):
     graph_safe = True
 
-    def __init__(self, hidden_size: int, intermediate_size: int):
+    def __init__(self, hidden_size: int, intermediate_size: int, gate_name: str = "gate_proj.weight", up_name: str = "up_proj.weight",
+                 down_name: str = "down_proj.weight"):
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.gate_name, self.up_name, self.down_name = gate_name, up_name, down_name
         self.w_gate_up = self.w_down = None
 
     def tensor_specs(self):
         h, i = self.hidden_size, self.intermediate_size
-        return {
-            "gate_proj.weight": TensorSpec((i, h)),
-            "up_proj.weight": TensorSpec((i, h)),
-            "down_proj.weight": TensorSpec((h, i)),
-        }
+        return {self.gate_name: TensorSpec((i, h)), self.up_name: TensorSpec((i, h)), self.down_name: TensorSpec((h, i))}
 
     def load(self, tensors):
-        gate, up = tensors["gate_proj.weight"], tensors["up_proj.weight"]
+        gate, up = tensors[self.gate_name], tensors[self.up_name]
         if gate.dtype != up.dtype:
             gate, up = gate.float(), up.float()
         self.w_gate_up = torch.stack([gate, up], dim=1).reshape(2 * gate.shape[0], gate.shape[1]).contiguous()
-        self.w_down = tensors["down_proj.weight"].contiguous()
+        self.w_down = tensors[self.down_name].contiguous()
 
     def weight_bytes(self):
         return sum(t.numel() * t.element_size() for t in (self.w_gate_up, self.w_down))

@@ -1,6 +1,6 @@
 """The norms that read the residual stream, each fused with the add of a pending branch output into it: RMSNorm,
-``weight * (x * rsqrt(mean(x^2) + eps))`` in 32-bit (src/layers/rmsnorm.py:11-16), and layer norm with a weight and no
-bias."""
+``weight * (x * rsqrt(mean(x^2) + eps))`` in 32-bit (src/layers/rmsnorm.py:11-16), and layer norm with a weight and an
+optional bias."""
 
 from __future__ import annotations
 
@@ -77,30 +77,43 @@ register_part("norm", "rmsnorm_scalar", ScalarRMSNorm)
 
 
 class LayerNorm(Norm):
-    """Layer norm with a weight and no bias, ``(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight`` in 32-bit, fused with
-    the add of a pending branch output into the stream; ``delta_scale`` multiplies that branch as it is added (a model
+    """Layer norm with a weight, ``(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight`` in 32-bit (plus a bias where
+    ``bias_name`` names its tensor), fused with the add of a pending branch output into the stream; ``delta_scale`` multiplies that branch as it is added (a model
     that scales every branch by one constant gives it to all its norms)."""
 
     graph_safe = True
 
-    def __init__(self, size: int, eps: float, weight_name: str = "weight", delta_scale: float = 1.0):
+    def __init__(self, size: int, eps: float, weight_name: str = "weight", delta_scale: float = 1.0, bias_name: str | None = None):
         self.size, self.eps, self.weight_name, self.delta_scale = int(size), float(eps), weight_name, float(delta_scale)
+        self.bias_name = bias_name
         self.weight: torch.Tensor | None = None
+        self.bias: torch.Tensor | None = None
 
     def tensor_specs(self):
-        return {self.weight_name: TensorSpec((self.size,), "vector")}
+        specs = {self.weight_name: TensorSpec((self.size,), "vector")}
+        if self.bias_name is not None:
+            specs[self.bias_name] = TensorSpec((self.size,), "vector", init=(0.0, 0.1))
+        return specs
 
     def load(self, tensors):
         self.weight = tensors[self.weight_name].float().contiguous()
+        if self.bias_name is not None:
+            self.bias = tensors[self.bias_name].float().contiguous()
 
     def weight_bytes(self):
-        return self.weight.numel() * self.weight.element_size()
+        return sum(t.numel() * t.element_size() for t in (self.weight, self.bias) if t is not None)
+
+    def rule(self) -> tuple[torch.Tensor, torch.Tensor, float]:
+        """What the kernel that merges branches needs of a norm with a bias."""
+        return self.weight, self.bias, self.eps
 
     def forward(self, h, delta, out_dtype, rows=None):
-        return F.add_layernorm(h, delta, self.weight, self.eps, out_dtype, rows, self.delta_scale)
+        return F.add_layernorm(h, delta, self.weight, self.eps, out_dtype, rows, self.delta_scale, bias=self.bias)
 
     def forward_conv_single(self, h, delta, conv_weight, state, ctx, update_state: bool):
         """The norm and the short convolution over time behind it as one kernel, in steps of one token a sequence."""
+        if self.bias is not None:
+            raise ValueError("the kernel of norm and convolution takes no bias")
         return F.add_layernorm_conv_single(h, delta, self.weight, self.eps, conv_weight, state, ctx.tok_pos, ctx.tok_seq, ctx.slots,
                                            ctx.dtype, self.delta_scale, update_state)
 

@@ -1,11 +1,12 @@
 """Grouped-query attention with a rule for the scores and a rule for the weights.
 
 ``q = W_q x`` (``n_q_heads`` heads of ``key_dim``), ``k = W_k x`` and ``v = W_v x`` (``n_kv_heads`` heads of ``key_dim``
-and ``value_dim``; query head ``h`` reads key/value head ``h // (n_q_heads / n_kv_heads)``), no biases.  The builder
-chooses what happens around the scores:
+and ``value_dim``; query head ``h`` reads key/value head ``h // (n_q_heads / n_kv_heads)``), no biases unless ``qkv_bias``.  The
+builder chooses what happens around the scores:
 
 * ``position``: the first ``position.dim`` entries of every q and k head are rotated by position (entry ``i`` paired with
-  ``i + dim/2``), the rest pass; without it positions enter only through the rules below;
+  ``i + dim/2``, or with ``pairing="neighbours"`` entry ``2i`` with ``2i + 1``), the rest pass; without it positions enter only
+  through the rules below;
 * ``unit_qk``: after the rotation every q and k head is divided by its root mean square (eps inside the root, no weight);
 * the score of key ``j`` for the token at ``i`` is ``q . k * scale``; with ``distance_bias`` the term
   ``r1_h * ln(1 + r2_h * (i - j))`` is taken off, ``r1`` and ``r2`` being a number per query head (tensors ``r1``, ``r2``);
@@ -16,6 +17,8 @@ chooses what happens around the scores:
 
 Further rules, each switched on by the builder:
 
+* ``qkv_bias``: ``q = W_q x + b_q`` and so for k and v (tensors ``q.b``, ``k.b``, ``v.b``); the sums are formed in 32-bit before
+  anything else;
 * ``wide_norm``: before anything else the whole query row (all heads at once) is divided by its root mean square and
   multiplied by a weight per entry (tensor ``q.norm``), and so is the whole key row (``k.norm``);
 * ``head_norm``: every query head is divided by its root mean square (eps inside the root) and multiplied by one weight of
@@ -40,9 +43,9 @@ Further rules, each switched on by the builder:
   back any of their readers look (None: every page is kept; by default the layer's own window or chunk).
 
 Scores, weights and the sums over keys are 32-bit.  A step's kernels: the packed projection q | k | v | g; one kernel for
-norms, rotation, unit lengths and the cache write; attention over the pages (on the tensor cores in bfloat16 with keys and
-values of 64 or 128 entries, where steps of few tokens are cut over the keys into parts; else the exact kernel); the
-read-outs' turn back and gate; the output projection.
+biases, norms, rotation, unit lengths and the cache write; attention over the pages (on the tensor cores in bfloat16 with keys
+of up to 128 and values of up to 256 entries, multiples of 8, where steps of few tokens are cut over the keys into parts;
+else the exact kernel); the read-outs' turn back and gate; the output projection.
 """
 
 from __future__ import annotations
@@ -53,11 +56,11 @@ import torch
 
 from ..ops import functional as F
 from ..ops.linear import linear
-from .base import KVRequest, Mixer, PositionEncoding, StepContext, TensorSpec, register_part
+from .base import KVRequest, PositionEncoding, ProjectedMixer, StepContext, TensorSpec, register_part
 from .delta_rule import _pad_rows
 
 _NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "r1": "r1", "r2": "r2", "pb": "pb", "q_norm": "q.norm", "k_norm": "k.norm",
-          "temp": "temp", "rel": "rel", "sink": "sink", "g": "g"}
+          "temp": "temp", "rel": "rel", "sink": "sink", "g": "g", "q_b": "q.b", "k_b": "k.b", "v_b": "v.b"}
 
 
 def distance_rows(rows: int, far: float) -> list[int]:
@@ -72,7 +75,7 @@ def distance_rows(rows: int, far: float) -> list[int]:
     return out
 
 
-class ScoredAttention(Mixer):
+class ScoredAttention(ProjectedMixer):
     graph_safe = True
 
     def __init__(self, hidden_size: int, n_q_heads: int, n_kv_heads: int, key_dim: int, value_dim: int, scale: float,
@@ -81,7 +84,8 @@ class ScoredAttention(Mixer):
                  names: dict[str, str] | None = None, wide_norm: bool = False, temperature: bool = False,
                  distance_table: tuple[int, float] | None = None, chunk: int | None = None, sink: str | None = None,
                  value_position: PositionEncoding | None = None, head_gate: bool = False, own_kv: bool = True,
-                 cache_span: int | None | str = "own", head_norm: bool = False, softcap: float | None = None):
+                 cache_span: int | None | str = "own", head_norm: bool = False, softcap: float | None = None,
+                 qkv_bias: bool = False, pairing: str = "halves"):
         if n_q_heads % n_kv_heads:
             raise ValueError("query heads must be a multiple of key heads")
         if weights not in ("softmax", "sigmoid"):
@@ -107,6 +111,11 @@ class ScoredAttention(Mixer):
             raise ValueError("norms per head come without rotation, unit lengths and norms over whole rows")
         if self.softcap and weights != "softmax":
             raise ValueError("capped scores belong to the softmax")
+        if pairing not in ("halves", "neighbours"):
+            raise ValueError(f"rotated entries are paired as 'halves' or 'neighbours', not {pairing!r}")
+        if qkv_bias and (self.wide_norm or not own_kv):
+            raise ValueError("biases come with keys and values of the layer's own and without norms over whole rows")
+        self.qkv_bias, self.pairing = bool(qkv_bias), pairing
         self.distance_table = None if distance_table is None else (int(distance_table[0]), float(distance_table[1]))
         self.dist_rows = None  # formed at load: the table's height is the tensor's
         self.chunk = None if not chunk else int(chunk)
@@ -120,7 +129,7 @@ class ScoredAttention(Mixer):
         else:  # the builder's word: a number of positions, or None for all
             self.cache_span = int(cache_span) if cache_span else None
         self.names = {**_NAMES, **(names or {})}
-        self.w_in = self.w_o = self.r1 = self.r2 = self.pb = None
+        self.w_in = self.w_o = self.r1 = self.r2 = self.pb = self.bias = None
         self.q_norm = self.k_norm = self.temp = self.dist_bias = self.sink = None
 
     def tensor_specs(self):
@@ -130,6 +139,9 @@ class ScoredAttention(Mixer):
             specs[n["k"]] = TensorSpec((self.n_kv * self.d, W))
             specs[n["v"]] = TensorSpec((self.n_kv * self.dv, W))
         specs[n["o"]] = TensorSpec((W, self.n_q * self.dv))
+        if self.qkv_bias:
+            for key, size in (("q_b", self.n_q * self.d), ("k_b", self.n_kv * self.d), ("v_b", self.n_kv * self.dv)):
+                specs[n[key]] = TensorSpec((size,), "vector", init=(0.0, 0.3))
         if self.distance_bias:
             specs[n["r1"]] = TensorSpec((self.n_q,), "vector", init=(0.3, 0.1))
             specs[n["r2"]] = TensorSpec((self.n_q,), "vector", init=(0.5, 0.1))
@@ -163,6 +175,8 @@ class ScoredAttention(Mixer):
             mats = [m.float() for m in mats]
         self.w_in = _pad_rows(torch.cat(mats, dim=0)).contiguous()
         self.w_o = tensors[n["o"]].contiguous()
+        if self.qkv_bias:
+            self.bias = torch.cat([tensors[n[key]].float() for key in ("q_b", "k_b", "v_b")]).contiguous()
         if self.distance_bias:
             self.r1, self.r2 = tensors[n["r1"]].float().contiguous(), tensors[n["r2"]].float().contiguous()
         if self.head_bias:
@@ -187,13 +201,21 @@ class ScoredAttention(Mixer):
             self.sink = torch.zeros(self.n_q, dtype=torch.float32, device=self.w_o.device)
 
     def weight_bytes(self):
-        return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o))
+        return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o) if t is not None)
 
     def cache_request(self):
         return KVRequest(self.n_kv, self.d, self.cache_span, value_dim=None if self.dv == self.d else self.dv,
                          keep_first=self.keep_first if self.cache_span == self.window else 0)
 
-    def forward(self, x, ctx: StepContext, cache: F.PagedKV) -> torch.Tensor:
+    @property
+    def packable(self) -> bool:
+        return self.own_kv and not (self.wide_norm or self.head_gate or self.value_position is not None)
+
+    @property
+    def out_columns(self) -> int:
+        return self.n_q * self.dv
+
+    def core(self, proj, at: int, ctx: StepContext, cache: F.PagedKV, out=None, out_at: int = 0, out_scale: float = 1.0) -> torch.Tensor:
         cos = sin = v_cos = v_sin = None
         if self.rot:
             cos, sin = self.position.cos, self.position.sin
@@ -201,31 +223,38 @@ class ScoredAttention(Mixer):
             v_cos, v_sin = self.value_position.cos, self.value_position.sin
         write = self.own_kv and not ctx.extras.get("cache_read_only", False)
         nq, nk = self.n_q * self.d, self.n_kv * self.d
-        proj = linear(x, self.w_in)
         if self.wide_norm:
             q = F.wide_norm_rope_write(proj, self.n_q, self.n_kv, self.d, self.q_norm, self.k_norm, self.norm_eps, None, None, 0,
                                        ctx.tok_pos, ctx.tok_seq, ctx.slots, cache, ctx.max_position, write,
                                        v_at=nq + nk if self.own_kv else None, has_k=self.own_kv)
         else:
-            k_at, v_at = (nq, nq + nk) if self.own_kv else (0, 0)
-            q = F.heads_prepare(proj, 0, k_at, v_at, self.n_q, self.n_kv, self.d, self.dv, ctx.tok_pos, ctx.tok_seq, ctx.slots,
+            k_at, v_at = (at + nq, at + nq + nk) if self.own_kv else (at, at)
+            q = F.heads_prepare(proj, at, k_at, v_at, self.n_q, self.n_kv, self.d, self.dv, ctx.tok_pos, ctx.tok_seq, ctx.slots,
                                 rot=self.rot, cos=cos, sin=sin, unit_eps=self.norm_eps if self.unit_qk or self.head_norm else None, kv=cache,
                                 w_q=self.q_norm if self.head_norm else None, w_k=self.k_norm if self.head_norm else None,
                                 write_kv=write, max_position=ctx.max_position, v_cos=v_cos if self.own_kv else None,
-                                v_sin=v_sin if self.own_kv else None)
-        rules = dict(chunk=self.chunk or 0, temp=self.temp, dist_bias=self.dist_bias, sink=self.sink, softcap=self.softcap)
-        if q.dtype == torch.bfloat16 and self.d == self.dv and self.d in (64, 128) and cache.page_size == 64:
+                                v_sin=v_sin if self.own_kv else None, bias=self.bias, bias_at=at, neighbours=self.pairing == "neighbours")
+        rules = dict(chunk=self.chunk or 0, temp=self.temp, dist_bias=self.dist_bias, sink=self.sink, softcap=self.softcap, out=out,
+                     out_at=out_at, out_scale=out_scale)
+        if q.dtype == torch.bfloat16 and F.attention_scored_fits(self.d, self.dv, self.softcap) and cache.page_size == 64:
             # what a row can see at most, whatever the lengths of later steps that replay this one from a graph
             spans = [s for s in (self.window + self.keep_first if self.window else None, self.chunk) if s]
             seen = -(-min(spans) // 64) + 2 if spans else cache.max_pages
             parts = F.scored_attention_parts(ctx.n_seqs, self.n_q, self.n_kv, ctx.max_q_len, min(seen, cache.max_pages),
                                              F.sm_count(q.device))
-            o = F.attention_scored(q, cache, ctx.cu_q, ctx.kv_len, ctx.slots, ctx.max_q_len, self.scale, self.window or 0,
-                                   self.keep_first, self.r1, self.r2, self.pb, self.weights, parts, **rules)
-        else:  # 32-bit runs and other head sizes
-            o = F.attention_scored_exact(q, cache, ctx.tok_pos, ctx.tok_seq, ctx.slots, self.scale, self.window or 0,
-                                         self.keep_first, self.r1, self.r2, self.pb, self.weights, **rules)
+            return F.attention_scored(q, cache, ctx.cu_q, ctx.kv_len, ctx.slots, ctx.max_q_len, self.scale, self.window or 0,
+                                      self.keep_first, self.r1, self.r2, self.pb, self.weights, parts, **rules)
+        # 32-bit runs and other head sizes
+        return F.attention_scored_exact(q, cache, ctx.tok_pos, ctx.tok_seq, ctx.slots, self.scale, self.window or 0,
+                                        self.keep_first, self.r1, self.r2, self.pb, self.weights, **rules)
+
+    def forward(self, x, ctx: StepContext, cache: F.PagedKV) -> torch.Tensor:
+        proj = linear(x, self.w_in)
+        o = self.core(proj, 0, ctx, cache)
         if self.value_position is not None or self.head_gate:
+            v_cos = v_sin = None
+            if self.value_position is not None:
+                v_cos, v_sin = self.value_position.cos, self.value_position.sin
             o = F.turn_back_gate(o, v_cos, v_sin, ctx.tok_pos, ctx.max_position, proj if self.head_gate else None, self.gate_at)
         return linear(o.view(ctx.n_tokens, self.n_q * self.dv), self.w_o)
 

@@ -88,3 +88,7 @@ def _ensure_builtin() -> None:
     from .models.topezen import build_topezen_plan
 
     register_architecture(TopezenConfig.ARCH_NAMES, TopezenConfig, build_topezen_plan)
+    from .config.katopel import KatopelConfig
+    from .models.katopel import build_katopel_plan
+
+    register_architecture(KatopelConfig.ARCH_NAMES, KatopelConfig, build_katopel_plan)
