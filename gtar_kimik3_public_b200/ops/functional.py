@@ -1448,6 +1448,41 @@ def conv_ring(proj: torch.Tensor, at: int, hd: DeltaHeads, ring: torch.Tensor, c
          ptr(kv_len), ptr(slots), kv_len.shape[0], hd.channels, hd.taps, stream_ptr())
 
 
+DELTA_CHUNK = 64                   # tokens a chunk of delta_chunked
+DELTA_WORKSPACE_BYTES = 128 << 20  # at most this much of chunks' matrices in flight
+
+
+def delta_chunked_fits(d: int, dv: int) -> bool:
+    """Whether :func:`delta_chunked` takes heads of these sizes: multiples of 8, keys of up to 128 entries."""
+    return bool(library().gk_delta_chunked_fits(int(d), int(dv)))
+
+
+def delta_chunked(x: DeltaInputs, state: torch.Tensor, cu_q: torch.Tensor, slots: torch.Tensor, n_seqs: int, max_q_len: int) -> torch.Tensor:
+    """The recurrence over the step's tokens of every sequence, in chunks of 64 tokens on the tensor cores, from and to ``state
+    [slots, n_heads, d, dv]`` (32-bit).  ``x`` holds rounded vectors; ``max_q_len`` bounds the sequences' token counts in this step.
+    Returns ``o [T, n_heads, dv]`` (32-bit)."""
+    require_device(x.q.device)
+    for name, t in (("q", x.q), ("k", x.k), ("v", x.v)):
+        _check(t, name, torch.bfloat16, 3)
+    for name, t in (("q_unit", x.q_unit), ("k_unit", x.k_unit), ("g", x.g), ("beta", x.beta)):
+        _check(t, name, torch.float32, 2)
+    _check(state, "state", torch.float32, 4)
+    T, n_kv, d = x.q.shape
+    n_heads, dv = x.v.shape[1], x.v.shape[2]
+    if tuple(state.shape[1:]) != (n_heads, d, dv) or x.k.shape != x.q.shape or not delta_chunked_fits(d, dv):
+        raise KernelError("delta_chunked: the state or the inputs have other sizes than the heads, or sizes that the chunks do not take")
+    dev = x.q.device
+    out = torch.empty((T, n_heads, dv), dtype=torch.float32, device=dev)
+    n_work, n_factors = library().gk_delta_chunked_work(0), library().gk_delta_chunked_work(1)
+    chunks = max(1, -(-int(max_q_len) // DELTA_CHUNK))
+    wave = max(1, min(chunks, DELTA_WORKSPACE_BYTES // max(1, 2 * n_work * n_seqs * n_heads)))
+    work = torch.empty((max(1, n_seqs) * wave * n_heads * n_work,), dtype=torch.bfloat16, device=dev)
+    factors = torch.empty((max(1, n_seqs) * wave * n_heads * n_factors,), dtype=torch.float32, device=dev)
+    call("gk_delta_chunked", ptr(x.q), ptr(x.k), ptr(x.v), ptr(x.q_unit), ptr(x.k_unit), ptr(x.g), ptr(x.beta), ptr(work), ptr(factors),
+         ptr(state), ptr(out), ptr(cu_q), ptr(slots), int(n_seqs), n_heads, n_kv, d, dv, int(max_q_len), wave, stream_ptr())
+    return out
+
+
 def delta_head_single_fits(d: int, dv: int) -> bool:
     """Whether :func:`delta_head_single` takes heads of these sizes (a block holds a head's state in registers)."""
     return bool(library().gk_delta_head_single_fits(int(d), int(dv)))

@@ -73,6 +73,9 @@ _SIGNATURES: dict[str, list] = {
     "gk_conv_ring": [P, I, L, P, P, P, P, I, I, I, P],
     "gk_delta_head_single": [P, I, L, P, P, P, P, P, P, P, P, P, P, L, F, F, I, I, I, I, I, I, P],
     "gk_delta_head_single_fits": [I, I],
+    "gk_delta_chunked_fits": [I, I],
+    "gk_delta_chunked_work": [I],
+    "gk_delta_chunked": [P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
     "gk_head_norm_gate": [P, P, P, I, L, P, I, L, I, I, F, P],
     "gk_route_groups": [P, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P, P],
     "gk_experts_up": [P, I, P, I, P, P, I, I, I, I, P],

@@ -198,12 +198,15 @@ class HeadDeltaRule(ProjectedMixer):
             F.delta_head_single(proj, at, hd, self.conv_w, ring, self.a_log, self.dt_bias, self.norm_w, state, ctx.tok_pos, ctx.tok_seq,
                                 ctx.slots, self.norm_eps, out, out_at, out_scale)
             return
-        chunked = False
+        chunked = ctx.dtype == torch.bfloat16 and proj.dtype == torch.bfloat16 and F.delta_chunked_fits(hd.d, hd.dv)
         x = F.delta_head_prepare(proj, at, hd, self.conv_w, ring, self.a_log, self.dt_bias, ctx.tok_pos, ctx.tok_seq, ctx.cu_q, ctx.slots,
                                  rounded=chunked)
         if ring is not None:
             F.conv_ring(proj, at, hd, ring, ctx.cu_q, ctx.kv_len, ctx.slots)
-        o = F.delta_scan(x.q, x.k, x.v, x.g, x.beta, state, ctx.cu_q, ctx.slots, ctx.n_seqs)
+        if chunked:
+            o = F.delta_chunked(x, state, ctx.cu_q, ctx.slots, ctx.n_seqs, ctx.max_q_len)
+        else:
+            o = F.delta_scan(x.q, x.k, x.v, x.g, x.beta, state, ctx.cu_q, ctx.slots, ctx.n_seqs)
         F.group_norm_gate(o.view(ctx.n_tokens, -1), hd.dv, self.norm_w, proj, at + hd.gate_at, self.norm_eps, ctx.dtype, "silu", out=out,
                           out_at=out_at, out_scale=out_scale)
 

@@ -82,7 +82,7 @@ def over_time(x: torch.Tensor, taps: torch.Tensor) -> torch.Tensor:
     """Per channel, x [T, C], taps [C, n]: y_t = sum_j taps[:, n-1-j] x_(t-j), zeros before the start."""
     n = taps.shape[1]
     y = torch.zeros_like(x)
-    for j in range(n):
+    for j in range(min(n, x.shape[0])):
         y[j:] += taps[:, n - 1 - j] * x[:x.shape[0] - j]
     return y
 
