@@ -15,7 +15,8 @@ from there), token ids are seeded uniform-random: there is no network for checkp
 The library runs on one GPU; with --gpus N > 1 a line says so and the exit code is 2.
 
 ``--compare pofadra`` and ``--compare rezulorn`` do the same for the Pofadra and the Rezulorn decoders; ``--compare zasorax`` puts the Zasorax decoder beside the Rezulorn decoder,
-``--compare topezen`` the Topezen decoder beside the Pofadra decoder.  ``--compare dasusun`` runs another workload instead and prints its own JSON line: the Dasusun decoder beside the transformer
+``--compare topezen`` and ``--compare katopel`` the Topezen and the Katopel decoders beside the Pofadra decoder.
+``--compare dasusun`` runs another workload instead and prints its own JSON line: the Dasusun decoder beside the transformer
 at equal layer sizes (prefill and decode throughput of both, and the new design's kernels one by one against their rooflines).
 """
 
@@ -1735,6 +1736,271 @@ def run_compare_topezen(args) -> dict:
             "results": results}
 
 
+# --compare katopel: the Katopel decoder (a layer norm on both sides of every branch, layers that run twice; the gated delta rule
+# with one decay per head, alone or beside chunked attention; dense and routed feed-forwards with a gated shared expert)
+# beside the Pofadra decoder (delta-rule layers, one attention in four, routed experts) at equal width, about equal bytes of
+# weights read per token and equally many layer runs, and its kernels one by one beside the like kernels.
+def _katopel_config(width, layers, heads, kv_heads, dim, vdim, conv, a_heads, a_kv, a_dim, a_vdim, chunk, rot, loop, ff, experts, top,
+                    expert_ff, shared_ff, vocab):
+    delta = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}
+    attention = {"heads": a_heads, "kv_heads": a_kv, "dim": a_dim, "vdim": a_vdim, "scale": a_dim ** -0.5, "mask": {"size": chunk},
+                 "rot": {"base": 500000.0, "dims": rot}}
+    pair = {"left": attention, "right": delta, "left_scale": 0.7, "right_scale": 1.0}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff}, "router": {"experts": experts, "top": top}}
+    kinds = [("delta", delta, dense), ("parallel", pair, moe), ("delta", delta, moe)]
+    stack = [dict(zip(("type", "mixer", "mlp"), kinds[i % 3])) for i in range(layers)]
+    return {"architecture": "Katopel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+            "loop": dict(zip(("start", "stop", "times"), loop)), "layers": stack, "initializer_range": 0.02, "max_position_embeddings": 4096}
+
+
+KATOPEL_SIZES = {
+    # name: (Katopel sizes, Pofadra sizes); 6 layers of which 2 run twice beside 8 layers, vocabulary 32,768; a routed layer's
+    # chosen and shared experts hold what the chosen experts of the other design hold, and so does a dense layer
+    "width1024": (dict(width=1024, layers=6, heads=8, kv_heads=8, dim=128, vdim=128, conv=4, a_heads=8, a_kv=2, a_dim=64, a_vdim=128, chunk=1024,
+                       rot=32, loop=(1, 3, 2), ff=3072, experts=32, top=3, expert_ff=768, shared_ff=768, vocab=32768),
+                  POFADRA_SIZES["width1024"][0]),
+    "width2048": (dict(width=2048, layers=6, heads=16, kv_heads=16, dim=128, vdim=128, conv=4, a_heads=16, a_kv=4, a_dim=128, a_vdim=256,
+                       chunk=1024, rot=64, loop=(1, 3, 2), ff=6144, experts=64, top=5, expert_ff=1024, shared_ff=1024, vocab=32768),
+                  POFADRA_SIZES["width2048"][0]),
+}
+
+
+def _katopel_runs(d: dict) -> list[int]:
+    """The layers in the order in which they run."""
+    start, stop, times = d["loop"]
+    return list(range(start)) + list(range(start, stop)) * times + list(range(stop, d["layers"]))
+
+
+def _katopel_prefill_flops(d: dict, tokens: int) -> float:
+    w, H, G, dk, dv = d["width"], d["heads"], d["kv_heads"], d["dim"], d["vdim"]
+    delta = 2 * w * (2 * G * dk + 3 * H * dv + 2 * H) + H * dv * 6 * dk
+    aq, ak, ad, av = d["a_heads"], d["a_kv"], d["a_dim"], d["a_vdim"]
+    attention = 2 * w * (aq * ad + ak * (ad + av) + aq * av)
+    seen = sum(t % d["chunk"] + 1 for t in range(tokens))
+    dense = 6 * w * d["ff"]
+    routed = 2 * w * (d["experts"] + 1) + 6 * w * (d["top"] * d["expert_ff"] + d["shared_ff"])
+    total = 0.0
+    for i in _katopel_runs(d):
+        total += tokens * (delta + (dense if i % 3 == 0 else routed))
+        if i % 3 == 1:
+            total += tokens * attention + aq * seen * 2 * (ad + av)
+    return total + 2 * w * d["vocab"]
+
+
+def _katopel_kernel_table(d: dict, f: dict, peak: dict) -> dict:
+    """The new design's kernels alone and the like kernels of the models that were here (the Pofadra decoder's recurrence,
+    convolutions, norm, gate, router and experts, the Rezulorn decoder's layer norm and cache write, the Zasorax decoder's chunked
+    attention), each with its share of its roofline."""
+    import torch
+
+    from gtar_kimik3_public_b200.ops import functional as F
+    from gtar_kimik3_public_b200.ops.linear import linear_grouped
+
+    dev = torch.device("cuda:0")
+    flush = torch.zeros(48 << 20, dtype=torch.float32, device=dev)  # 192 MB: larger than the 126 MB L2
+    hbm, tflops = peak["hbm_gbs"] * 1e9, peak["bf16_tflops"] * 1e12
+    out = {}
+
+    def record(name, ms, n_bytes, flops=0.0):
+        floor = max(n_bytes / hbm, flops / tflops) * 1e3
+        out[name] = {"us": round(ms * 1e3, 2), "roofline_us": round(floor * 1e3, 2), "frac": round(floor / ms, 4),
+                     "bound": "hbm" if n_bytes / hbm >= flops / tflops else "tensor"}
+
+    w, H, G, dk, dv, taps = d["width"], d["heads"], d["kv_heads"], d["dim"], d["vdim"], d["conv"]
+    aq, ak, ad, av, chunk = d["a_heads"], d["a_kv"], d["a_dim"], d["a_vdim"], d["chunk"]
+    bf = torch.bfloat16
+    for label, tokens, n_seqs in (("prefill_2048", 2048, 1), ("decode_b8_ctx2048", 8, 8)):
+        each = tokens // n_seqs
+        past = 0 if n_seqs == 1 else 2047
+        length = past + each
+        pages_each = -(-length // 64)
+        table = torch.arange(n_seqs * pages_each, dtype=torch.int32, device=dev).view(n_seqs, pages_each)
+        tok_seq = torch.arange(n_seqs, dtype=torch.int32, device=dev).repeat_interleave(each)
+        tok_pos = (torch.arange(each, dtype=torch.int32, device=dev) + past).repeat(n_seqs)
+        cu_q = torch.arange(n_seqs + 1, dtype=torch.int32, device=dev) * each
+        slots = torch.arange(n_seqs, dtype=torch.int32, device=dev)
+        kv_len = torch.full((n_seqs,), length, dtype=torch.int32, device=dev)
+        timed = dict(flush=flush, inner=1 if n_seqs == 1 else 20)
+        # ---- the stream
+        hs, first, step = torch.randn(tokens, w, device=dev), torch.randn(tokens, w, device=dev), torch.randn(w, device=dev)
+        branch = torch.randn(tokens, w, device=dev).to(bf)
+        norm = (torch.ones(w, device=dev), torch.zeros(w, device=dev), 1e-5)
+        ms = _event_ms(lambda: F.layernorm_merge(hs, branch, norm, norm_z=norm, z_dtype=bf, x_out=hs), **timed)
+        record(f"katopel norm, add, next norm, {label}", ms, tokens * w * (4 + 2 + 4 + 2))
+        ms = _event_ms(lambda: F.layernorm_merge(hs, branch, norm, first=first, step=step, norm_z=norm, z_dtype=bf, x_out=hs), **timed)
+        record(f"katopel norm, add, a pass's adds, next norm, {label}", ms, tokens * w * (4 + 2 + 4 + 4 + 2))
+        ms = _event_ms(lambda: F.branch_merge(hs, branch, norm[0], 1e-5, next_weight=norm[0], next_eps=1e-5, next_dtype=bf, x_out=hs), **timed)
+        record(f"dasusun norm, add, next norm (RMS), {label}", ms, tokens * w * (4 + 2 + 4 + 2))
+        ms = _event_ms(lambda: F.add_layernorm(hs, branch, norm[0], 1e-5, bf), **timed)
+        record(f"rezulorn add with next layer norm, {label}", ms, tokens * w * (4 + 2 + 4 + 2))
+        # ---- the delta rule, from the packed projection to the gated read-outs
+        hd = F.DeltaHeads(H, G, dk, dv, taps)
+        proj = (torch.randn(tokens, -(-hd.columns // 8) * 8, device=dev) * 0.5).to(bf)
+        conv_w, ring = torch.randn(taps, hd.channels, device=dev) * 0.3, torch.zeros(n_seqs, taps, hd.channels, device=dev)
+        a_log, dt_bias, head_w = torch.randn(H, device=dev) - 1, torch.randn(H, device=dev) - 1, torch.ones(dv, device=dev)
+        state = torch.zeros(n_seqs, H, dk, dv, device=dev)
+        read = torch.empty(tokens, H * dv, dtype=bf, device=dev)
+        weights_of = (conv_w, ring, a_log, dt_bias)
+        place = (tok_pos, tok_seq, cu_q, slots)
+        state_bytes = 8 * n_seqs * H * dk * dv
+        io_bytes = 2 * tokens * (hd.columns + H * dv)
+        delta_flops = tokens * H * 6 * dk * dv
+
+        def norm_gate(o):
+            return F.group_norm_gate(o.view(tokens, -1), dv, head_w, proj, hd.gate_at, 1e-5, bf, "silu", out=read)
+
+        if n_seqs == 1:
+            ms = _event_ms(lambda: F.delta_head_prepare(proj, 0, hd, *weights_of, *place, rounded=True), **timed)
+            record(f"katopel convolutions, unit lengths, decays and beta, {label}", ms, 2 * tokens * (2 * hd.channels + 2 * H) + 8 * tokens * (G + H))
+            x = F.delta_head_prepare(proj, 0, hd, *weights_of, *place, rounded=True)
+            ms = _event_ms(lambda: F.delta_chunked(x, state, cu_q, slots, n_seqs, each), **timed)
+            record(f"katopel delta rule recurrence in chunks, {label}", ms, tokens * (2 * hd.channels + 8 * (G + H) + 4 * H * dv) + state_bytes, delta_flops)
+            o = F.delta_chunked(x, state, cu_q, slots, n_seqs, each)
+            ms = _event_ms(lambda: norm_gate(o), **timed)
+            record(f"katopel head norm and gate, {label}", ms, tokens * H * dv * (4 + 2 + 2))
+
+            def whole():
+                x = F.delta_head_prepare(proj, 0, hd, *weights_of, *place, rounded=True)
+                F.conv_ring(proj, 0, hd, ring, cu_q, kv_len, slots)
+                norm_gate(F.delta_chunked(x, state, cu_q, slots, n_seqs, each))
+        else:
+            def whole():
+                F.delta_head_single(proj, 0, hd, *weights_of, head_w, state, tok_pos, tok_seq, slots, 1e-5, read)
+        ms = _event_ms(whole, **timed)
+        record(f"katopel delta rule: everything between the products, {label}", ms, io_bytes + state_bytes, delta_flops)
+        xf = F.delta_head_prepare(proj, 0, hd, *weights_of, *place)
+        ms = _event_ms(lambda: F.delta_scan(xf.q, xf.k, xf.v, xf.g, xf.beta, state, cu_q, slots, n_seqs), **timed)
+        record(f"katopel delta rule recurrence token by token (32-bit run), {label}", ms, 4 * tokens * (hd.channels + H * dv + 2 * H) + state_bytes)
+        # ---- the same of the Pofadra decoder
+        fh, fg, fk, fv = f["heads"], f["kv_heads"], f["dim"], f["vdim"]
+        fc = 2 * fg * fk + fh * fv
+        f_proj = (torch.randn(tokens, fc + fh + (-(fc + fh)) % 8, device=dev) * 0.5).to(bf)
+        low = torch.randn(tokens, fh * (fk + fv), device=dev)
+        f_conv, f_conv_state = torch.randn(fc, taps, device=dev) * 0.3, torch.zeros(n_seqs, taps - 1, fc, device=dev)
+        f_log, f_dt = torch.randn(fh, device=dev) - 1, torch.randn(fh * fk, device=dev) - 1
+        f_state, f_w = torch.zeros(n_seqs, fh, fk, fv, device=dev), torch.ones(fv, device=dev)
+        prepare = lambda: F.delta_prepare(f_proj, low, f_conv, f_conv_state, f_log, f_dt, *place, fh, fg, fk, fv, taps, roll_single=n_seqs > 1)
+        ms = _event_ms(prepare, **timed)
+        record(f"pofadra convolutions, unit lengths, decays and beta, {label}", ms, tokens * (2 * (fc + fh) + 4 * fh * fk + 4 * (fc + fh * fk + fh)))
+        fx = prepare()
+        ms = _event_ms(lambda: F.delta_scan(*fx, f_state, cu_q, slots, n_seqs), **timed)
+        f_state_bytes = 8 * n_seqs * fh * fk * fv
+        record(f"pofadra delta rule recurrence, {label}", ms, 4 * tokens * (2 * fg * fk + fh * fk + 2 * fh * fv + fh) + f_state_bytes)
+        f_o = F.delta_scan(*fx, f_state, cu_q, slots, n_seqs)
+        ms = _event_ms(lambda: F.head_norm_gate(f_o, f_w, low, fh * fk, 1e-6, bf), **timed)
+        record(f"pofadra head norm and gate, {label}", ms, tokens * fh * fv * (4 + 4 + 2))
+
+        def pofadra_whole():
+            fx = prepare()
+            if n_seqs == 1:
+                F.conv_roll(f_proj, f_conv_state, cu_q, slots, n_seqs, fc)
+            F.head_norm_gate(F.delta_scan(*fx, f_state, cu_q, slots, n_seqs), f_w, low, fh * fk, 1e-6, bf)
+
+        ms = _event_ms(pofadra_whole, **timed)
+        record(f"pofadra delta rule: everything between the products, {label}", ms,
+               tokens * (2 * (fc + fh) + 4 * fh * (fk + fv) + 2 * fh * fv) + f_state_bytes, tokens * fh * 6 * fk * fv)
+        # ---- chunked attention
+        kv = F.PagedKV(torch.randn(n_seqs * pages_each, ak, 64, ad, device=dev).to(bf) * 0.1,
+                       torch.randn(n_seqs * pages_each, ak, 64, av, device=dev).to(bf) * 0.1, table, F.DecodeWork(dev))
+        wide = torch.randn(tokens, aq * ad + ak * (ad + av), device=dev).to(bf)
+        bias = torch.randn(wide.shape[1], device=dev)
+        angle = torch.arange(length, dtype=torch.float32, device=dev)[:, None] * torch.rand(d["rot"] // 2, device=dev)[None, :]
+        cos, sin = angle.cos().contiguous(), angle.sin().contiguous()
+        columns = (wide, 0, aq * ad, (aq + ak) * ad, aq, ak, ad, av, tok_pos, tok_seq, slots)
+        ms = _event_ms(lambda: F.heads_prepare(*columns, rot=d["rot"], cos=cos, sin=sin, kv=kv, max_position=length - 1, bias=bias,
+                                               neighbours=True), **timed)
+        record(f"katopel biases, rotation, cache write, {label}", ms, tokens * 4 * wide.shape[1])
+        ms = _event_ms(lambda: F.heads_prepare(*columns, rot=d["rot"], cos=cos, sin=sin, unit_eps=1e-6, kv=kv, max_position=length - 1), **timed)
+        record(f"rezulorn rotation, unit q and k, cache write (same sizes), {label}", ms, tokens * 4 * wide.shape[1])
+        qa = torch.randn(tokens, aq, ad, device=dev).to(bf)
+        seen = sum(p % chunk + 1 for p in range(past, length)) * n_seqs
+        keys = sum(min(length - c, chunk) for c in range(past // chunk * chunk, length, chunk)) * n_seqs
+        parts = F.scored_attention_parts(n_seqs, aq, ak, each, -(-chunk // 64) + 2, F.sm_count(dev))
+        ms = _event_ms(lambda: F.attention_scored(qa, kv, cu_q, kv_len, slots, each, ad ** -0.5, n_parts=parts, chunk=chunk), **timed)
+        record(f"katopel attention: keys of {ad}, values of {av}, chunks of {chunk}, {label}", ms,
+               2 * (tokens * aq * (ad + av) + keys * ak * (ad + av)), 2 * aq * (ad + av) * seen)
+        z_kv = F.PagedKV(kv.k, torch.randn_like(kv.k) * 0.1, table, F.DecodeWork(dev))
+        temp, dist = torch.ones(aq, device=dev), torch.randn(chunk, aq, device=dev) * 0.1
+        ms = _event_ms(lambda: F.attention_scored(qa, z_kv, cu_q, kv_len, slots, each, ad ** -0.5, n_parts=parts, chunk=chunk, temp=temp,
+                                                  dist_bias=dist, sink=temp), **timed)
+        record(f"zasorax attention: keys and values of {ad}, chunks of {chunk}, distance table, sink, {label}", ms,
+               2 * (tokens * aq * 2 * ad + keys * ak * 2 * ad), 4 * aq * ad * seen)
+        # ---- routers and experts
+        h = torch.randn(tokens, w, device=dev).to(bf)
+        E, top, ff = d["experts"], d["top"], d["expert_ff"]
+        w_r, none = torch.randn(E + 1, w, device=dev) * 0.05, torch.zeros(E, device=dev)
+        ms = _event_ms(lambda: F.route_groups(h, w_r, none, top, 1, 1, 1.0, logits=True, shared="pair"), **timed)
+        record(f"katopel router with the shared expert's weight, {label}", ms, tokens * w * 2 + (E + 1) * w * 4)
+        f_r, f_bias = torch.randn(f["experts"], w, device=dev) * 0.05, torch.randn(f["experts"], device=dev) * 0.1
+        ms = _event_ms(lambda: F.route_groups(h, f_r, f_bias, f["top"], f["groups"], f["keep"], 1.0), **timed)
+        record(f"pofadra router, {label}", ms, tokens * w * 2 + f["experts"] * w * 4)
+        for arch, (ids, share), n_experts, inner_ff in (
+                ("katopel", F.route_groups(h, w_r, none, top, 1, 1, 1.0, logits=True, shared="pair"), E + 1, ff),
+                ("pofadra", F.route_groups(h, f_r, f_bias, f["top"], f["groups"], f["keep"], 1.0), f["experts"], f["ff"])):
+            gate_up = (torch.randn(n_experts, 2, inner_ff, w, device=dev) * 0.02).to(bf)
+            down = (torch.randn(n_experts, w, inner_ff, device=dev) * 0.02).to(bf)
+            pairs = ids.shape[1]
+            expert_bytes = int(torch.unique(ids).numel()) * 3 * inner_ff * w * 2
+            flops = tokens * pairs * 6 * w * inner_ff
+            if n_seqs == 1:
+                def grouped():
+                    ends, place_of, pair_at = F.experts_sort(ids, n_experts)
+                    act = F.swiglu(linear_grouped(F.gather_rows(h, pair_at, pairs), gate_up.view(n_experts, 2 * inner_ff, w), ends))
+                    return F.experts_combine(linear_grouped(act, down, ends), place_of, share, None)
+                ms = _event_ms(grouped, **timed)
+                record(f"{arch} experts (sorted, grouped products), {label}", ms, expert_bytes + tokens * pairs * (w * 4 + inner_ff * 6), flops)
+            else:
+                ms = _event_ms(lambda: F.experts_pairwise(h, gate_up, down, ids, share, None), **timed)
+                record(f"{arch} experts (pair by pair), {label}", ms, expert_bytes, flops)
+            del gate_up, down
+    return out
+
+
+def run_compare_katopel(args) -> dict:
+    import gc
+
+    import torch
+
+    from gtar_kimik3_public_b200.ops.library import require_device
+
+    require_device(torch.device("cuda:0"))
+    peak, peak_source = peaks()
+    results = {}
+    for name, (d, f) in KATOPEL_SIZES.items():
+        entry = {}
+        for arch, raw, flops in (("katopel", _katopel_config(**d), _katopel_prefill_flops(d, PREFILL_TOKENS)),
+                                 ("pofadra", _pofadra_config(**f), _pofadra_prefill_flops(f, PREFILL_TOKENS))):
+            model = _device_model(raw)
+            ms = _time_prefill_ms(model, PREFILL_TOKENS)
+            decode = time_decode(model, args.batch, min(args.steps, 64), args.warmup)
+            # a step's weight bytes count the experts ONE token reads; a batch reads every distinct expert its tokens
+            # choose: with uniform choices E (1 - (1 - top / E)^batch) of them in every routed layer run
+            sizes, expert_ff = (d, d["expert_ff"]) if arch == "katopel" else (f, f["ff"])
+            distinct = sizes["experts"] * (1.0 - (1.0 - sizes["top"] / sizes["experts"]) ** args.batch)
+            routed = sum(1 for e in model.plan.run_list if raw["layers"][e.layer]["mlp"]["kind"] == "moe")
+            more = routed * (distinct - sizes["top"]) * 3 * expert_ff * sizes["width"] * 2
+            seconds = decode["ms_per_step"] / 1e3
+            entry[arch] = {
+                "weight_bytes_per_step": model.weight_bytes_per_step(), "layer_runs": len(model.plan.run_list),
+                "prefill_tokens_per_s": round(PREFILL_TOKENS / (ms / 1e3), 1), "prefill_ms": round(ms, 3),
+                "prefill_frac_of_bf16_peak": round(flops / (ms / 1e3) / (peak["bf16_tflops"] * 1e12), 4),
+                "decode_tokens_per_s": round(decode["tokens_per_s"], 1), "decode_ms_per_step": round(decode["ms_per_step"], 4),
+                "decode_frac_of_hbm_peak": round(decode["bytes_per_step"] / seconds / 1e9 / peak["hbm_gbs"], 4),
+                "decode_frac_of_hbm_peak_with_distinct_experts": round((decode["bytes_per_step"] + more) / seconds / 1e9 / peak["hbm_gbs"], 4),
+                "decode_launches_per_step": decode["launches"] // max(1, min(args.steps, 64)),
+            }
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+        entry["kernels"] = _katopel_kernel_table(d, f, peak)
+        results[name] = {"sizes": {"katopel": d, "pofadra": f}, **entry}
+    return {"compare": "katopel beside pofadra at equal width", "batch": args.batch, "prompt_tokens": PROMPT_LEN,
+            "prefill_tokens": PREFILL_TOKENS, "dtype": "bf16", "data": "synthetic: random token ids, random weights drawn on the device",
+            "peaks": dict(peak, source=peak_source), "l2": "single kernels: a 192 MB buffer is written between the timed calls of the 2,048-token cases; the 8-token cases are 20 calls back to back from a CUDA graph",
+            "results": results}
+
+
 def main() -> int:
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -1744,13 +2010,14 @@ def main() -> int:
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--layers", type=int, default=None, help="fewer layers than the configuration (named in config)")
     parser.add_argument("--no-large", action="store_true", help="leave out the points at the 4B and 8B layer sizes")
-    parser.add_argument("--compare", default=None, choices=["dasusun", "pofadra", "rezulorn", "zasorax", "topezen"],
+    parser.add_argument("--compare", default=None, choices=["dasusun", "pofadra", "rezulorn", "zasorax", "topezen", "katopel"],
                         help="instead of the default workload: this architecture beside the transformer at equal layer sizes")
     args = parser.parse_args()
     if args.compare:
         if args.warmup < 3:
             args.warmup = 3
-        runner = {"pofadra": run_compare_pofadra, "rezulorn": run_compare_rezulorn, "zasorax": run_compare_zasorax, "topezen": run_compare_topezen, "dasusun": run_compare}[args.compare]
+        runner = {"pofadra": run_compare_pofadra, "rezulorn": run_compare_rezulorn, "zasorax": run_compare_zasorax, "topezen": run_compare_topezen,
+                  "katopel": run_compare_katopel, "dasusun": run_compare}[args.compare]
         print(json.dumps(runner(args)))
         return 0
     if args.impl == "reference":
