@@ -277,19 +277,20 @@ __global__ void __launch_bounds__(128) attention_scored_join_kernel(const float*
     const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
     if (item >= n_items) return;
     const int lane = threadIdx.x & 31;
-    float top = -INFINITY;
-    if (!SIGMOID)
-        for (int s = 0; s < n_split; ++s) top = fmaxf(top, part_ml[((size_t)s * n_items + item) * 2]);
-    float acc[DV / 32], denom = 0.f;
+    // a lane has a part's maximum and sum (there are at most 32 parts)
+    float share = 1.f, denom = 0.f;
+    if (!SIGMOID) {
+        const float2 ml = lane < n_split ? *reinterpret_cast<const float2*>(part_ml + ((size_t)lane * n_items + item) * 2) : make_float2(-INFINITY, 0.f);
+        const float top = warp_max(ml.x);
+        share = ml.x == -INFINITY ? 0.f : exp2_fast(ml.x - top);
+        denom = warp_sum(ml.y * share);
+    }
+    float acc[DV / 32];
 #pragma unroll
     for (int c = 0; c < DV / 32; ++c) acc[c] = 0.f;
+#pragma unroll 4
     for (int s = 0; s < n_split; ++s) {
-        float w = 1.f;
-        if (!SIGMOID) {
-            const float2 ml = *reinterpret_cast<const float2*>(part_ml + ((size_t)s * n_items + item) * 2);
-            w = ml.x == -INFINITY ? 0.f : exp2_fast(ml.x - top);
-            denom = fmaf(ml.y, w, denom);
-        }
+        const float w = SIGMOID ? 1.f : __shfl_sync(0xffffffffu, share, s);
         const float* src = part_o + ((size_t)s * n_items + item) * dv;
 #pragma unroll
         for (int c = 0; c < DV / 32; ++c)
@@ -358,7 +359,7 @@ GK_EXPORT int gk_attention_scored_bf16(const void* q, const void* k_pages, const
     GK_REQUIRE(window >= 0 && keep_first >= 0 && max_q_len >= 0, "attention_scored_mma: bad window, kept keys or length");
     GK_REQUIRE((r1 == nullptr) == (r2 == nullptr), "attention_scored_mma: the distance term needs both of its numbers");
     GK_REQUIRE(weights == 0 || weights == 1, "attention_scored_mma: weights are softmax (0) or sigmoid (1)");
-    GK_REQUIRE(n_split >= 1 && (n_split == 1 || (part_o != nullptr && (weights == 1 || part_ml != nullptr))),
+    GK_REQUIRE(n_split >= 1 && n_split <= 32 && (n_split == 1 || (part_o != nullptr && (weights == 1 || part_ml != nullptr))),
                "attention_scored_mma: %d parts need their workspaces", n_split);
     GK_REQUIRE(chunk >= 0 && (dist_bias == nullptr || n_dist > 0), "attention_scored_mma: bad chunk or distance table");
     GK_REQUIRE(sink == nullptr || weights == 0, "attention_scored_mma: a sink belongs to the softmax");

@@ -15,9 +15,10 @@
 // with Delta Rule".)
 //
 //   inner   a block per chunk and head: M, P and the factors of the chunk's tokens
-//   walk    a warp per head and 16 value columns.  It keeps S^T in the accumulators of its products; an accumulator of one
-//           product is the left operand of the next without leaving the registers, so the chain over the chunks has no
-//           barrier but the one around the shared tiles.
+//   walk    a block per head and 16 value columns, the chunks in sequence.  Four warps carry S^T in the accumulators of their
+//           products (a quarter of the key entries each) and four form the read-outs beside them; what a product leaves for
+//           the next one passes through shared memory, three barriers a chunk.  The next chunk's tiles are on their way
+//           meanwhile.
 //
 // K, Q and V are bfloat16 numbers; every other operand (the state, v less its prediction, u, M, P) is a 32-bit number split into
 // two bfloat16 halves, the rounded number and the rounded rest; what is left out is 2^-17 of a product.  Sums are 32-bit.
@@ -47,12 +48,13 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
 
 // 64 rows of d entries (a multiple of 8, at most D), `ld` apart, into a swizzled tile with rows of D; the rest is zero.
 template <int D>
-__device__ __forceinline__ void stage_rows(bf16* tile, const bf16* __restrict__ src, long long ld, int valid, int d, int n_threads) {
+__device__ __forceinline__ void stage_rows(bf16* tile, const bf16* __restrict__ src, int ld, int valid, int d, int thread, int n_threads) {
     constexpr int PIECES = D / 8;
-    for (int i = threadIdx.x; i < CHUNK * PIECES; i += n_threads) {
+#pragma unroll 4
+    for (int i = thread; i < CHUNK * PIECES; i += n_threads) {
         const int row = i / PIECES, piece = i % PIECES;
         const bool in = row < valid && piece * 8 < d;
-        cp_async_16(reinterpret_cast<uint4*>(tile) + swz<D>(row, piece), src + (in ? (size_t)row * ld + piece * 8 : 0), in);
+        cp_async_16(reinterpret_cast<uint4*>(tile) + swz<D>(row, piece), src + (in ? row * ld + piece * 8 : 0), in);
     }
 }
 
@@ -106,8 +108,8 @@ __global__ void __launch_bounds__(INNER_THREADS) delta_inner_kernel(
     if (first >= len) return;
     const int n = min(CHUNK, len - first), tok0 = t0 + first;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    stage_rows<D>(qs, q + ((size_t)tok0 * n_kv + hk) * d, (long long)n_kv * d, n, d, INNER_THREADS);
-    stage_rows<D>(ks, k + ((size_t)tok0 * n_kv + hk) * d, (long long)n_kv * d, n, d, INNER_THREADS);
+    stage_rows<D>(qs, q + ((size_t)tok0 * n_kv + hk) * d, n_kv * d, n, d, tid, INNER_THREADS);
+    stage_rows<D>(ks, k + ((size_t)tok0 * n_kv + hk) * d, n_kv * d, n, d, tid, INNER_THREADS);
     cp_async_commit();
     if (tid < CHUNK) {
         const bool in = tid < n;
@@ -192,200 +194,259 @@ __global__ void __launch_bounds__(INNER_THREADS) delta_inner_kernel(
     }
 }
 
-template <int D, int NW>
-struct WalkStage {
-    bf16 k[CHUNK * D], q[CHUNK * D];
-    bf16 work[WORK_BF16];
-    bf16 v[CHUNK * (NW * 16 + 8)];
-    float factors[WORK_F32];
+constexpr int STRIP = 16;  // value columns of a block of the walk
+constexpr int WALK_THREADS = 256;
+
+template <int D>
+struct WalkSmem {
+    struct Stage {
+        bf16 k[CHUNK * D], q[CHUNK * D];
+        bf16 work[WORK_BF16];
+        bf16 v[CHUNK * (STRIP + 8)];
+        float factors[WORK_F32];
+    } stage[2];
+    // what the warps hand one another, each as a rounded half and a rest, rows of value columns
+    bf16 state[2][STRIP][D + 8];          // S^T before the chunk
+    bf16 rest[2][STRIP][CHUNK + 8];       // v less its prediction
+    bf16 u[2][STRIP][CHUNK + 8];          // u
+    bf16 scaled[2][STRIP][CHUNK + 8];     // u times e^(c_last - c) a
 };
 
-// NW warps of 16 value columns each.
-template <int D, int NW>
-__global__ void __launch_bounds__(NW * 32) delta_walk_kernel(
+// the left operand's four registers for the 16 entries from k0 on
+__device__ __forceinline__ void left_operand(uint32_t (&a)[4], const bf16* rows, int ld, int k0, int lane) {
+    ldmatrix_x4(a, rows + ((lane & 7) + (((lane >> 3) & 1) << 3)) * ld + k0 + ((lane >> 4) << 3));
+}
+
+// Four warps (`walk`) carry the state, each a quarter of the key entries and 16 of a chunk's tokens; four more (`read`) form the
+// read-outs of 16 tokens each beside them.
+template <int D>
+__global__ void __launch_bounds__(WALK_THREADS) delta_walk_kernel(
     const bf16* __restrict__ q, const bf16* __restrict__ k, const bf16* __restrict__ v, const bf16* __restrict__ work,
     const float* __restrict__ factors, float* __restrict__ state /* [slots, H, d, dv] */, float* __restrict__ out /* [T, H, dv] */,
     const int* __restrict__ cu_q, const int* __restrict__ slots, int n_heads, int n_kv, int d, int dv, int chunk0, int wave) {
-    constexpr int NT = NW * 32, V_LD = NW * 16 + 8;
+    constexpr int V_LD = STRIP + 8, SD = D + 8, CD = CHUNK + 8, OWN = D / 4;
     extern __shared__ __align__(128) unsigned char smem_raw[];
-    WalkStage<D, NW>* stages = reinterpret_cast<WalkStage<D, NW>*>(smem_raw);
+    WalkSmem<D>& sm = *reinterpret_cast<WalkSmem<D>*>(smem_raw);
     pdl_launch_dependents();
-    const int head = blockIdx.y, seq = blockIdx.z, hk = head / (n_heads / n_kv), v0 = blockIdx.x * NW * 16;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int head = blockIdx.y, seq = blockIdx.z, hk = head / (n_heads / n_kv), v0 = blockIdx.x * STRIP;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = warp & 3;
+    const bool walks = warp < 4;
     pdl_wait();
     const int t0 = cu_q[seq], len = cu_q[seq + 1] - t0;
     const int here = min(wave, (len + CHUNK - 1) / CHUNK - chunk0);
     if (here <= 0) return;
-    auto issue = [&](int i) {
+    // the tiles of chunk i, by n_threads threads of which this is the thread-th
+    auto issue = [&](int i, int thread, int n_threads) {
         if (i < here) {
-            WalkStage<D, NW>& st = stages[i & 1];
+            auto& st = sm.stage[i & 1];
             const int first = (chunk0 + i) * CHUNK, n = min(CHUNK, len - first);
             const size_t tok0 = (size_t)(t0 + first);
             const size_t unit = ((size_t)seq * wave + i) * n_heads + head;
-            stage_rows<D>(st.k, k + (tok0 * n_kv + hk) * d, (long long)n_kv * d, n, d, NT);
-            stage_rows<D>(st.q, q + (tok0 * n_kv + hk) * d, (long long)n_kv * d, n, d, NT);
-            for (int p = threadIdx.x; p < WORK_BF16 / 8; p += NT) cp_async_16(st.work + p * 8, work + unit * WORK_BF16 + p * 8, true);
-            for (int p = threadIdx.x; p < WORK_F32 / 4; p += NT) cp_async_16(st.factors + p * 4, factors + unit * WORK_F32 + p * 4, true);
-            for (int p = threadIdx.x; p < CHUNK * NW * 2; p += NT) {
-                const int row = p / (NW * 2), col = (p % (NW * 2)) * 8;
+            stage_rows<D>(st.k, k + (tok0 * n_kv + hk) * d, n_kv * d, n, d, thread, n_threads);
+            stage_rows<D>(st.q, q + (tok0 * n_kv + hk) * d, n_kv * d, n, d, thread, n_threads);
+            const bf16* w = work + unit * WORK_BF16;
+#pragma unroll 4
+            for (int p = thread; p < WORK_BF16 / 8; p += n_threads) {
+                const int row = (p >> 3) & (CHUNK - 1), piece = (p & 7) ^ (row & 7);  // M and P are lower triangular
+                if (piece < 2 * (row / 16 + 1)) cp_async_16(st.work + p * 8, w + p * 8, true);
+            }
+            if (thread < WORK_F32 / 4) cp_async_16(st.factors + thread * 4, factors + unit * WORK_F32 + thread * 4, true);
+            if (thread < CHUNK * 2) {
+                const int row = thread >> 1, col = (thread & 1) * 8;
                 const bool in = row < n && v0 + col < dv;
                 cp_async_16(st.v + row * V_LD + col, v + (in ? (tok0 + row) * n_heads * dv + (size_t)head * dv + v0 + col : 0), in);
             }
         }
         cp_async_commit();
     };
-    issue(0);
-    // S^T: rows are the warp's value columns, columns the key entries
-    const int vrow = v0 + warp * 16 + (lane >> 2), kcol = (lane & 3) * 2;
+    issue(0, threadIdx.x, WALK_THREADS);
+    const int vrow = lane >> 2, pair = (lane & 3) * 2;                               // an accumulator's row and first column
+    const int brow = (lane & 7) + ((lane >> 4) << 3), bpiece = (lane >> 3) & 1;      // operand rows of [n][k] tiles
+    const int trow = (lane & 7) + (((lane >> 3) & 1) << 3), tpiece = lane >> 4;      // of [k][n] tiles, transposed on the way
     float* mine = state + ((size_t)slots[seq] * n_heads + head) * (size_t)d * dv;
-    float S[D / 8][4];
+    float S[OWN / 8][4];  // S^T: rows value columns, columns the warp's key entries
+    auto publish_state = [&]() {
 #pragma unroll
-    for (int nt = 0; nt < D / 8; ++nt)
+        for (int nt = 0; nt < OWN / 8; ++nt)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int row = vrow + 8 * (i >> 1), col = nt * 8 + kcol + (i & 1);
-            S[nt][i] = row < dv && col < d ? mine[(size_t)col * dv + row] : 0.f;
-        }
-    const int brow = (lane & 7) + ((lane >> 4) << 3), bpiece = (lane >> 3) & 1;     // operand rows of [n][k] tiles
-    const int trow = (lane & 7) + (((lane >> 3) & 1) << 3), tpiece = lane >> 4;     // of [k][n] tiles, transposed on the way
+            for (int h = 0; h < 2; ++h) {
+                uint32_t hi, lo;
+                split2(S[nt][2 * h], S[nt][2 * h + 1], hi, lo);
+                const int col = part * OWN + nt * 8 + pair;
+                *reinterpret_cast<uint32_t*>(&sm.state[0][vrow + 8 * h][col]) = hi;
+                *reinterpret_cast<uint32_t*>(&sm.state[1][vrow + 8 * h][col]) = lo;
+            }
+    };
+    if (walks) {
+#pragma unroll
+        for (int nt = 0; nt < OWN / 8; ++nt)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int row = v0 + vrow + 8 * (i >> 1), col = part * OWN + nt * 8 + pair + (i & 1);
+                S[nt][i] = row < dv && col < d ? mine[(size_t)col * dv + row] : 0.f;
+            }
+        publish_state();
+    }
+    const int tok = part * 16;  // the warp's tokens of a chunk
     for (int i = 0; i < here; ++i) {
-        issue(i + 1);
-        cp_async_wait<1>();
-        __syncthreads();
-        const WalkStage<D, NW>& st = stages[i & 1];
-        float U[8][4], O[8][4];
+        cp_async_wait<0>();
+        __syncthreads();  // the chunk's tiles and the state before it are there; the other stage is free
+        const auto& st = sm.stage[i & 1];
+        // S0^T K^T (walk) or S0^T Q^T (read) for the warp's tokens; the two halves of the state add up on their own
+        const bf16* rows = walks ? st.k : st.q;
+        float acc[2][4], low[2][4];
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
+        for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) U[nt][e] = O[nt][e] = 0.f;
-        // S0^T K^T and S0^T Q^T
+            for (int e = 0; e < 4; ++e) acc[nt][e] = low[nt][e] = 0.f;
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks) {
-            uint32_t hi[4], lo[4];
-            split2(S[2 * ks][0], S[2 * ks][1], hi[0], lo[0]);
-            split2(S[2 * ks][2], S[2 * ks][3], hi[1], lo[1]);
-            split2(S[2 * ks + 1][0], S[2 * ks + 1][1], hi[2], lo[2]);
-            split2(S[2 * ks + 1][2], S[2 * ks + 1][3], hi[3], lo[3]);
-#pragma unroll
-            for (int g = 0; g < 4; ++g) {
-                uint32_t bk[4], bq[4];
-                ldmatrix_x4(bk, reinterpret_cast<const uint4*>(st.k) + swz<D>(g * 16 + brow, ks * 2 + bpiece));
-                ldmatrix_x4(bq, reinterpret_cast<const uint4*>(st.q) + swz<D>(g * 16 + brow, ks * 2 + bpiece));
-                mma_16816(U[2 * g], hi, bk[0], bk[1]);
-                mma_16816(U[2 * g + 1], hi, bk[2], bk[3]);
-                mma_16816(O[2 * g], hi, bq[0], bq[1]);
-                mma_16816(O[2 * g + 1], hi, bq[2], bq[3]);
-                mma_16816(U[2 * g], lo, bk[0], bk[1]);
-                mma_16816(U[2 * g + 1], lo, bk[2], bk[3]);
-                mma_16816(O[2 * g], lo, bq[0], bq[1]);
-                mma_16816(O[2 * g + 1], lo, bq[2], bq[3]);
-            }
+            uint32_t hi[4], lo[4], b[4];
+            left_operand(hi, &sm.state[0][0][0], SD, ks * 16, lane);
+            left_operand(lo, &sm.state[1][0][0], SD, ks * 16, lane);
+            ldmatrix_x4(b, reinterpret_cast<const uint4*>(rows) + swz<D>(tok + brow, ks * 2 + bpiece));
+            mma_16816(acc[0], hi, b[0], b[1]);
+            mma_16816(acc[1], hi, b[2], b[3]);
+            mma_16816(low[0], lo, b[0], b[1]);
+            mma_16816(low[1], lo, b[2], b[3]);
         }
-        // v less its prediction, split into the left operand of the product with M; the read-outs from before the chunk
-        uint32_t yh[4][4], yl[4][4];
+        const float* f = st.factors + (walks ? 0 : CHUNK) + tok + pair;
+        const float2 f0 = *reinterpret_cast<const float2*>(f), f1 = *reinterpret_cast<const float2*>(f + 8);
+        const float fs[2][2] = {{f0.x, f0.y}, {f1.x, f1.y}};
 #pragma unroll
-        for (int g = 0; g < 4; ++g) {
-            uint32_t vt[4];  // (tokens 0-7, columns 0-7), (0-7, 8-15), (8-15, 0-7), (8-15, 8-15) of the group, transposed
-            ldmatrix_x4_trans(vt, st.v + (g * 16 + (lane & 7) + ((lane >> 4) << 3)) * V_LD + warp * 16 + ((lane >> 3) & 1) * 8);
+        for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int nt = 2 * g + half;
-                const float2 ez = *reinterpret_cast<const float2*>(st.factors + nt * 8 + kcol);
-                const float2 eq = *reinterpret_cast<const float2*>(st.factors + CHUNK + nt * 8 + kcol);
-                const float2 va = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&vt[2 * half]));
-                const float2 vb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&vt[2 * half + 1]));
-                split2(fmaf(-ez.x, U[nt][0], va.x), fmaf(-ez.y, U[nt][1], va.y), yh[g][2 * half], yl[g][2 * half]);
-                split2(fmaf(-ez.x, U[nt][2], vb.x), fmaf(-ez.y, U[nt][3], vb.y), yh[g][2 * half + 1], yl[g][2 * half + 1]);
-                O[nt][0] *= eq.x, O[nt][1] *= eq.y, O[nt][2] *= eq.x, O[nt][3] *= eq.y;
-            }
+            for (int e = 0; e < 4; ++e) acc[nt][e] = (acc[nt][e] + low[nt][e]) * fs[nt][e & 1];
+        if (walks) {  // v less its prediction
+            uint32_t vt[4];  // transposed: (tokens 0-7, columns 0-7), (0-7, 8-15), (8-15, 0-7), (8-15, 8-15)
+            ldmatrix_x4_trans(vt, st.v + (tok + (lane & 7) + ((lane >> 4) << 3)) * V_LD + ((lane >> 3) & 1) * 8);
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int h = 0; h < 2; ++h) {
+                    const float2 val = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&vt[2 * nt + h]));
+                    uint32_t hi, lo;
+                    split2(val.x - acc[nt][2 * h], val.y - acc[nt][2 * h + 1], hi, lo);
+                    *reinterpret_cast<uint32_t*>(&sm.rest[0][vrow + 8 * h][tok + nt * 8 + pair]) = hi;
+                    *reinterpret_cast<uint32_t*>(&sm.rest[1][vrow + 8 * h][tok + nt * 8 + pair]) = lo;
+                }
         }
-        // u: M is lower triangular, a group of tokens reads the groups up to its own
+        __syncthreads();
+        bf16(*u)[STRIP][CD] = sm.u;
+        if (walks) {  // u of the warp's tokens: M is lower triangular
+            float x[2][4], y[2][4];
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
+            for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) U[nt][e] = 0.f;
+                for (int e = 0; e < 4; ++e) x[nt][e] = y[nt][e] = 0.f;
 #pragma unroll
-        for (int ks = 0; ks < 4; ++ks)
-#pragma unroll
-            for (int g = ks; g < 4; ++g) {
-                uint32_t mh[4], ml[4];
-                const int at = swz<CHUNK>(g * 16 + brow, ks * 2 + bpiece);
+            for (int ks = 0; ks < 4; ++ks) {
+                if (ks > part) break;
+                uint32_t hi[4], lo[4], mh[4], ml[4];
+                left_operand(hi, &sm.rest[0][0][0], CD, ks * 16, lane);
+                left_operand(lo, &sm.rest[1][0][0], CD, ks * 16, lane);
+                const int at = swz<CHUNK>(tok + brow, ks * 2 + bpiece);
                 ldmatrix_x4(mh, reinterpret_cast<const uint4*>(st.work) + at);
                 ldmatrix_x4(ml, reinterpret_cast<const uint4*>(st.work + TILE) + at);
-                mma_16816(U[2 * g], yh[ks], mh[0], mh[1]);
-                mma_16816(U[2 * g + 1], yh[ks], mh[2], mh[3]);
-                mma_16816(U[2 * g], yl[ks], mh[0], mh[1]);
-                mma_16816(U[2 * g + 1], yl[ks], mh[2], mh[3]);
-                mma_16816(U[2 * g], yh[ks], ml[0], ml[1]);
-                mma_16816(U[2 * g + 1], yh[ks], ml[2], ml[3]);
+                mma_16816(x[0], hi, mh[0], mh[1]);
+                mma_16816(x[1], hi, mh[2], mh[3]);
+                mma_16816(y[0], lo, mh[0], mh[1]);
+                mma_16816(y[1], lo, mh[2], mh[3]);
+                mma_16816(y[0], hi, ml[0], ml[1]);
+                mma_16816(y[1], hi, ml[2], ml[3]);
             }
-        // the state behind the chunk
-        const float g_last = st.factors[3 * CHUNK];
+            const float2 e0 = *reinterpret_cast<const float2*>(st.factors + 2 * CHUNK + tok + pair);
+            const float2 e1 = *reinterpret_cast<const float2*>(st.factors + 2 * CHUNK + tok + 8 + pair);
+            const float es[2][2] = {{e0.x, e0.y}, {e1.x, e1.y}};
 #pragma unroll
-        for (int nt = 0; nt < D / 8; ++nt)
+            for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) S[nt][e] *= g_last;
-#pragma unroll
-        for (int ks = 0; ks < 4; ++ks) {
-            uint32_t hi[4], lo[4];
-#pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int nt = 2 * ks + half;
-                const float2 ek = *reinterpret_cast<const float2*>(st.factors + 2 * CHUNK + nt * 8 + kcol);
-                split2(U[nt][0] * ek.x, U[nt][1] * ek.y, hi[2 * half], lo[2 * half]);
-                split2(U[nt][2] * ek.x, U[nt][3] * ek.y, hi[2 * half + 1], lo[2 * half + 1]);
-            }
-#pragma unroll
-            for (int j = 0; j < D / 16; ++j) {
-                uint32_t bk[4];
-                ldmatrix_x4_trans(bk, reinterpret_cast<const uint4*>(st.k) + swz<D>(ks * 16 + trow, j * 2 + tpiece));
-                mma_16816(S[2 * j], hi, bk[0], bk[1]);
-                mma_16816(S[2 * j + 1], hi, bk[2], bk[3]);
-                mma_16816(S[2 * j], lo, bk[0], bk[1]);
-                mma_16816(S[2 * j + 1], lo, bk[2], bk[3]);
-            }
+                for (int h = 0; h < 2; ++h) {
+                    const float ux = x[nt][2 * h] + y[nt][2 * h], uy = x[nt][2 * h + 1] + y[nt][2 * h + 1];
+                    const int row = vrow + 8 * h, col = tok + nt * 8 + pair;
+                    uint32_t hi, lo;
+                    split2(ux, uy, hi, lo);
+                    *reinterpret_cast<uint32_t*>(&u[0][row][col]) = hi;
+                    *reinterpret_cast<uint32_t*>(&u[1][row][col]) = lo;
+                    split2(ux * es[nt][0], uy * es[nt][1], hi, lo);
+                    *reinterpret_cast<uint32_t*>(&sm.scaled[0][row][col]) = hi;
+                    *reinterpret_cast<uint32_t*>(&sm.scaled[1][row][col]) = lo;
+                }
+        } else {
+            issue(i + 1, threadIdx.x - WALK_THREADS / 2, WALK_THREADS / 2);  // these warps have nothing else to do here
         }
-        // the read-outs' part from inside the chunk
+        __syncthreads();
+        if (walks) {  // the state behind the chunk
+            const float g_last = st.factors[3 * CHUNK];
+            float y[OWN / 8][4];
 #pragma unroll
-        for (int ks = 0; ks < 4; ++ks) {
-            uint32_t hi[4], lo[4];
+            for (int nt = 0; nt < OWN / 8; ++nt)
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                split2(U[2 * ks + half][0], U[2 * ks + half][1], hi[2 * half], lo[2 * half]);
-                split2(U[2 * ks + half][2], U[2 * ks + half][3], hi[2 * half + 1], lo[2 * half + 1]);
+                for (int e = 0; e < 4; ++e) {
+                    S[nt][e] *= g_last;
+                    y[nt][e] = 0.f;
+                }
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks) {
+                uint32_t hi[4], lo[4];
+                left_operand(hi, &sm.scaled[0][0][0], CD, ks * 16, lane);
+                left_operand(lo, &sm.scaled[1][0][0], CD, ks * 16, lane);
+#pragma unroll
+                for (int j = 0; j < OWN / 16; ++j) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, reinterpret_cast<const uint4*>(st.k) + swz<D>(ks * 16 + trow, part * (OWN / 8) + j * 2 + tpiece));
+                    mma_16816(S[2 * j], hi, b[0], b[1]);
+                    mma_16816(S[2 * j + 1], hi, b[2], b[3]);
+                    mma_16816(y[2 * j], lo, b[0], b[1]);
+                    mma_16816(y[2 * j + 1], lo, b[2], b[3]);
+                }
             }
 #pragma unroll
-            for (int g = ks; g < 4; ++g) {
-                uint32_t ph[4], pl[4];
-                const int at = swz<CHUNK>(g * 16 + brow, ks * 2 + bpiece);
+            for (int nt = 0; nt < OWN / 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) S[nt][e] += y[nt][e];
+            publish_state();  // its readers of this chunk are behind two barriers
+        } else {  // the read-outs' part from inside the chunk
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) low[nt][e] = 0.f;
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks) {
+                if (ks > part) break;
+                uint32_t hi[4], lo[4], ph[4], pl[4];
+                left_operand(hi, &u[0][0][0], CD, ks * 16, lane);
+                left_operand(lo, &u[1][0][0], CD, ks * 16, lane);
+                const int at = swz<CHUNK>(tok + brow, ks * 2 + bpiece);
                 ldmatrix_x4(ph, reinterpret_cast<const uint4*>(st.work + 2 * TILE) + at);
                 ldmatrix_x4(pl, reinterpret_cast<const uint4*>(st.work + 3 * TILE) + at);
-                mma_16816(O[2 * g], hi, ph[0], ph[1]);
-                mma_16816(O[2 * g + 1], hi, ph[2], ph[3]);
-                mma_16816(O[2 * g], lo, ph[0], ph[1]);
-                mma_16816(O[2 * g + 1], lo, ph[2], ph[3]);
-                mma_16816(O[2 * g], hi, pl[0], pl[1]);
-                mma_16816(O[2 * g + 1], hi, pl[2], pl[3]);
+                mma_16816(acc[0], hi, ph[0], ph[1]);
+                mma_16816(acc[1], hi, ph[2], ph[3]);
+                mma_16816(low[0], lo, ph[0], ph[1]);
+                mma_16816(low[1], lo, ph[2], ph[3]);
+                mma_16816(low[0], hi, pl[0], pl[1]);
+                mma_16816(low[1], hi, pl[2], pl[3]);
             }
+            const int first = (chunk0 + i) * CHUNK, n = min(CHUNK, len - first);
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int t = tok + nt * 8 + pair + (e & 1), row = v0 + vrow + 8 * (e >> 1);
+                    if (t < n && row < dv) out[((size_t)(t0 + first + t) * n_heads + head) * dv + row] = acc[nt][e] + low[nt][e];
+                }
         }
-        const int first = (chunk0 + i) * CHUNK, n = min(CHUNK, len - first);
-#pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int t = nt * 8 + kcol + (e & 1), row = vrow + 8 * (e >> 1);
-                if (t < n && row < dv) out[((size_t)(t0 + first + t) * n_heads + head) * dv + row] = O[nt][e];
-            }
-        __syncthreads();  // the stage is free for the load after next
     }
     cp_async_wait<0>();
+    if (walks) {
 #pragma unroll
-    for (int nt = 0; nt < D / 8; ++nt)
+        for (int nt = 0; nt < OWN / 8; ++nt)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int row = vrow + 8 * (i >> 1), col = nt * 8 + kcol + (i & 1);
-            if (row < dv && col < d) mine[(size_t)col * dv + row] = S[nt][i];
-        }
+            for (int i = 0; i < 4; ++i) {
+                const int row = v0 + vrow + 8 * (i >> 1), col = part * OWN + nt * 8 + pair + (i & 1);
+                if (row < dv && col < d) mine[(size_t)col * dv + row] = S[nt][i];
+            }
+    }
 }
 
 }  // namespace
@@ -412,39 +473,27 @@ GK_EXPORT int gk_delta_chunked(const void* q, const void* k, const void* v, cons
         return gk_fail(GK_CUDA_ERROR, "delta_chunked: shared memory")
         GK_ATTR((delta_inner_kernel<64>), 2 * CHUNK * 64 * 2 + CHUNK * LDA * 4);
         GK_ATTR((delta_inner_kernel<128>), 2 * CHUNK * 128 * 2 + CHUNK * LDA * 4);
-        GK_ATTR((delta_walk_kernel<64, 1>), 2 * sizeof(WalkStage<64, 1>));
-        GK_ATTR((delta_walk_kernel<64, 2>), 2 * sizeof(WalkStage<64, 2>));
-        GK_ATTR((delta_walk_kernel<64, 4>), 2 * sizeof(WalkStage<64, 4>));
-        GK_ATTR((delta_walk_kernel<128, 1>), 2 * sizeof(WalkStage<128, 1>));
-        GK_ATTR((delta_walk_kernel<128, 2>), 2 * sizeof(WalkStage<128, 2>));
-        GK_ATTR((delta_walk_kernel<128, 4>), 2 * sizeof(WalkStage<128, 4>));
+        GK_ATTR((delta_walk_kernel<64>), sizeof(WalkSmem<64>));
+        GK_ATTR((delta_walk_kernel<128>), sizeof(WalkSmem<128>));
 #undef GK_ATTR
         prepared = true;
     }
     cudaStream_t s = (cudaStream_t)stream;
-    const int chunks = (max_len + CHUNK - 1) / CHUNK, strips = (dv + 15) / 16;
-    // few strips: a warp a block, so that every warp has a multiprocessor's tensor cores and loads for itself
-    const long long warps = (long long)strips * n_heads * n_seqs;
-    const int nw = warps <= 148 ? 1 : warps <= 296 ? 2 : 4;
+    const int chunks = (max_len + CHUNK - 1) / CHUNK, strips = (dv + STRIP - 1) / STRIP;
     for (int chunk0 = 0; chunk0 < chunks; chunk0 += wave) {
         const int here = chunks - chunk0 < wave ? chunks - chunk0 : wave;
 #define GK_INNER(D)                                                                                                                \
     gk_launch(delta_inner_kernel<D>, dim3(here, n_heads, n_seqs), dim3(INNER_THREADS), (size_t)2 * CHUNK * D * 2 + CHUNK * LDA * 4, s, \
               (const bf16*)q, (const bf16*)k, q_unit, k_unit, log_g, beta, (bf16*)work, factors, cu_q, n_heads, n_kv, d, chunk0, wave)
-#define GK_WALK(D, NW)                                                                                                               \
-    gk_launch(delta_walk_kernel<D, NW>, dim3((strips + NW - 1) / NW, n_heads, n_seqs), dim3(NW * 32), 2 * sizeof(WalkStage<D, NW>), s, \
-              (const bf16*)q, (const bf16*)k, (const bf16*)v, (const bf16*)work, (const float*)factors, state, out, cu_q, slots, n_heads,   \
-              n_kv, d, dv, chunk0, wave)
+#define GK_WALK(D)                                                                                                                 \
+    gk_launch(delta_walk_kernel<D>, dim3(strips, n_heads, n_seqs), dim3(WALK_THREADS), sizeof(WalkSmem<D>), s, (const bf16*)q, (const bf16*)k, \
+              (const bf16*)v, (const bf16*)work, (const float*)factors, state, out, cu_q, slots, n_heads, n_kv, d, dv, chunk0, wave)
         if (d <= 64) {
             GK_INNER(64);
-            if (nw == 1) GK_WALK(64, 1);
-            else if (nw == 2) GK_WALK(64, 2);
-            else GK_WALK(64, 4);
+            GK_WALK(64);
         } else {
             GK_INNER(128);
-            if (nw == 1) GK_WALK(128, 1);
-            else if (nw == 2) GK_WALK(128, 2);
-            else GK_WALK(128, 4);
+            GK_WALK(128);
         }
 #undef GK_WALK
 #undef GK_INNER

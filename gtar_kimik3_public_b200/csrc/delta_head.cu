@@ -33,6 +33,9 @@ __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
+// with the hardware's exponential and division, where the result is rounded to bfloat16
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
 struct HeadSizes {
     int n_heads, n_kv, d, dv, taps;
     __device__ __forceinline__ int qk() const { return n_kv * d; }
@@ -151,7 +154,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_head_prepare_kernel(
                     float y = w[TAPS - 1][e][x] * own[x];
 #pragma unroll
                     for (int j = 1; j < TAPS; ++j) y = fmaf(w[TAPS - 1 - j][e][x], past[j - 1][e][x], y);
-                    act[e][x] = silu_f(y);
+                    act[e][x] = ROUNDED ? silu_fast(y) : silu_f(y);
                 }
                 if constexpr (TAPS > 1) {
 #pragma unroll
@@ -173,7 +176,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_head_prepare_kernel(
                     for (int x = 0; x < VEC; ++x) y[x] = fmaf(wj[x], v[x], y[x]);
                 }
 #pragma unroll
-                for (int x = 0; x < VEC; ++x) act[e][x] = silu_f(y[x]);
+                for (int x = 0; x < VEC; ++x) act[e][x] = ROUNDED ? silu_fast(y[x]) : silu_f(y[x]);
             }
             if (is_qk) {
 #pragma unroll
@@ -230,7 +233,8 @@ __global__ void conv_ring_kernel(const T* __restrict__ proj, long long ld, float
 
 // One token a sequence.  A block per (head, sequence); NT threads as CG groups of 4 columns by NT / CG groups of rows, R rows
 // a thread.  Sums over the rows meet in shared memory in the order of the row groups.
-template <typename T, int NT, int CG, int R>
+// TAPS: 4, or 0 for any number of taps.
+template <typename T, int NT, int CG, int R, int TAPS>
 __global__ void __launch_bounds__(NT) delta_head_single_kernel(
     const T* __restrict__ proj, long long ld, const float* __restrict__ conv_w, float* ring, const float* __restrict__ a_log,
     const float* __restrict__ dt_bias, const float* __restrict__ norm_w, float* __restrict__ state /* [slots, H, d, dv] */,
@@ -250,6 +254,18 @@ __global__ void __launch_bounds__(NT) delta_head_single_kernel(
     const int group = sz.n_heads / sz.n_kv, hk = head / group;
     const int cg = threadIdx.x % CG, rg = threadIdx.x / CG, lane = threadIdx.x & 31;
     const bool live = cg * 4 < dv;
+    // the channels of the head's q, k and v: at most three a thread
+    constexpr int TURNS = 3;
+    auto channel = [&](int i) { return i < d ? hk * d + i : i < 2 * d ? sz.qk() + hk * d + (i - d) : 2 * sz.qk() + head * dv + (i - 2 * d); };
+    float w[TURNS][TAPS > 0 ? TAPS : 1];
+    if constexpr (TAPS > 0) {  // no kernel in flight writes the weights
+#pragma unroll
+        for (int n = 0; n < TURNS; ++n) {
+            const int i = n * NT + threadIdx.x;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) w[n][j] = i < 2 * d + dv ? conv_w[(size_t)(TAPS - 1 - j) * C + channel(i)] : 0.f;
+        }
+    }
     pdl_wait();
     const size_t slot = (size_t)slots[tok_seq[t]];
     const int pos = tok_pos[t];
@@ -263,18 +279,47 @@ __global__ void __launch_bounds__(NT) delta_head_single_kernel(
         if (live && row < d) load_vec<float, 4>(mine + (size_t)row * dv, S[r]);
     }
     const T* row_t = proj + (size_t)t * ld;
+    const T* gate = row_t + sz.gate_at() + (size_t)head * dv;
+    const float my_gate = (int)threadIdx.x < dv ? to_float(gate[threadIdx.x]) : 0.f;  // dv <= NT
+    const float my_weight = (int)threadIdx.x < dv ? norm_w[threadIdx.x] : 0.f;
     const float beta = sigmoid_f(to_float(row_t[sz.b_at() + head]));
     const float g = expf(-expf(a_log[head]) * softplus_f(to_float(row_t[sz.a_at() + head]) + dt_bias[head]));
     // the convolutions of the head's q, k and v; the first head of a group leaves q's and k's inputs in the ring
     float* ring_rows = ring + slot * taps * C;
     const bool owner = head % group == 0;
-    for (int i = threadIdx.x; i < 2 * d + dv; i += NT) {
-        const int c = i < d ? hk * d + i : i < 2 * d ? sz.qk() + hk * d + (i - d) : 2 * sz.qk() + head * dv + (i - 2 * d);
-        const float own = to_float(row_t[c]);
-        float y = conv_w[(size_t)(taps - 1) * C + c] * own;
-        for (int j = 1; j < taps && j <= pos; ++j) y = fmaf(conv_w[(size_t)(taps - 1 - j) * C + c], ring_rows[(size_t)((pos - j) % taps) * C + c], y);
-        if (taps > 1 && (owner || i >= 2 * d)) ring_rows[(size_t)(pos % taps) * C + c] = own;
-        (i < d ? sq[i] : i < 2 * d ? sk[i - d] : sv[i - 2 * d]) = silu_f(y);
+    if constexpr (TAPS > 0) {
+        float x[TURNS][TAPS];  // all inputs on their way before the first store to the ring
+#pragma unroll
+        for (int n = 0; n < TURNS; ++n) {
+            const int i = n * NT + threadIdx.x;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                x[n][j] = 0.f;
+                if (i < 2 * d + dv) {
+                    if (j == 0) x[n][j] = to_float(row_t[channel(i)]);
+                    else if (j <= pos) x[n][j] = ring_rows[(size_t)((pos - j) % TAPS) * C + channel(i)];
+                }
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < TURNS; ++n) {
+            const int i = n * NT + threadIdx.x;
+            if (i >= 2 * d + dv) continue;
+            float y = w[n][0] * x[n][0];
+#pragma unroll
+            for (int j = 1; j < TAPS; ++j) y = fmaf(w[n][j], x[n][j], y);
+            if (TAPS > 1 && (owner || i >= 2 * d)) ring_rows[(size_t)(pos % TAPS) * C + channel(i)] = x[n][0];
+            (i < d ? sq[i] : i < 2 * d ? sk[i - d] : sv[i - 2 * d]) = silu_f(y);
+        }
+    } else {
+        for (int i = threadIdx.x; i < 2 * d + dv; i += NT) {
+            const int c = channel(i);
+            const float own = to_float(row_t[c]);
+            float y = conv_w[(size_t)(taps - 1) * C + c] * own;
+            for (int j = 1; j < taps && j <= pos; ++j) y = fmaf(conv_w[(size_t)(taps - 1 - j) * C + c], ring_rows[(size_t)((pos - j) % taps) * C + c], y);
+            if (taps > 1 && (owner || i >= 2 * d)) ring_rows[(size_t)(pos % taps) * C + c] = own;
+            (i < d ? sq[i] : i < 2 * d ? sk[i - d] : sv[i - 2 * d]) = silu_f(y);
+        }
     }
     __syncthreads();
     float qq = 0.f, kk = 0.f, qk = 0.f;  // every warp forms the three sums for itself
@@ -333,9 +378,8 @@ __global__ void __launch_bounds__(NT) delta_head_single_kernel(
     for (int i = lane; i < dv; i += 32) ss = fmaf(so[i], so[i], ss);
     ss = warp_sum(ss);
     const float r = out_scale / sqrtf(ss / (float)dv + eps);
-    const T* gate = row_t + sz.gate_at() + (size_t)head * dv;
-    T* orow = out + (size_t)t * ld_out + (size_t)head * dv;
-    for (int i = threadIdx.x; i < dv; i += NT) orow[i] = from_float<T>(so[i] * r * norm_w[i] * silu_f(to_float(gate[i])));
+    if ((int)threadIdx.x < dv)
+        out[(size_t)t * ld_out + (size_t)head * dv + threadIdx.x] = from_float<T>(so[threadIdx.x] * r * my_weight * silu_f(my_gate));
 }
 
 bool sizes_ok(int n_heads, int n_kv, int d, int dv, int taps) {
@@ -449,9 +493,14 @@ GK_EXPORT int gk_delta_head_single(const void* proj, int dtype, long long ld, co
     const HeadSizes sz{n_heads, n_kv, d, dv, taps};
     cudaStream_t s = (cudaStream_t)stream;
     const size_t vectors = (size_t)(2 * ((d + 3) & ~3) + 2 * ((dv + 3) & ~3)) * sizeof(float);
-#define GK_SINGLE(NT, CG, R)                                                                                                          \
-    gk_launch(delta_head_single_kernel<T, NT, CG, R>, dim3(n_heads, n_tokens), dim3(NT), vectors + (size_t)NT * 8 * sizeof(float), s, \
+#define GK_SINGLE_AS(NT, CG, R, TAPS)                                                                                                       \
+    gk_launch(delta_head_single_kernel<T, NT, CG, R, TAPS>, dim3(n_heads, n_tokens), dim3(NT), vectors + (size_t)NT * 8 * sizeof(float), s, \
               (const T*)proj, ld, conv_w, ring, a_log, dt_bias, norm_w, state, tok_pos, tok_seq, slots, (T*)out, ld_out, out_scale, eps, sz)
+#define GK_SINGLE(NT, CG, R)                     \
+    do {                                         \
+        if (taps == 4) GK_SINGLE_AS(NT, CG, R, 4); \
+        else GK_SINGLE_AS(NT, CG, R, 0);         \
+    } while (0)
     GK_DISPATCH_DTYPE(dtype, T, {
         switch (shape) {
             case 1: GK_SINGLE(256, 8, 4); break;
@@ -465,6 +514,7 @@ GK_EXPORT int gk_delta_head_single(const void* proj, int dtype, long long ld, co
         }
     })
 #undef GK_SINGLE
+#undef GK_SINGLE_AS
     GK_CHECK_LAUNCH("delta_head_single");
     return GK_OK;
 }

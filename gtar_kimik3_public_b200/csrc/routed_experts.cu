@@ -72,6 +72,95 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_scores_kernel(const T*
         }
 }
 
+// The same for many bfloat16 tokens: a block has 16 tokens and 16 NJ rows of the router, the reduction in pieces of 64 entries
+// that come through a two-stage cp.async ring.  Its threads are four groups of 64 that take a quarter of every piece each, a
+// thread 4 tokens x NJ rows; the groups' sums meet at the end in their order.  A score depends on the token's row alone.
+constexpr int SCORE_K = 64, SCORE_ROWS = 16, SCORE_LDW = SCORE_K + 4, SCORE_LDH = SCORE_K + 8;
+
+__device__ __forceinline__ void score_copy16(void* smem, const void* gmem, bool in) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem), "r"(in ? 16 : 0) : "memory");
+}
+
+template <int NJ>
+__global__ void __launch_bounds__(256) route_scores_tiled_kernel(const __nv_bfloat16* __restrict__ h, const float* __restrict__ w_router,
+                                                                 float* __restrict__ z, int n_tokens, int width, int n_rows) {
+    constexpr int BN = 16 * NJ;
+    __shared__ __align__(16) float ws[2][BN * SCORE_LDW];
+    __shared__ __align__(16) __nv_bfloat16 hs[2][SCORE_ROWS * SCORE_LDH];
+    const int tid = threadIdx.x, kg = tid >> 6, eg = tid & 15, tg = (tid >> 4) & 3;
+    const int t0 = blockIdx.x * SCORE_ROWS, n0 = blockIdx.y * BN;
+    pdl_launch_dependents();
+    const int pieces = (width + SCORE_K - 1) / SCORE_K;
+    auto issue_weights = [&](int p) {
+        for (int i = tid; i < BN * (SCORE_K / 4); i += 256) {
+            const int row = i / (SCORE_K / 4), k = (i % (SCORE_K / 4)) * 4, at = p * SCORE_K + k;
+            const bool in = n0 + row < n_rows && at < width;
+            score_copy16(&ws[p & 1][row * SCORE_LDW + k], in ? w_router + (size_t)(n0 + row) * width + at : w_router, in);
+        }
+    };
+    auto issue_tokens = [&](int p) {
+        if (tid < SCORE_ROWS * (SCORE_K / 8)) {
+            const int row = tid / (SCORE_K / 8), k = (tid % (SCORE_K / 8)) * 8, at = p * SCORE_K + k;
+            const bool in = t0 + row < n_tokens && at < width;
+            score_copy16(&hs[p & 1][row * SCORE_LDH + k], in ? h + (size_t)(t0 + row) * width + at : h, in);
+        }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    issue_weights(0);  // no kernel in flight writes them
+    pdl_wait();
+    issue_tokens(0);
+    float acc[4][NJ];
+#pragma unroll
+    for (int a = 0; a < 4; ++a)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) acc[a][j] = 0.f;
+    for (int p = 0; p < pieces; ++p) {
+        asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        __syncthreads();
+        if (p + 1 < pieces) {
+            issue_weights(p + 1);
+            issue_tokens(p + 1);
+        }
+        const float* wp = &ws[p & 1][eg * SCORE_LDW + kg * 16];
+        const __nv_bfloat16* hp = &hs[p & 1][tg * 4 * SCORE_LDH + kg * 16];
+#pragma unroll
+        for (int k = 0; k < 16; k += 4) {
+            float x[4][4];
+#pragma unroll
+            for (int a = 0; a < 4; ++a) {
+                const uint2 raw = *reinterpret_cast<const uint2*>(hp + a * SCORE_LDH + k);
+                const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+                const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+                x[a][0] = lo.x, x[a][1] = lo.y, x[a][2] = hi.x, x[a][3] = hi.y;
+            }
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) {
+                const float4 w = *reinterpret_cast<const float4*>(wp + j * 16 * SCORE_LDW + k);
+#pragma unroll
+                for (int a = 0; a < 4; ++a) {
+                    acc[a][j] = fmaf(x[a][0], w.x, acc[a][j]);
+                    acc[a][j] = fmaf(x[a][1], w.y, acc[a][j]);
+                    acc[a][j] = fmaf(x[a][2], w.z, acc[a][j]);
+                    acc[a][j] = fmaf(x[a][3], w.w, acc[a][j]);
+                }
+            }
+        }
+        // the next turn's first barrier stands before anything is written into this stage again
+    }
+    __syncthreads();
+    float* sums = &ws[0][0];  // [4][SCORE_ROWS][BN]
+#pragma unroll
+    for (int a = 0; a < 4; ++a)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) sums[(kg * SCORE_ROWS + tg * 4 + a) * BN + eg + 16 * j] = acc[a][j];
+    __syncthreads();
+    for (int i = tid; i < SCORE_ROWS * BN; i += 256) {
+        const int t = t0 + i / BN, n = n0 + i % BN;
+        if (t < n_tokens && n < n_rows)
+            z[(size_t)t * n_rows + n] = ((sums[i] + sums[SCORE_ROWS * BN + i]) + sums[2 * SCORE_ROWS * BN + i]) + sums[3 * SCORE_ROWS * BN + i];
+    }
+}
+
 enum RouteFlags : int { ROUTE_LOGITS = 1, ROUTE_SOFTMAX = 2, ROUTE_GROUP_BEST = 4, ROUTE_RENORMALISE = 8 };
 
 // The choice from the scores: one warp per token.  z has n_scores = n_experts or n_experts + 1 entries a token; ids and
@@ -444,7 +533,17 @@ GK_EXPORT int gk_route_groups(const void* h, int dtype, const float* w_router, c
     const long long units = (long long)token_groups * ((n_scores + per_warp - 1) / per_warp);
     GK_REQUIRE(units / ROUTE_WARPS < 2147483647LL, "route_groups: too many tokens");
     const dim3 score_grid((unsigned)((units + ROUTE_WARPS - 1) / ROUTE_WARPS));
-    GK_DISPATCH_DTYPE(dtype, T, {
+    if (dtype == GK_BF16 && n_tokens >= 256 && width % 8 == 0 && (((uintptr_t)h | (uintptr_t)w_router) & 15) == 0) {
+        const int tiles = (n_scores + 63) / 64, nj = ((n_scores + tiles - 1) / tiles + 15) / 16;
+        const dim3 grid((n_tokens + SCORE_ROWS - 1) / SCORE_ROWS, tiles);
+#define GK_TILED(NJ) \
+    gk_launch(route_scores_tiled_kernel<NJ>, grid, dim3(256), 0, s, (const __nv_bfloat16*)h, w_router, z, n_tokens, width, n_scores)
+        if (nj == 1) GK_TILED(1);
+        else if (nj == 2) GK_TILED(2);
+        else if (nj == 3) GK_TILED(3);
+        else GK_TILED(4);
+#undef GK_TILED
+    } else GK_DISPATCH_DTYPE(dtype, T, {
         if (per_warp == 8)
             gk_launch(route_scores_kernel<T, 8, 4>, score_grid, dim3(ROUTE_WARPS * 32), 0, s, (const T*)h, w_router, z, n_tokens, width, n_scores);
         else

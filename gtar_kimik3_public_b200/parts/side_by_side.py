@@ -21,6 +21,10 @@ def _as_list(request) -> list:
     return list(request) if isinstance(request, (list, tuple)) else [request]
 
 
+def _up8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
 class SideBySide(Mixer):
     def __init__(self, left: Mixer, right: Mixer, left_scale: float = 1.0, right_scale: float = 1.0,
                  names: dict[str, str] | None = None):
@@ -47,7 +51,13 @@ class SideBySide(Mixer):
                 and self.left.w_o.dtype == self.right.w_o.dtype):
             self.right_at = self.left.w_in.shape[0]
             self.w_in = torch.cat([part.w_in for part in pair], dim=0).contiguous()
-            self.w_o = torch.cat([part.w_o for part in pair], dim=1).contiguous()
+            # each mixer's read-outs begin at a multiple of 8 columns; no read-out stands in the columns between
+            self.read_at = [0, _up8(self.left.out_columns)]
+            self.read_columns = self.read_at[1] + _up8(self.right.out_columns)
+            w_o = self.left.w_o.new_zeros((self.left.w_o.shape[0], self.read_columns))
+            for part, at in zip(pair, self.read_at):
+                w_o[:, at:at + part.out_columns] = part.w_o
+            self.w_o = w_o
             for part in pair:  # held here from now on
                 part.w_in = part.w_o = None
 
@@ -73,10 +83,10 @@ class SideBySide(Mixer):
         right_views = self._views(self.right.cache_request(), views)
         if self.w_in is not None:
             proj = linear(x, self.w_in)
-            split = self.left.out_columns
-            rows = torch.empty((ctx.n_tokens, split + self.right.out_columns), dtype=ctx.dtype, device=x.device)
-            self.left.core(proj, 0, ctx, left_views, rows, 0, self.left_scale)
-            self.right.core(proj, self.right_at, ctx, right_views, rows, split, self.right_scale)
+            gaps = self.read_columns > self.left.out_columns + self.right.out_columns
+            rows = (torch.zeros if gaps else torch.empty)((ctx.n_tokens, self.read_columns), dtype=ctx.dtype, device=x.device)
+            self.left.core(proj, 0, ctx, left_views, rows, self.read_at[0], self.left_scale)
+            self.right.core(proj, self.right_at, ctx, right_views, rows, self.read_at[1], self.right_scale)
             return linear(rows, self.w_o)
         left = self.left.forward(x, ctx, left_views)
         right = self.right.forward(x, ctx, right_views)
