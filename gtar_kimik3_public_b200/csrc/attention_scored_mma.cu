@@ -267,16 +267,20 @@ __global__ void __launch_bounds__(SC_WARPS * 32, (MORE == 2 && D == 64 && !PADDE
     }
 }
 
-// One warp per (token, query head): the parts' sums brought to one maximum and added.
-template <int DV, bool SIGMOID>
+// One warp per (token, query head) and 64 value columns: the parts' sums brought to one maximum and added.
+template <bool SIGMOID>
 __global__ void __launch_bounds__(128) attention_scored_join_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                                     __nv_bfloat16* __restrict__ out, long long n_items, int n_split,
                                                                     int n_q, int dv, long long ld_out, float out_scale) {
     pdl_launch_dependents();
     pdl_wait();
-    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    const int pieces = (dv + 63) / 64;
+    const long long unit = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    const long long item = unit / pieces;
     if (item >= n_items) return;
     const int lane = threadIdx.x & 31;
+    const int col = (int)(unit - item * pieces) * 64 + lane * 2;  // dv is even
+    const bool in = col < dv;
     // a lane has a part's maximum and sum (there are at most 32 parts)
     float share = 1.f, denom = 0.f;
     if (!SIGMOID) {
@@ -285,22 +289,19 @@ __global__ void __launch_bounds__(128) attention_scored_join_kernel(const float*
         share = ml.x == -INFINITY ? 0.f : exp2_fast(ml.x - top);
         denom = warp_sum(ml.y * share);
     }
-    float acc[DV / 32];
-#pragma unroll
-    for (int c = 0; c < DV / 32; ++c) acc[c] = 0.f;
-#pragma unroll 4
+    float2 acc = make_float2(0.f, 0.f);
+    const float* src = part_o + (size_t)item * dv + (in ? col : 0);
+    const size_t step = (size_t)n_items * dv;
+#pragma unroll 8
     for (int s = 0; s < n_split; ++s) {
         const float w = SIGMOID ? 1.f : __shfl_sync(0xffffffffu, share, s);
-        const float* src = part_o + ((size_t)s * n_items + item) * dv;
-#pragma unroll
-        for (int c = 0; c < DV / 32; ++c)
-            if (lane + 32 * c < dv) acc[c] = fmaf(src[lane + 32 * c], w, acc[c]);
+        const float2 x = *reinterpret_cast<const float2*>(src + (size_t)s * step);
+        acc.x = fmaf(x.x, w, acc.x);
+        acc.y = fmaf(x.y, w, acc.y);
     }
     const float inv = SIGMOID ? out_scale : out_scale / denom;
-    __nv_bfloat16* orow = out + (size_t)(item / n_q) * ld_out + (size_t)(item % n_q) * dv;
-#pragma unroll
-    for (int c = 0; c < DV / 32; ++c)
-        if (lane + 32 * c < dv) orow[lane + 32 * c] = __float2bfloat16(acc[c] * inv);
+    if (in)
+        *reinterpret_cast<uint32_t*>(out + (size_t)(item / n_q) * ld_out + (size_t)(item % n_q) * dv + col) = pack_bf16(acc.x * inv, acc.y * inv);
 }
 
 template <int D, int DV, bool PADDED, bool SIGMOID, int MORE, bool CAP>
@@ -326,8 +327,8 @@ int launch_scored(const void* q, const void* k_pages, const void* v_pages, void*
               out_scale);
     GK_CHECK_LAUNCH("attention_scored_mma");
     if (n_split > 1) {
-        const long long items = (long long)n_tokens * n_q;
-        gk_launch(attention_scored_join_kernel<DV, SIGMOID>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, (const float*)part_o,
+        const long long items = (long long)n_tokens * n_q, units = items * ((dv + 63) / 64);
+        gk_launch(attention_scored_join_kernel<SIGMOID>, dim3((unsigned)((units + 3) / 4)), dim3(128), 0, stream, (const float*)part_o,
                   (const float*)part_ml, (__nv_bfloat16*)out, items, n_split, n_q, dv, ld_out, out_scale);
         GK_CHECK_LAUNCH("attention_scored_join");
     }

@@ -30,6 +30,20 @@ namespace {
 constexpr int ROUTE_WARPS = 4;
 
 
+// four neighbouring numbers of a row (which start on four elements), zeros where `in` is false
+template <typename T>
+__device__ __forceinline__ void load_four(const T* p, bool in, float (&v)[4]) {
+    if constexpr (sizeof(T) == 4) {
+        const float4 x = in ? *reinterpret_cast<const float4*>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[0] = x.x, v[1] = x.y, v[2] = x.z, v[3] = x.w;
+    } else {
+        const uint2 raw = in ? *reinterpret_cast<const uint2*>(p) : make_uint2(0u, 0u);
+        const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        v[0] = lo.x, v[1] = lo.y, v[2] = hi.x, v[3] = hi.y;
+    }
+}
+
 // z[t, e] = h_t . w_router[e] in 32-bit.  One warp per (SCORE_TOKENS tokens, SCORE_EXPERTS experts): four and eight where
 // tokens are many (a router row is fetched once for four tokens; eight tokens a warp measured slower: 66 against 60 us
 // for 2,048 tokens of 1,024 and 32 experts), four and two where they are few and the launch would otherwise be a handful
@@ -51,6 +65,22 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_scores_kernel(const T*
     for (int a = 0; a < SCORE_TOKENS; ++a)
 #pragma unroll
         for (int j = 0; j < SCORE_EXPERTS; ++j) acc[a][j] = 0.f;
+    if (width % 4 == 0) {  // four neighbouring elements a lane and turn
+#pragma unroll 2
+        for (int i = lane * 4; i < width; i += 128) {
+            float xv[SCORE_TOKENS][4], wv[SCORE_EXPERTS][4];
+#pragma unroll
+            for (int a = 0; a < SCORE_TOKENS; ++a) load_four(h + (size_t)(t0 + a) * width + i, t0 + a < n_tokens, xv[a]);
+#pragma unroll
+            for (int j = 0; j < SCORE_EXPERTS; ++j) load_four(w_router + (size_t)(e0 + j) * width + i, e0 + j < n_experts, wv[j]);
+#pragma unroll
+            for (int a = 0; a < SCORE_TOKENS; ++a)
+#pragma unroll
+                for (int j = 0; j < SCORE_EXPERTS; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) acc[a][j] = fmaf(xv[a][e], wv[j][e], acc[a][j]);
+        }
+    } else
 #pragma unroll 4
     for (int i = lane; i < width; i += 32) {
         float xv[SCORE_TOKENS], wv[SCORE_EXPERTS];
@@ -260,45 +290,6 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_choose_kernel(
     }
 }
 
-template <typename TW>
-__device__ __forceinline__ float dot_smem(const float* __restrict__ x, const TW* __restrict__ w, int n, int lane);
-
-template <>
-__device__ __forceinline__ float dot_smem<float>(const float* __restrict__ x, const float* __restrict__ w, int n, int lane) {
-    float acc = 0.f;
-    if ((n & 3) == 0) {
-#pragma unroll 4
-        for (int i = lane * 4; i < n; i += 128) {
-            const float4 a = *reinterpret_cast<const float4*>(w + i);
-            acc = fmaf(x[i], a.x, acc); acc = fmaf(x[i + 1], a.y, acc); acc = fmaf(x[i + 2], a.z, acc); acc = fmaf(x[i + 3], a.w, acc);
-        }
-    } else {
-        for (int i = lane; i < n; i += 32) acc = fmaf(x[i], w[i], acc);
-    }
-    return warp_sum(acc);
-}
-
-template <>
-__device__ __forceinline__ float dot_smem<__nv_bfloat16>(const float* __restrict__ x, const __nv_bfloat16* __restrict__ w, int n, int lane) {
-    float acc = 0.f;
-    if ((n & 7) == 0) {
-#pragma unroll 4
-        for (int i = lane * 8; i < n; i += 256) {
-            const uint4 raw = *reinterpret_cast<const uint4*>(w + i);
-            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                const float2 f = __bfloat1622float2(p[c]);
-                acc = fmaf(x[i + 2 * c], f.x, acc);
-                acc = fmaf(x[i + 2 * c + 1], f.y, acc);
-            }
-        }
-    } else {
-        for (int i = lane; i < n; i += 32) acc = fmaf(x[i], __bfloat162float(w[i]), acc);
-    }
-    return warp_sum(acc);
-}
-
 // A lane's share of NR dot products of one vector in shared memory with NR rows in memory, summed in index order; the
 // rows' loads are independent, so all of them are on their way together.  The caller finishes each with warp_sum.
 template <typename TW, int NR>
@@ -335,6 +326,48 @@ __device__ __forceinline__ void dot_parts(const float* __restrict__ x, const TW*
             for (int j = 0; j < NR; ++j) acc[j] = fmaf(x[i], to_float(rows[j][i]), acc[j]);
     }
 }
+
+// The same for NR vectors in shared memory, x_stride apart, each with a row of its own.
+template <typename TW, int NR>
+__device__ __forceinline__ void dot_pairs(const float* __restrict__ x, int x_stride, const TW* const (&rows)[NR], int n, int lane, float (&acc)[NR]) {
+#pragma unroll
+    for (int j = 0; j < NR; ++j) acc[j] = 0.f;
+    constexpr int VEC = 16 / sizeof(TW);
+    if (n % VEC == 0) {
+#pragma unroll 2
+        for (int i = lane * VEC; i < n; i += 32 * VEC) {
+            uint4 raw[NR];
+#pragma unroll
+            for (int j = 0; j < NR; ++j) raw[j] = *reinterpret_cast<const uint4*>(rows[j] + i);
+#pragma unroll
+            for (int j = 0; j < NR; ++j) {
+                const float* xj = x + j * x_stride + i;
+                if constexpr (sizeof(TW) == 2) {
+                    const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw[j]);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) {
+                        const float2 f = __bfloat1622float2(p[c]);
+                        acc[j] = fmaf(xj[2 * c], f.x, acc[j]);
+                        acc[j] = fmaf(xj[2 * c + 1], f.y, acc[j]);
+                    }
+                } else {
+                    const float* f = reinterpret_cast<const float*>(&raw[j]);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) acc[j] = fmaf(xj[c], f[c], acc[j]);
+                }
+            }
+        }
+    } else {
+        for (int i = lane; i < n; i += 32)
+#pragma unroll
+            for (int j = 0; j < NR; ++j) acc[j] = fmaf(x[j * x_stride + i], to_float(rows[j][i]), acc[j]);
+    }
+}
+
+template <int N>
+struct Count {
+    static constexpr int value = N;
+};
 
 constexpr int UP_WARPS = 8;
 
@@ -395,18 +428,20 @@ __global__ void __launch_bounds__(UP_WARPS * 32) experts_down_kernel(
         float acc = add != nullptr ? to_float(add[(size_t)t * width + c]) : 0.f;
         if (add_weight != nullptr) acc *= add_weight[t];
         int kk = 0;
-        for (; kk + 1 < top; kk += 2) {  // two experts' rows in flight; the sum still takes them in the order they were chosen
-            const int e0 = ids[(size_t)t * top + kk], e1 = ids[(size_t)t * top + kk + 1];
-            const float d0 = dot_smem<TW>(as + (size_t)kk * ff, w_down + ((size_t)e0 * width + c) * ff, ff, lane);
-            const float d1 = dot_smem<TW>(as + (size_t)(kk + 1) * ff, w_down + ((size_t)e1 * width + c) * ff, ff, lane);
-            acc = fmaf(weights[(size_t)t * top + kk], d0, acc);
-            acc = fmaf(weights[(size_t)t * top + kk + 1], d1, acc);
-        }
-        if (kk < top) {
-            const int e = ids[(size_t)t * top + kk];
-            const float d = dot_smem<TW>(as + (size_t)kk * ff, w_down + ((size_t)e * width + c) * ff, ff, lane);
-            acc = fmaf(weights[(size_t)t * top + kk], d, acc);
-        }
+        auto add_pairs = [&](auto count) {  // their rows in flight together; the sum still takes them in the order they were chosen
+            constexpr int NR = decltype(count)::value;
+            const TW* rows[NR];
+            float part[NR];
+#pragma unroll
+            for (int j = 0; j < NR; ++j) rows[j] = w_down + ((size_t)ids[(size_t)t * top + kk + j] * width + c) * ff;
+            dot_pairs<TW, NR>(as + (size_t)kk * ff, ff, rows, ff, lane, part);
+#pragma unroll
+            for (int j = 0; j < NR; ++j) acc = fmaf(weights[(size_t)t * top + kk + j], warp_sum(part[j]), acc);
+            kk += NR;
+        };
+        while (kk + 4 <= top) add_pairs(Count<4>{});
+        if (kk + 2 <= top) add_pairs(Count<2>{});
+        if (kk < top) add_pairs(Count<1>{});
         if (lane == 0) out[(size_t)t * width + c] = acc;
     }
 }
