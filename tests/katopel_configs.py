@@ -72,7 +72,7 @@ KAT_A = model(300, 88, 0.01, 3.0, [
 KAT_B = model(257, 64, 0.004, None, [
     layer(pair(attention(4, 2, 64, 64, 0.125, chunk=64, rot=32), delta(2, 1, 64, 64, 4), 0.8, 0.4), moe(40, 4, 4, shared=40)),
     layer(delta(4, 4, 16, 16, 4), dense(96)),
-    layer(pair(attention(2, 1, 128, 128, 0.07, rot=128, base=500.0), delta(2, 2, 128, 32, 4), 1.1, 0.6), moe(32, 3, 3, shared=16)),
+    layer(pair(attention(2, 1, 128, 128, 0.07, rot=128, base=500.0), delta(2, 2, 128, 32, 4), 1.2, 0.55), moe(32, 3, 3, shared=16)),
 ], loop=(0, 3, 2))
 
 # values wider than keys, 128 and 256 among them; the last layer alone runs twice; a pass that is the only one

@@ -361,7 +361,7 @@ def _plain_chunked(q, k, v, scale, chunk):
 
 SIZES = [
     # H, G, d, dv, chunk
-    (6, 2, 16, 24, 17), (4, 1, 64, 128, 64), (2, 2, 40, 8, 65), (3, 1, 128, 256, 100), (4, 2, 96, 192, 50), (5, 1, 8, 64, 1),
+    (6, 2, 16, 24, 17), (4, 1, 64, 128, 64), (2, 2, 40, 8, 65), (3, 1, 128, 256, 100), (3, 1, 96, 200, 50), (5, 1, 8, 64, 1),
     (4, 2, 128, 64, 0), (2, 1, 72, 136, 200), (4, 4, 64, 64, 130), (2, 1, 128, 128, 33), (3, 1, 10, 14, 20), (8, 1, 64, 104, 128),
 ]
 
@@ -411,10 +411,10 @@ EDGES = [
     (0, 700, 63, True),      # the last place of the first page
     (0, 700, 64, True),      # the first place of the second
     (0, 700, 700, True),     # the token itself
-    (96, 671, 576, True),    # the last place of a chunk reads the first
-    (96, 671, 575, False),   # and not the one before it
-    (96, 672, 671, False),   # the first place of a chunk does not read its neighbour
-    (96, 672, 672, True),
+    (80, 639, 560, True),    # the last place of a chunk reads the first
+    (80, 639, 559, False),   # and not the one before it
+    (80, 640, 639, False),   # the first place of a chunk does not read its neighbour
+    (80, 640, 640, True),
     (64, 127, 64, True),     # chunks that are pages
     (64, 128, 127, False),
     (200, 399, 200, True),   # an edge in the middle of a page
@@ -433,7 +433,7 @@ EDGES = [
 
 
 @pytest.mark.parametrize("dtype,d,dv,parts", [(torch.float32, 16, 20, 0), (torch.bfloat16, 10, 14, 0), (torch.bfloat16, 64, 64, 4),
-                                              (torch.bfloat16, 96, 192, 1), (torch.bfloat16, 64, 128, 4), (torch.bfloat16, 128, 256, 4)])
+                                              (torch.bfloat16, 88, 176, 1), (torch.bfloat16, 64, 128, 4), (torch.bfloat16, 128, 256, 4)])
 @pytest.mark.parametrize("chunk,i,j,seen", EDGES)
 def test_chunked_attention_sees_one_key_or_not(dtype, d, dv, parts, chunk, i, j, seen):
     """Among hundreds of small keys one is made to stand out for the query at ``i`` (its score is large, its value is 100 in one

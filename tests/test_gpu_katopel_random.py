@@ -45,8 +45,8 @@ def drawn_config(rng: random.Random, all_chosen: bool) -> dict:
             vdim = dim if rng.random() < 0.4 else rng.choice([6, 10, 16, 48, 64, 80, 128, 256])
             left = attention(G * rng.choice([1, 2, 4, 5]), G, dim, vdim, rng.choice([1.0, 2.0, 0.5]) * dim ** -0.5,
                              chunk=rng.choice([None, 1, 2, 31, 64, 65, 100, 200]), rot=rng.choice([None, 2, 4, dim // 4 * 2, dim]),
-                             base=rng.choice([37.0, 1e4, 2.5e5]))
-            mixer = pair(left, drawn_delta(rng), rng.choice([None, 0.6, -1.2]), rng.choice([None, 1.1, 0.4]))
+                             base=rng.choice([37.0, 1e4, 3e5]))
+            mixer = pair(left, drawn_delta(rng), rng.choice([None, 0.65, -1.2]), rng.choice([None, 1.2, 0.4]))
         ff = rng.choice(["dense", "moe", "moe", None])
         if ff == "dense":
             mlp = dense(rng.choice([24, 50, 200]))
